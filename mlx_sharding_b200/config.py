@@ -21,7 +21,7 @@ MODEL_REMAPPING = {
     "mistral": "llama",  # reference utils.py:15
 }
 
-SUPPORTED_ARCHS = ("llama", "gemma2", "deepseek_v2", "perelorn", "gusolorn", "gifetar", "gokapel")
+SUPPORTED_ARCHS = ("llama", "gemma2", "deepseek_v2", "perelorn", "gusolorn", "gifetar", "gokapel", "podurax")
 
 
 @dataclass(frozen=True)
@@ -149,9 +149,9 @@ class ModelConfig:
     layer_specs: Optional[list] = None
     token_side_dim: int = 0
     logit_scale: float = 1.0
-    # gifetar: every sublayer's (normed) output enters the residual stream times this factor
+    # gifetar, gokapel, podurax: every sublayer's output enters the residual stream times this factor
     residual_mult: float = 1.0
-    # gokapel: number of residual streams (hyper-connections) and the factor on the embedding rows
+    # gokapel: number of residual streams (hyper-connections); gokapel, podurax: the factor on the embedding rows
     streams: int = 1
     embedding_scale: float = 1.0
     # quantisation (mlx affine) + sharding
@@ -172,6 +172,8 @@ class ModelConfig:
             d = _gifetar_flat(d)
         elif "model_type" not in d and str(d.get("architecture", "")).lower() == "gokapel":
             d = _gokapel_flat(d)
+        elif "model_type" not in d and str(d.get("architecture", "")).lower() == "podurax":
+            d = _podurax_flat(d)
         mt = d.get("model_type", "llama")
         if mt == "phi-msft":
             raise ValueError(
@@ -455,6 +457,62 @@ def gokapel_config(width=2048, vocab=32000, blocks=2, heads=16, kv_heads=4, dim=
                    dict(type="parallel", mixer=dict(par), mlp=dict(dense)), dict(type="parallel", mixer=dict(par), mlp=dict(moe))]
     d = dict(architecture="Gokapel", embedding=dict(scale=1.0), layers=layers, norm=dict(eps=1e-6), residual_mult=0.5, streams=streams,
              vocab=vocab, width=width)
+    d.update(overrides)
+    return d
+
+
+def _podurax_flat(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Podurax's nested config.json (``layers`` = list of {type, mixer, mlp}; ``norm.eps``; ``residual_mult``; ``embedding.scale``; ``vocab``;
+    ``width``) -> the flat fields of :class:`ModelConfig`.  Mixers: ``mamba1`` (inner, state, dt_rank, conv) and ``attention`` (heads,
+    kv_heads, dim, vdim, scale, optional rot.{base, dims, scaling.{factor, original, fast, slow}}, optional mask.{size, keep_first},
+    v_mix).  Feed-forward: ``dense`` (ff) or none.  Every size is read from the file."""
+    layers = [dict(type=str(L["type"]), mixer=dict(L["mixer"]), mlp=(dict(L["mlp"]) if L.get("mlp") else None)) for L in d["layers"]]
+    first = None                       # the layer whose values the later ``v_mix`` layers mix in
+    for i, L in enumerate(layers):
+        m = L["mixer"]
+        if L["type"] not in ("mamba1", "attention"):
+            raise ValueError(f"Podurax: unknown mixer type '{L['type']}'")
+        if L["mlp"] is not None and L["mlp"].get("kind", "dense") != "dense":
+            raise ValueError(f"Podurax: unknown feed-forward kind '{L['mlp'].get('kind')}'")
+        if L["type"] == "mamba1":
+            if min(int(m[k]) for k in ("inner", "state", "dt_rank", "conv")) < 1:
+                raise ValueError(f"Podurax layer {i}: inner, state, dt_rank and conv must be positive")
+            continue
+        if int(m["heads"]) % int(m["kv_heads"]) != 0:
+            raise ValueError(f"Podurax layer {i}: heads must be a multiple of kv_heads")
+        rot = m.get("rot") or {}
+        if int(rot.get("dims", 0)) % 2 != 0 or int(rot.get("dims", 0)) > int(m["dim"]):
+            raise ValueError(f"Podurax layer {i}: rot.dims must be even and at most dim")
+        mask = m.get("mask") or {}
+        if mask and (int(mask["size"]) < 1 or int(mask.get("keep_first", 0) or 0) < 0):
+            raise ValueError(f"Podurax layer {i}: mask.size must be positive, mask.keep_first must not be negative")
+        if m.get("v_mix"):
+            if first is None:
+                first = m
+            elif (int(m["kv_heads"]), int(m["vdim"])) != (int(first["kv_heads"]), int(first["vdim"])):
+                raise ValueError(f"Podurax layer {i}: v_mix layers must have the same kv_heads and vdim")
+    out = {k: v for k, v in d.items() if k not in ("architecture", "layers", "norm", "vocab", "width", "residual_mult", "embedding")}
+    ff = [L["mlp"]["ff"] for L in layers if L["mlp"]]
+    out.update(model_type="podurax", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               rms_norm_eps=float(d["norm"]["eps"]), layer_specs=layers, intermediate_size=int(max(ff)) if ff else 0,
+               residual_mult=float(d.get("residual_mult", 1.0)), embedding_scale=float((d.get("embedding") or {}).get("scale", 1.0)),
+               num_attention_heads=max([int(L["mixer"]["heads"]) for L in layers if L["type"] == "attention"], default=1))
+    return out
+
+
+def podurax_config(width=2048, vocab=32000, blocks=2, heads=16, kv_heads=4, dim=128, vdim=128, ff=8192, window=1024, keep_first=16, inner=None,
+                   state=16, dt_rank=None, **overrides) -> Dict[str, Any]:
+    """A Podurax config.json with layer sizes that resemble a real model: ``blocks`` x (selective scan, windowed attention, windowed
+    attention, selective scan), each with a dense feed-forward."""
+    scan = dict(conv=4, dt_rank=dt_rank or max(1, width // 16), inner=inner or 2 * width, state=state)
+    att = dict(dim=dim, heads=heads, kv_heads=kv_heads, mask=dict(keep_first=keep_first, size=window),
+               rot=dict(base=10000.0, dims=dim // 2, scaling=dict(factor=4.0, fast=32.0, original=4096, slow=1.0)), scale=dim ** -0.5, v_mix=True, vdim=vdim)
+    dense = dict(kind="dense", ff=ff)
+    one = lambda t, m: dict(type=t, mixer=dict(m), mlp=dict(dense))
+    layers = []
+    for _ in range(blocks):
+        layers += [one("mamba1", scan), one("attention", att), one("attention", att), one("mamba1", scan)]
+    d = dict(architecture="Podurax", embedding=dict(scale=1.0), layers=layers, norm=dict(eps=1e-6), residual_mult=0.5, vocab=vocab, width=width)
     d.update(overrides)
     return d
 

@@ -52,8 +52,14 @@ def llama_rope_spec(cfg: ModelConfig) -> RopeSpec:
     return RopeSpec(inv_freq=inv, rot_dim=dim, interleaved=bool(cfg.rope_traditional) and cfg.model_type != "deepseek_v2")
 
 
-def _yarn_find_correction_dim(num_rot, dim, base, max_pos):
-    return (dim * math.log(max_pos / (num_rot * 2 * math.pi))) / (2 * math.log(base))
+def yarn_inv_freq(dim: int, base: float, factor: float, original: float, fast: float, slow: float) -> torch.Tensor:
+    """YaRN frequencies of ``dim / 2`` rotary pairs (fp32, computed in fp64): pairs that turn more than ``fast`` times over ``original``
+    positions keep ``base^(-2i/dim)``, pairs that turn less than ``slow`` times are divided by ``factor``, a linear ramp in between."""
+    f = float(base) ** (-2.0 * torch.arange(dim // 2, dtype=torch.float64) / dim)
+    pair = lambda turns: (dim * math.log(original / (turns * 2 * math.pi))) / (2 * math.log(base))      # pair index that turns so often
+    low, high = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), dim - 1)
+    ramp = ((torch.arange(dim // 2, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0, 1)
+    return (f / factor * ramp + f * (1.0 - ramp)).float()
 
 
 def deepseek_rope_spec(cfg: ModelConfig) -> RopeSpec:
@@ -63,19 +69,10 @@ def deepseek_rope_spec(cfg: ModelConfig) -> RopeSpec:
     if not rs or rs.get("type", rs.get("rope_type")) not in ("yarn",):
         return RopeSpec(default_inv_freq(dim, base), dim, interleaved=True)
     factor = float(rs["factor"])
-    orig = float(rs.get("original_max_position_embeddings", 4096))
-    beta_fast, beta_slow = float(rs.get("beta_fast", 32)), float(rs.get("beta_slow", 1))
-    freq_extra = base ** (torch.arange(0, dim, 2, dtype=torch.float32) / dim)
-    freq_inter = factor * freq_extra
-    low = max(math.floor(_yarn_find_correction_dim(beta_fast, dim, base, orig)), 0)
-    high = min(math.ceil(_yarn_find_correction_dim(beta_slow, dim, base, orig)), dim - 1)
-    if low == high:
-        high += 0.001
-    ramp = ((torch.arange(dim // 2, dtype=torch.float32) - low) / (high - low)).clamp(0, 1)
-    mask = 1.0 - ramp
-    freqs = (freq_inter * freq_extra) / (freq_inter * mask + freq_extra * (1 - mask))
+    inv = yarn_inv_freq(dim, base, factor, float(rs.get("original_max_position_embeddings", 4096)), float(rs.get("beta_fast", 32)),
+                        float(rs.get("beta_slow", 1)))
     mscale = yarn_get_mscale(factor, rs.get("mscale", 1)) / yarn_get_mscale(factor, rs.get("mscale_all_dim", 0))
-    return RopeSpec(inv_freq=1.0 / freqs, rot_dim=dim, interleaved=True, mscale=float(mscale))
+    return RopeSpec(inv_freq=inv, rot_dim=dim, interleaved=True, mscale=float(mscale))
 
 
 # --------------------------------------------------------------------------------------------- base

@@ -38,20 +38,16 @@ from __future__ import annotations
 import torch
 
 from ..ops import BatchMeta, LinearWeight, RopeSpec
-from .base import StageModel
-from .perelorn import _pad_rows
+from .hybrid import HybridStage
 
 
-class GokapelStage(StageModel):
+class GokapelStage(HybridStage):
     arch = "gokapel"
     PREFILL_GEMM_MIN_ROWS = 32
     UNIT_EPS = 1e-6            # inside the root of the unit vectors of the delta rule (fixed by the design)
 
     def __init__(self, cfg, spec=None, dtype=torch.bfloat16, device="cpu", backend=None):
         super().__init__(cfg, spec, dtype, device, backend)
-        if not (self.spec.is_first and self.spec.is_last):
-            raise NotImplementedError("Gokapel runs as a single stage (fp32 residual streams: the pipeline hand-off does not carry them)")
-        self.specs = cfg.layer_specs
         self.seg = {}              # layer -> {segment name: (first column, width)} of its fused input projection
 
     # ---- cache geometry ---------------------------------------------------------------------------------------------
@@ -68,44 +64,10 @@ class GokapelStage(StageModel):
                             {"S": ((int(m["right"]["width"]),), torch.float32)}))
         return out
 
-    def kv_geometry(self):
-        raise NotImplementedError("hybrid stack: see cache_layout()")
-
     # ---- weights ----------------------------------------------------------------------------------------------------
-    def _lw(self, w: torch.Tensor, bias: torch.Tensor = None) -> LinearWeight:
-        """Linear weight ``[out, in]`` in the model dtype; output rows zero-padded to a multiple of 8 (GEMM tile rule), the real row
-        count kept in ``n_real``."""
-        lw = LinearWeight(weight=_pad_rows(w.to(device=self.device, dtype=self.dtype)))
-        if bias is not None:
-            lw.bias = _pad_rows(bias.to(device=self.device, dtype=self.dtype)[:, None])[:, 0].contiguous()
-        lw.n_real = w.shape[0]
-        return lw
-
-    def _fused(self, parts):
-        """One projection for several matrices that read the same input: ``parts`` = ``[(name, weight [rows, in], bias or None)]``.  Every
-        segment starts at a multiple of 8 columns (a later product may read it in place).  Returns ``(LinearWeight, {name: (col0, rows)})``."""
-        ws, bs, seg, col = [], [], {}, 0
-        any_bias = any(b is not None for _, _, b in parts)
-        for name, w, b in parts:
-            n = w.shape[0]
-            pad = (-n) % 8
-            seg[name] = (col, n)
-            ws.append(torch.cat([w, w.new_zeros(pad, w.shape[1])]) if pad else w)
-            if any_bias:
-                bb = b if b is not None else w.new_zeros(n)
-                bs.append(torch.cat([bb, bb.new_zeros(pad)]) if pad else bb)
-            col += n + pad
-        return self._lw(torch.cat(ws), torch.cat(bs) if any_bias else None), seg
-
-    def _f32(self, sd, key) -> torch.Tensor:
-        return sd.pop(key).to(device=self.device, dtype=torch.float32).contiguous()
-
     def _dyt(self, sd, key):
         """``(alpha, weight, bias)`` of a dynamic-tanh norm; the scalar is taken to the host once, at load."""
         return float(sd.pop(key + ".alpha").float()), self._f32(sd, key), self._f32(sd, key + ".b")
-
-    def sanitize(self, sd):
-        return dict(sd)
 
     def _sublayer_weights(self, sd, p, q, w):
         S, dev = int(self.cfg.streams), self.device
@@ -194,20 +156,11 @@ class GokapelStage(StageModel):
         return self
 
     # ---- forward ----------------------------------------------------------------------------------------------------
-    def _mm(self, x, W: LinearWeight, f32: bool = False, act: str = "none"):
-        y = self.ops.linear_any(x, W, torch.float32 if f32 else self.dtype, act)
-        return y if y.shape[1] == W.n_real else y[:, :W.n_real]
-
-    @staticmethod
-    def _cols(u, seg, name):
-        c0, n = seg[name]
-        return u[:, c0:c0 + n]
-
     def _channel_delta(self, w, m, ha, meta, st):
         """Returns ``(mixer output fp32 [T, width], gate logits of the gated residual or None)``."""
         O, eps, seg = self.ops, self.cfg.rms_norm_eps, w["seg"]
         H, G, D, V = (int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
-        u = self.ops.linear_any(ha, w["proj"], self.dtype)                            # [q k v | b | a1 | g1 | rg]
+        u = O.linear_any(ha, w["proj"], self.dtype)                            # [q k v | b | a1 | g1 | rg]
         C = 2 * G * D + H * V                                                        # q, k, v are adjacent: one convolution over all
         qkv = O.causal_conv_silu(u[:, :C], w["conv"], w["conv_b"], st["conv"], meta)
         dt = self._mm(self._cols(u, seg, "a1"), w["a2"], True)                        # fp32 raw step sizes [T, H * D]
@@ -221,7 +174,7 @@ class GokapelStage(StageModel):
         a = m["left"]
         H, D, V, R = int(a["heads"]), int(a["dim"]), int(a["vdim"]), int(m["right"]["width"])
         T = ha.shape[0]
-        u = self.ops.linear_any(ha, w["proj"], self.dtype)                            # [q | k | v | z | x | g | rg], biases added
+        u = O.linear_any(ha, w["proj"], self.dtype)                            # [q | k | v | z | x | g | rg], biases added
         q = O.qk_norm_rope_append(u, seg["q"][0], seg["k"][0], seg["v"][0], H, D, w["qn"], w["kn"], eps, w["inv_freq"], kpool, vpool, meta)
         both = torch.zeros(T, w["o_split"] + R, dtype=self.dtype, device=u.device) if w["o_split"] != H * V else \
             torch.empty(T, H * V + R, dtype=self.dtype, device=u.device)

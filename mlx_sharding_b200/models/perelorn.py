@@ -27,13 +27,7 @@ import torch
 
 from ..ops import BatchMeta, LinearWeight, RopeSpec
 from .base import StageModel
-
-
-def _pad_rows(w: torch.Tensor, mult: int = 8) -> torch.Tensor:
-    n = w.shape[0]
-    if n % mult == 0:
-        return w.contiguous()
-    return torch.cat([w, w.new_zeros((mult - n % mult, w.shape[1]))]).contiguous()
+from .hybrid import pad_rows as _pad_rows
 
 
 class PerelornStage(StageModel):

@@ -606,8 +606,8 @@ def latent_attention_prefill(q, pool, sink, meta: BatchMeta, scale: float, kv_ra
 from .reference import mlstm_col_block  # noqa: E402,F401  (a pure function of the value width: shared by both backends and the cache layout)
 
 
-def scaled_add_norm_(x, y, ls, w, eps: float, act_dtype, extra=None, extra_gate=None):
-    return C().hy_scaled_add_norm_(x, y, ls, w, float(eps), _is32(act_dtype), extra, extra_gate)
+def scaled_add_norm_(x, y, ls, w, eps: float, act_dtype, extra=None, extra_gate=None, mult: float = 1.0):
+    return C().hy_scaled_add_norm_(x, y, ls, w, float(eps), _is32(act_dtype), extra, extra_gate, float(mult))
 
 
 def mlstm_scan(qkv, gates, gate_bias, state: dict, meta: BatchMeta, heads: int, dim: int, vdim: int, cap: float, q_scale: float):
@@ -808,33 +808,49 @@ def delta_scan(qkv, beta, dt, dt_bias, A_log, state, meta: BatchMeta, heads: int
                              int(vdim), float(q_scale), float(unit_eps), int(meta.max_q_len))
 
 
-def qk_norm_rope_append(rows, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w, kn_w, eps: float, inv_freq, kpool, vpool, meta: BatchMeta):
+def qk_norm_rope_append(rows, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w, kn_w, eps: float, inv_freq, kpool, vpool, meta: BatchMeta,
+                        half: bool = False, norm_after: bool = False, rot_mult: float = 1.0, v_first=None, v_lambda: float = 0.0):
     return C().hy_qk_norm_rope_append(rows, int(q_col0), int(k_col0), int(v_col0), int(heads), int(dim), qn_w, kn_w, float(eps), inv_freq, kpool, vpool,
-                                      meta.slot_mapping, meta.positions)
+                                      meta.slot_mapping, meta.positions, bool(half), bool(norm_after), float(rot_mult), v_first, float(v_lambda))
+
+
+SINK_FLASH_MIN_ROWS = 16         # portions of at least so many tokens take the tensor-core kernel (64 query rows per CTA)
+
+
+def _sink_flash_ok(kpool, vpool, meta: BatchMeta, out, out_col0: int) -> bool:
+    return (kpool.dtype == torch.bfloat16 and meta.max_q_len >= SINK_FLASH_MIN_ROWS and C().hy_sink_flash_supported(kpool.shape[3], vpool.shape[3])
+            and (out is None or (out.stride(0) % 2 == 0 and out_col0 % 2 == 0)))
 
 
 def sink_attention(q, kpool, vpool, sink, meta: BatchMeta, scale: float, block: int = 0, window: int = 0, out_mult: float = 1.0, out_dtype=None,
-                   out=None, out_col0: int = 0):
+                   out=None, out_col0: int = 0, keep_first: int = 0, gate=None):
+    """bf16 steps with long portions: the tensor-core kernel on the whole ragged batch (``attention_prefill.cu``); decode steps, short
+    portions, exact mode and odd head sizes: ``sinkattn.cu``."""
+    if _sink_flash_ok(kpool, vpool, meta, out, out_col0):
+        return C().hy_sink_flash(q, kpool, vpool, sink, meta.block_tables, meta.context_lens, meta.cu_seqlens, float(scale), int(block), int(window),
+                                 float(out_mult), out, int(out_col0), int(keep_first), gate)
     return C().hy_sink_attention(q, kpool, vpool, sink, meta.block_tables, meta.positions, meta.cu_seqlens, float(scale), int(block), int(window),
-                                 float(out_mult), int(meta.max_ctx_len), out, int(out_col0))
+                                 float(out_mult), int(meta.max_ctx_len), out, int(out_col0), int(keep_first), gate)
 
 
 SINK_PREFILL_MIN_BLOCK = 256     # blocks of fewer positions: the products are too small to pay for their launches; the ragged kernel runs
 
 
 def sink_attention_prefill(q, kpool, vpool, sink, meta: BatchMeta, scale: float, block: int = 0, window: int = 0, out_mult: float = 1.0, out_dtype=None,
-                           out=None, out_col0: int = 0):
+                           out=None, out_col0: int = 0, keep_first: int = 0, gate=None):
     """:func:`sink_attention` for a step that holds ONE sequence with many query rows (a prompt or a portion of one), as matrix products per
     block of positions and key / value head ``g``: gather the sequence's cached keys ``K_g`` and values ``V_g`` from the first visible
     position on, then for every block that holds queries of this step ``S = Q K_g[block]^T`` (fp32 out) for the ``H / G`` query heads of the
     group at once, the causal softmax with the sink (``hy_sink_softmax``; all keys of the slice lie in the queries' own block, so no lower
     limit is needed), ``O = P V_g[block]``.  The products run on the tensor cores (tcgen05 GEMM; cuBLAS fp32 in exact mode); query rows go in
-    pieces so that a score matrix stays below 256 MB.  Sliding windows, blocks that are small or not a multiple of 8 positions: the kernel."""
+    pieces so that a score matrix stays below 256 MB.  Head sizes of the tensor-core kernel, sliding windows, kept first tokens, gates, blocks
+    that are small or not a multiple of 8 positions: :func:`sink_attention`."""
     T, H, D = q.shape
     P, G, page, _ = kpool.shape
     V, Rg, adt = vpool.shape[3], H // G, kpool.dtype
-    if window > 0 or meta.num_seqs != 1 or (block > 0 and (block % 8 != 0 or block < SINK_PREFILL_MIN_BLOCK)):
-        return sink_attention(q, kpool, vpool, sink, meta, scale, block, window, out_mult, out_dtype, out, out_col0)
+    if (_sink_flash_ok(kpool, vpool, meta, out, out_col0) or window > 0 or keep_first > 0 or gate is not None or meta.num_seqs != 1
+            or (block > 0 and (block % 8 != 0 or block < SINK_PREFILL_MIN_BLOCK))):
+        return sink_attention(q, kpool, vpool, sink, meta, scale, block, window, out_mult, out_dtype, out, out_col0, keep_first, gate)
     ctx = int(meta.max_ctx_len)
     ctx0 = ctx - T
     first = ctx0 // block * block if block > 0 else 0                # first position any query of this step sees
@@ -925,3 +941,18 @@ def moe_relu2_experts(x, idx, w, Wu: LinearWeight, Wd: LinearWeight):
             y[r0:r0 + n] = torch.matmul(h[r0:r0 + n], wd[e].t()).float()
         r0 += n
     return c.hy_gather_sum(y, pair_row, int(k), wts)
+
+
+# ---- selective scan with one step size per channel, GELU-GLU feed-forward (``ops/csrc/selscan.cu``; same functions as in ``ops/reference.py``)
+def selective_scan(x, dt_raw, dt_bias, A_log, bc, b_col0: int, c_col0: int, D, gate, state, meta: BatchMeta):
+    return C().hy_selective_scan(x, dt_raw, dt_bias, A_log, bc, int(b_col0), int(c_col0), D, gate, state, meta.cu_seqlens, meta.context_lens, _slots(meta),
+                                 int(meta.max_q_len))
+
+
+def gelu_gated_up(x, Wg: LinearWeight, Wu: LinearWeight):
+    """Both projections and the GELU-GLU in ONE tcgen05 GEMM (two accumulators in TMEM, activation in the epilogue); exact mode and odd
+    sizes: two cuBLAS products and the elementwise kernel."""
+    if _tc_ok(x, Wg.weight, Wu.weight):
+        return C().linear(x, Wg.weight, Wu.weight, None, None, ACT_IDS["gelu_tanh"], 0.0, False, None, 0, 0, 0)
+    lin = torch.nn.functional.linear
+    return C().hy_clamped_glu(lin(x, Wg.weight), lin(x, Wu.weight), 0.0, None, None, 2)

@@ -11,9 +11,14 @@
 // the FA-2 register pipeline (S accumulators are re-used as the A operand of PV); softmax is online in
 // registers with exp2.  NOTE: this is the legacy (HMMA) tensor path — the tcgen05/TMEM version of this
 // kernel is the planned replacement; the GEMMs that dominate prefill FLOPs already run on tcgen05.
+//
+// SINK form (attention of sinkattn.cu for long portions): keys visible inside blocks of positions or a sliding window beside kept first
+// tokens (only tiles with visible keys are walked), a sink that joins the softmax denominator, a gate per head, fp32 queries, and run-time
+// head sizes up to DK / DV (multiples of 8; the missing key columns are zeros).
 #include "kernels.h"
 #include "launch.h"
 #include "ptx.cuh"
+#include "sinkattn.h"
 
 namespace b200 {
 
@@ -40,13 +45,20 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* 
                : "r"(smem_u32(smem)));
 }
 
-template <int DK, int DV>
+struct SinkForm {                            // what the SINK form adds (unused otherwise)
+  const float* q32;                          // [T, heads, d]
+  const float* sink; const __nv_bfloat16* gate; long long ld_gate;
+  int d, v, block, window, keep;
+  float out_mult;
+};
+
+template <int DK, int DV, bool SINK>
 __global__ void __launch_bounds__(kThreads)
 flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long long q_ld_h,
                      const __nv_bfloat16* __restrict__ kpool, const __nv_bfloat16* __restrict__ vpool,
                      const int* __restrict__ block_tables, int max_blocks, const int* __restrict__ cu_seqlens,
                      const int* __restrict__ context_lens, int num_seqs, int q_heads, int kv_heads, int page, float scale_log2,
-                     __nv_bfloat16* __restrict__ out, long long o_ld_t) {
+                     __nv_bfloat16* __restrict__ out, long long o_ld_t, const SinkForm x) {
   pdl_sync();  // PDL: predecessor's writes visible; let the successor start its prologue
   constexpr int KS = DK + 8, VS = DV + 8;  // padded row strides (elements): (stride/2) % 32 == 4 -> conflict free
   extern __shared__ __align__(16) uint8_t smem_raw[];
@@ -70,7 +82,17 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   const int ctx_after = context_lens[seq];
   const int pos0 = ctx_after - qlen + q0;            // absolute position of the tile's first query
   const int kv_end = min(ctx_after, pos0 + rows);    // causal: keys 0 .. last query position
-  const int ntiles = (kv_end + kBN - 1) / kBN;
+  const int D = SINK ? x.d : DK, V = SINK ? x.v : DV;
+  // SINK: key tiles that hold visible keys: those of the kept first tokens in front of the window, then from the first window key on
+  auto first_key = [&](int p) {
+    int lo = x.block > 0 ? p / x.block * x.block : 0;
+    if (x.window > 0) lo = max(lo, p - x.window + 1);
+    return lo;
+  };
+  const int lo0 = SINK ? first_key(pos0) : 0;
+  const int nkept = SINK ? (min(x.keep, lo0) + kBN - 1) / kBN : 0, w0 = SINK ? max(nkept, lo0 / kBN) : 0;
+  const int ntiles = nkept + max(0, (kv_end + kBN - 1) / kBN - w0);
+  auto tile_at = [&](int i) { return SINK ? (i < nkept ? i : w0 + i - nkept) : i; };
   const int* bt = block_tables + (size_t)seq * max_blocks;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -79,15 +101,15 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   auto load_tile = [&](int j, int buf) {
     __nv_bfloat16* dK = sK + buf * kBN * KS;
     __nv_bfloat16* dV = sV + buf * kBN * VS;
-    constexpr int KC = DK / 8, VC = DV / 8;
+    const int KC = D / 8, VC = V / 8;
     for (int i = threadIdx.x; i < kBN * (KC + VC); i += kThreads) {
       const int r = i / (KC + VC), c = i % (KC + VC);
       int pos = j * kBN + r;
       if (pos >= kv_end) pos = kv_end - 1;  // clamp: masked later
       const size_t pg = bt[pos / page];
       const size_t row = (pg * kv_heads + hk) * page + (pos % page);
-      if (c < KC) cp_async16(dK + r * KS + c * 8, kpool + row * DK + c * 8);
-      else cp_async16(dV + r * VS + (c - KC) * 8, vpool + row * DV + (c - KC) * 8);
+      if (c < KC) cp_async16(dK + r * KS + c * 8, kpool + row * D + c * 8);
+      else cp_async16(dV + r * VS + (c - KC) * 8, vpool + row * V + (c - KC) * 8);
     }
     cp_async_commit();
   };
@@ -96,6 +118,26 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   uint32_t qa[DK / 16][4];
   {
     const int ra = warp * 16 + r_lo, rb = ra + 8;
+    if constexpr (SINK) {
+      const float* fa = x.q32 + ((size_t)(tok0 + ra) * q_heads + hq) * D;
+      const float* fb = fa + (size_t)8 * q_heads * D;
+      auto pair = [&](const float* p, bool ok, int c) {          // d is a multiple of 8: a pair is inside or outside as a whole
+        if (!ok || c >= D) return 0u;
+        const float2 f = *reinterpret_cast<const float2*>(p + c);
+        return pack_bf16(f.x, f.y);
+      };
+#pragma unroll
+      for (int ks = 0; ks < DK / 16; ++ks) {
+        qa[ks][0] = pair(fa, ra < rows, ks * 16 + c2);
+        qa[ks][1] = pair(fb, rb < rows, ks * 16 + c2);
+        qa[ks][2] = pair(fa, ra < rows, ks * 16 + 8 + c2);
+        qa[ks][3] = pair(fb, rb < rows, ks * 16 + 8 + c2);
+      }
+      if (D < DK) {                            // key columns behind d: zeros in both buffers (the copies never touch them)
+        const int pad = DK - D;
+        for (int i = threadIdx.x; i < 2 * kBN * pad; i += kThreads) sK[(i / pad) * KS + D + i % pad] = __float2bfloat16(0.f);
+      }
+    } else {
     const __nv_bfloat16* qra = q + (size_t)(tok0 + ra) * q_ld_t + (size_t)hq * q_ld_h;
     const __nv_bfloat16* qrb = q + (size_t)(tok0 + rb) * q_ld_t + (size_t)hq * q_ld_h;
 #pragma unroll
@@ -105,6 +147,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
       qa[ks][2] = ra < rows ? *reinterpret_cast<const uint32_t*>(qra + ks * 16 + 8 + c2) : 0u;
       qa[ks][3] = rb < rows ? *reinterpret_cast<const uint32_t*>(qrb + ks * 16 + 8 + c2) : 0u;
     }
+    }
   }
   float o[DV / 8][4];
 #pragma unroll
@@ -112,10 +155,11 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
   const int qpos_a = pos0 + warp * 16 + r_lo, qpos_b = qpos_a + 8;
 
-  load_tile(0, 0);
+  const int lo_a = SINK ? first_key(qpos_a) : 0, lo_b = SINK ? first_key(qpos_b) : 0;
+  load_tile(tile_at(0), 0);
   for (int j = 0; j < ntiles; ++j) {
     const int buf = j & 1;
-    if (j + 1 < ntiles) { load_tile(j + 1, buf ^ 1); cp_async_wait<1>(); }
+    if (j + 1 < ntiles) { load_tile(tile_at(j + 1), buf ^ 1); cp_async_wait<1>(); }
     else cp_async_wait<0>();
     __syncthreads();
     const __nv_bfloat16* tK = sK + buf * kBN * KS;
@@ -134,15 +178,16 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
       }
     }
     // ---- scale, causal mask, online softmax (base 2)
-    const int kbase = j * kBN;
+    const int kbase = tile_at(j) * kBN;
     float mx_a = m_a, mx_b = m_b;
 #pragma unroll
     for (int nt = 0; nt < kBN / 8; ++nt) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int kpos = kbase + nt * 8 + c2 + e;
-        s[nt][e] = (kpos <= qpos_a) ? s[nt][e] * scale_log2 : -INFINITY;
-        s[nt][2 + e] = (kpos <= qpos_b) ? s[nt][2 + e] * scale_log2 : -INFINITY;
+        const bool va = kpos <= qpos_a && (!SINK || kpos >= lo_a || kpos < x.keep), vb = kpos <= qpos_b && (!SINK || kpos >= lo_b || kpos < x.keep);
+        s[nt][e] = va ? s[nt][e] * scale_log2 : -INFINITY;
+        s[nt][2 + e] = vb ? s[nt][2 + e] * scale_log2 : -INFINITY;
         mx_a = fmaxf(mx_a, s[nt][e]);
         mx_b = fmaxf(mx_b, s[nt][2 + e]);
       }
@@ -183,21 +228,32 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   // ---- normalise and store
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 1); l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1); l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-  const float ia = l_a > 0.f ? 1.f / l_a : 0.f, ib = l_b > 0.f ? 1.f / l_b : 0.f;
   const int ra = warp * 16 + r_lo, rb = ra + 8;
+  float fa = 1.f, fb = 1.f;
+  if constexpr (SINK) {
+    if (x.sink != nullptr) { const float sk = x.sink[hq] * 1.4426950408889634f; l_a += exp2f(sk - m_a); l_b += exp2f(sk - m_b); }
+    fa = fb = x.out_mult;
+    if (x.gate != nullptr) {
+      auto sig = [&](int r) { return 1.f / (1.f + expf(-__bfloat162float(x.gate[(size_t)(tok0 + r) * x.ld_gate + hq]))); };
+      if (ra < rows) fa *= sig(ra);
+      if (rb < rows) fb *= sig(rb);
+    }
+  }
+  const float ia = l_a > 0.f ? fa / l_a : 0.f, ib = l_b > 0.f ? fb / l_b : 0.f;
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) {
+    if (SINK && i * 8 >= V) break;
     if (ra < rows)
-      *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + ra) * o_ld_t + (size_t)hq * DV + i * 8 + c2) = pack_bf16(o[i][0] * ia, o[i][1] * ia);
+      *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + ra) * o_ld_t + (size_t)hq * V + i * 8 + c2) = pack_bf16(o[i][0] * ia, o[i][1] * ia);
     if (rb < rows)
-      *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + rb) * o_ld_t + (size_t)hq * DV + i * 8 + c2) = pack_bf16(o[i][2] * ib, o[i][3] * ib);
+      *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + rb) * o_ld_t + (size_t)hq * V + i * 8 + c2) = pack_bf16(o[i][2] * ib, o[i][3] * ib);
   }
 }
 
 template <int DK, int DV>
 cudaError_t launch_prefill(const FlashPrefillArgs& a, cudaStream_t s) {
   constexpr int smem = 2 * kBN * ((DK + 8) + (DV + 8)) * 2;
-  auto kern = flash_prefill_kernel<DK, DV>;
+  auto kern = flash_prefill_kernel<DK, DV, false>;
   static bool configured = false;
   if (!configured) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -208,7 +264,24 @@ cudaError_t launch_prefill(const FlashPrefillArgs& a, cudaStream_t s) {
   (void)launch_pdl(kern, dim3(grid), dim3(kThreads), smem, s, static_cast<const __nv_bfloat16*>(a.q), a.q_ld_t, a.q_ld_h,
                                     static_cast<const __nv_bfloat16*>(a.kpool), static_cast<const __nv_bfloat16*>(a.vpool),
                                     a.block_tables, a.max_blocks, a.cu_seqlens, a.context_lens, a.num_seqs, a.q_heads, a.kv_heads,
-                                    a.page, a.scale * 1.4426950408889634f, static_cast<__nv_bfloat16*>(a.out), a.o_ld_t);
+                                    a.page, a.scale * 1.4426950408889634f, static_cast<__nv_bfloat16*>(a.out), a.o_ld_t, SinkForm{});
+  return cudaGetLastError();
+}
+
+template <int DK, int DV>
+cudaError_t launch_sink(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s) {
+  constexpr int smem = 2 * kBN * ((DK + 8) + (DV + 8)) * 2;
+  auto kern = flash_prefill_kernel<DK, DV, true>;
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return e;
+    configured = true;
+  }
+  const SinkForm x{a.q, a.sink, static_cast<const __nv_bfloat16*>(a.gate), a.ld_gate, a.D, a.V, a.block, a.window, a.keep, a.out_mult};
+  kern<<<dim3(max_tiles, a.H), kThreads, smem, s>>>(nullptr, 0, 0, static_cast<const __nv_bfloat16*>(a.kpool), static_cast<const __nv_bfloat16*>(a.vpool),
+                                                    a.block_tables, a.max_blocks, a.cu, context_lens, a.B, a.H, a.G, a.page, a.scale * 1.4426950408889634f,
+                                                    static_cast<__nv_bfloat16*>(a.out), a.ld_out, x);
   return cudaGetLastError();
 }
 
@@ -225,6 +298,16 @@ cudaError_t flash_prefill_launch(const FlashPrefillArgs& a, cudaStream_t s) {
   if (a.dk_ == 128 && a.dv_ == 128) return launch_prefill<128, 128>(a, s);
   if (a.dk_ == 64 && a.dv_ == 64) return launch_prefill<64, 64>(a, s);
   return cudaErrorNotSupported;
+}
+
+bool sink_flash_supported(int D, int V) { return D % 8 == 0 && V % 8 == 0 && D >= 8 && V >= 8 && D <= 192 && V <= 128; }
+
+cudaError_t sink_flash_launch(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s) {
+  if (!sink_flash_supported(a.D, a.V) || a.ld_out % 2 != 0 || a.keep < 0) return cudaErrorInvalidValue;
+  if (a.B == 0 || max_tiles == 0) return cudaSuccess;
+  if (a.D <= 64 && a.V <= 64) return launch_sink<64, 64>(a, context_lens, max_tiles, s);
+  if (a.D <= 128) return launch_sink<128, 128>(a, context_lens, max_tiles, s);
+  return launch_sink<192, 128>(a, context_lens, max_tiles, s);
 }
 
 }  // namespace b200

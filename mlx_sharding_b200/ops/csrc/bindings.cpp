@@ -12,6 +12,8 @@
 #include "kernels.h"
 #include "hybrid.h"
 #include "diffattn.h"
+#include "selscan.h"
+#include "sinkattn.h"
 #include "streams.h"
 
 namespace py = pybind11;
@@ -994,7 +996,7 @@ Tensor hy_sink_softmax(const Tensor& s, const c10::optional<Tensor>& sink, int64
 
 // x += (y + extra * sigmoid(gate)) * ls on the fp32 residual stream (in place); returns rms(x) * w in the activation type
 Tensor hy_scaled_add_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor>& ls, const Tensor& w, double eps, bool act_f32,
-                           const c10::optional<Tensor>& extra, const c10::optional<Tensor>& gate) {
+                           const c10::optional<Tensor>& extra, const c10::optional<Tensor>& gate, double mult) {
   check_f32c(x, "x"); check_f32c(w, "w"); check_rows(y, "y");
   TORCH_CHECK(y.is_cuda() && y.scalar_type() == torch::kFloat32 && x.dim() == 2 && y.size(0) == x.size(0) && y.size(1) == x.size(1) && w.numel() == x.size(1));
   const float* lsp = nullptr; const float* ep = nullptr; const float* gp = nullptr; long long lde = 0, ldg = 0;
@@ -1009,7 +1011,7 @@ Tensor hy_scaled_add_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor
   Tensor xa = torch::empty({x.size(0), x.size(1)}, x.options().dtype(act_type(act_f32)));
   if (x.size(0) == 0) return xa;
   LAUNCH_OK(b200::scaled_add_norm_launch(x.data_ptr<float>(), y.data_ptr<float>(), y.stride(0), lsp, ep, lde, gp, ldg, w.data_ptr<float>(), xa.data_ptr(),
-                                         act_f32, (int)x.size(1), (float)eps, (int)x.size(0), cur_stream()));
+                                         act_f32, (int)x.size(1), (float)eps, (float)mult, (int)x.size(0), cur_stream()));
   return xa;
 }
 
@@ -1270,64 +1272,137 @@ Tensor hy_mingru_scan(const Tensor& rows, int64_t z0, int64_t x0, int64_t g0, in
   return out;
 }
 
-Tensor hy_qk_norm_rope_append(const Tensor& rows, int64_t q0, int64_t k0, int64_t v0, int64_t H, int64_t D, const Tensor& qn, const Tensor& kn, double eps,
-                              const Tensor& inv_freq, Tensor kpool, Tensor vpool, const Tensor& slot_map, const Tensor& positions) {
-  check_act(rows, "rows"); check_rows(rows, "rows"); check_f32c(qn, "q norm"); check_f32c(kn, "k norm"); check_f32c(inv_freq, "inv_freq");
-  check_i32(slot_map, "slot_mapping"); check_i32(positions, "positions");
+// qn, kn, v_first optional
+Tensor hy_qk_norm_rope_append(const Tensor& rows, int64_t q0, int64_t k0, int64_t v0, int64_t H, int64_t D, const c10::optional<Tensor>& qn,
+                              const c10::optional<Tensor>& kn, double eps, const Tensor& inv_freq, Tensor kpool, Tensor vpool, const Tensor& slot_map,
+                              const Tensor& positions, bool half, bool norm_after, double rot_mult, const c10::optional<Tensor>& v_first, double lam) {
+  check_act(rows, "rows"); check_rows(rows, "rows"); check_f32c(inv_freq, "inv_freq"); check_i32(slot_map, "slot_mapping"); check_i32(positions, "positions");
+  if (qn.has_value()) { check_f32c(*qn, "q norm"); TORCH_CHECK(qn->numel() == D); }
+  if (kn.has_value()) { check_f32c(*kn, "k norm"); TORCH_CHECK(kn->numel() == D); }
   TORCH_CHECK(kpool.dim() == 4 && vpool.dim() == 4 && kpool.is_contiguous() && vpool.is_contiguous() && kpool.scalar_type() == rows.scalar_type() &&
               vpool.scalar_type() == rows.scalar_type() && kpool.size(0) == vpool.size(0) && kpool.size(1) == vpool.size(1) && kpool.size(2) == vpool.size(2) &&
               kpool.size(3) == D, "pools [pages, kv_heads, page, d] in the activation type");
   const int64_t T = rows.size(0), G = kpool.size(1), V = vpool.size(3), rot = 2 * inv_freq.numel();
   TORCH_CHECK(q0 >= 0 && k0 >= 0 && v0 >= 0 && q0 + H * D <= rows.size(1) && k0 + G * D <= rows.size(1) && v0 + G * V <= rows.size(1) && rot <= D &&
-              qn.numel() == D && kn.numel() == D && slot_map.numel() >= T && positions.numel() >= T);
+              slot_map.numel() >= T && positions.numel() >= T);
+  if (v_first.has_value()) {
+    check_rows(*v_first, "v_first");
+    TORCH_CHECK(v_first->is_cuda() && v_first->scalar_type() == rows.scalar_type() && v_first->size(0) == T && v_first->size(1) == G * V, "v_first must be [T, kv_heads * vdim]");
+  }
   const c10::cuda::CUDAGuard guard(rows.device());
   Tensor q = torch::empty({T, H, D}, rows.options().dtype(torch::kFloat32));
   if (T == 0) return q;
-  LAUNCH_OK(b200::qk_norm_rope_append_launch(rows.data_ptr(), rows.stride(0), (int)q0, (int)k0, (int)v0, (int)H, (int)G, (int)D, (int)V, qn.data_ptr<float>(),
-                                             kn.data_ptr<float>(), (float)eps, inv_freq.data_ptr<float>(), (int)rot, positions.data_ptr<int>(),
-                                             slot_map.data_ptr<int>(), (int)kpool.size(2), q.data_ptr<float>(), kpool.data_ptr(), vpool.data_ptr(), is_f32(rows),
-                                             (int)T, cur_stream()));
+  LAUNCH_OK(b200::qk_norm_rope_append_launch(rows.data_ptr(), rows.stride(0), (int)q0, (int)k0, (int)v0, (int)H, (int)G, (int)D, (int)V,
+                                             qn.has_value() ? qn->data_ptr<float>() : nullptr, kn.has_value() ? kn->data_ptr<float>() : nullptr, (float)eps,
+                                             inv_freq.data_ptr<float>(), (int)rot, positions.data_ptr<int>(), slot_map.data_ptr<int>(), (int)kpool.size(2),
+                                             q.data_ptr<float>(), kpool.data_ptr(), vpool.data_ptr(), is_f32(rows), half, norm_after, (float)rot_mult,
+                                             v_first.has_value() ? v_first->data_ptr() : nullptr, v_first.has_value() ? v_first->stride(0) : 0, (float)lam, (int)T,
+                                             cur_stream()));
   return q;
 }
 
-Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
-                         const Tensor& positions, const Tensor& cu, double scale, int64_t block, int64_t window, double out_mult, int64_t max_ctx,
-                         const c10::optional<Tensor>& out_, int64_t col0) {
-  check_f32c(q, "q"); check_i32(block_tables, "block_tables"); check_i32(positions, "positions"); check_i32(cu, "cu_seqlens");
+namespace {
+// the arguments both forms of the attention with a sink share; `out` is allocated when it is not given
+b200::SinkAttnArgs sink_args(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
+                             const Tensor& cu, double scale, int64_t block, int64_t window, int64_t keep, double out_mult, const c10::optional<Tensor>& gate,
+                             Tensor& out, const c10::optional<Tensor>& out_, int64_t col0) {
+  check_f32c(q, "q"); check_i32(block_tables, "block_tables"); check_i32(cu, "cu_seqlens");
   TORCH_CHECK(q.dim() == 3 && kpool.dim() == 4 && vpool.dim() == 4 && kpool.is_contiguous() && vpool.is_contiguous() && kpool.scalar_type() == vpool.scalar_type() &&
               kpool.size(1) == vpool.size(1) && kpool.size(2) == vpool.size(2) && kpool.size(3) == q.size(2),
               "q fp32 [T, heads, dim]; pools [pages, kv_heads, page, dim] / [pages, kv_heads, page, vdim]");
   check_act(kpool, "key pool");
-  const int64_t T = q.size(0), H = q.size(1), D = q.size(2), G = kpool.size(1), V = vpool.size(3);
-  TORCH_CHECK(H % G == 0 && V <= 512 && block >= 0 && window >= 0 && positions.numel() >= T, "attention with a sink: vdim <= 512");
-  if (sink.has_value()) { check_f32c(*sink, "sink"); TORCH_CHECK(sink->numel() == H); }
-  const c10::cuda::CUDAGuard guard(q.device());
-  Tensor out = out_.has_value() ? *out_ : torch::empty({T, H * V}, kpool.options());
+  const int64_t T = q.size(0), H = q.size(1), G = kpool.size(1), V = vpool.size(3);
+  TORCH_CHECK(H % G == 0 && block >= 0 && window >= 0 && keep >= 0 && block_tables.dim() == 2);
+  b200::SinkAttnArgs a{};
+  if (sink.has_value()) { check_f32c(*sink, "sink"); TORCH_CHECK(sink->numel() == H); a.sink = sink->data_ptr<float>(); }
+  if (gate.has_value()) {
+    check_rows(*gate, "gate");
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == kpool.scalar_type() && gate->size(0) == T && gate->size(1) == H, "gate must be [T, heads] in the activation type");
+    a.gate = gate->data_ptr(); a.ld_gate = gate->stride(0);
+  }
+  out = out_.has_value() ? *out_ : torch::empty({T, H * V}, kpool.options());
   check_rows(out, "out");
   TORCH_CHECK(out.scalar_type() == kpool.scalar_type() && out.size(0) == T && col0 >= 0 && col0 + H * V <= out.size(1));
+  a.q = q.data_ptr<float>(); a.kpool = kpool.data_ptr(); a.vpool = vpool.data_ptr();
+  a.block_tables = block_tables.data_ptr<int>(); a.max_blocks = (int)block_tables.size(1); a.cu = cu.data_ptr<int>(); a.B = (int)(cu.numel() - 1);
+  a.H = (int)H; a.G = (int)G; a.D = (int)q.size(2); a.V = (int)V; a.page = (int)kpool.size(2);
+  a.block = (int)block; a.window = (int)window; a.keep = (int)keep; a.scale = (float)scale; a.out_mult = (float)out_mult;
+  a.out = static_cast<char*>(out.data_ptr()) + col0 * out.element_size(); a.ld_out = out.stride(0);
+  a.nsplit = 1; a.chunk = 1 << 30;
+  return a;
+}
+}  // namespace
+
+Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
+                         const Tensor& positions, const Tensor& cu, double scale, int64_t block, int64_t window, double out_mult, int64_t max_ctx,
+                         const c10::optional<Tensor>& out_, int64_t col0, int64_t keep, const c10::optional<Tensor>& gate) {
+  check_i32(positions, "positions");
+  const c10::cuda::CUDAGuard guard(q.device());
+  Tensor out;
+  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0);
+  const int64_t T = q.size(0), H = a.H, G = a.G, V = a.V;
+  TORCH_CHECK(V <= 512 && positions.numel() >= T, "attention with a sink: vdim <= 512");
   if (T == 0) return out;
+  a.positions = positions.data_ptr<int>();
   // the most keys any query of this step can see
   int64_t span = max_ctx;
-  if (block > 0) span = std::min(span, block);
-  if (window > 0) span = std::min(span, window);
+  if (block > 0) span = std::min(span, block + keep);
+  if (window > 0) span = std::min(span, window + keep);
   // few query rows over long spans (decode): split the keys over CTAs so the grid fills the GPU; a second kernel merges the parts
-  const int nw = b200::sink_attention_warps((int)H, (int)G);
-  const int64_t ctas = T * G * ((H / G + nw - 1) / nw);
-  int64_t nsplit = 1, chunk = 1 << 30;
+  const int nw = b200::sink_attention_heads_per_cta(a.H, a.G, a.D, a.V);
+  const int64_t ctas = T * G * ((H / G + nw - 1) / nw), unit = b200::sink_attention_chunk_unit();
   if (ctas < 6 * sm_count() && span > 256) {
-    nsplit = std::min<int64_t>({(6 * sm_count() + ctas - 1) / ctas, (span + 127) / 128, (int64_t)32});
-    chunk = ((span + nsplit - 1) / nsplit + 31) / 32 * 32;
+    int64_t nsplit = std::min<int64_t>({(6 * sm_count() + ctas - 1) / ctas, (span + 127) / 128, (int64_t)32});
+    const int64_t chunk = ((span + nsplit - 1) / nsplit + unit - 1) / unit * unit;
     nsplit = (span + chunk - 1) / chunk;
+    if (nsplit > 1) { a.nsplit = (int)nsplit; a.chunk = (int)chunk; }
   }
   Tensor part;
-  if (nsplit > 1) part = torch::empty({T * H * nsplit * (V + 2)}, q.options());
-  else chunk = 1 << 30;
-  LAUNCH_OK(b200::sink_attention_launch(q.data_ptr<float>(), kpool.data_ptr(), vpool.data_ptr(), sink.has_value() ? sink->data_ptr<float>() : nullptr,
-                                        block_tables.data_ptr<int>(), (int)block_tables.size(1), positions.data_ptr<int>(), cu.data_ptr<int>(),
-                                        (int)(cu.numel() - 1), (int)H, (int)G, (int)D, (int)V, (int)kpool.size(2), (int)block, (int)window, (float)scale,
-                                        (float)out_mult, static_cast<char*>(out.data_ptr()) + col0 * out.element_size(), out.stride(0), is_f32(kpool), (int)T,
-                                        (int)nsplit, (int)chunk, nsplit > 1 ? part.data_ptr<float>() : nullptr, cur_stream()));
-  if (nsplit > 1) ++g_launches;
+  if (a.nsplit > 1) { part = torch::empty({T * H * a.nsplit * (V + 2)}, q.options()); a.part = part.data_ptr<float>(); }
+  LAUNCH_OK(b200::sink_attention_launch(a, is_f32(kpool), (int)T, cur_stream()));
+  if (a.nsplit > 1) ++g_launches;
+  return out;
+}
+
+// bf16, any number of sequences and query rows, tensor cores
+Tensor hy_sink_flash(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
+                     const Tensor& ctx, const Tensor& cu, double scale, int64_t block, int64_t window, double out_mult, const c10::optional<Tensor>& out_,
+                     int64_t col0, int64_t keep, const c10::optional<Tensor>& gate) {
+  check_i32(ctx, "context_lens"); check_bf16(kpool, "kpool");
+  const c10::cuda::CUDAGuard guard(q.device());
+  Tensor out;
+  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0);
+  TORCH_CHECK(ctx.numel() >= a.B && out.stride(0) % 2 == 0 && col0 % 2 == 0, "tensor-core attention: even output columns and rows");
+  if (q.size(0) == 0) return out;
+  LAUNCH_OK(b200::sink_flash_launch(a, ctx.data_ptr<int>(), (int)((q.size(0) + 63) / 64 + a.B), cur_stream()));
+  return out;
+}
+
+// out[t] = (selective scan of x) * silu(gate)   (activation type of x)
+Tensor hy_selective_scan(const Tensor& x, const Tensor& dt, const Tensor& dt_bias, const Tensor& A_log, const Tensor& bc, int64_t b0, int64_t c0, const Tensor& D,
+                         const c10::optional<Tensor>& gate, Tensor state, const Tensor& cu, const Tensor& ctx, const Tensor& slots, int64_t max_q) {
+  check_act(x, "x"); check_rows(x, "x"); check_rows(dt, "dt"); check_f32c(dt_bias, "dt_bias"); check_f32c(A_log, "A_log"); check_rows(bc, "bc"); check_f32c(D, "D");
+  check_f32c(state, "state"); check_i32(cu, "cu_seqlens"); check_i32(ctx, "context_lens"); check_i32(slots, "state_slots");
+  const int64_t T = x.size(0), I = x.size(1), N = A_log.size(1), B = slots.numel();
+  TORCH_CHECK(A_log.dim() == 2 && A_log.size(0) == I && dt_bias.numel() == I && D.numel() == I && dt.is_cuda() && dt.scalar_type() == torch::kFloat32 &&
+              dt.size(0) == T && dt.size(1) == I && cu.numel() == B + 1 && ctx.numel() >= B);
+  TORCH_CHECK(bc.is_cuda() && bc.scalar_type() == x.scalar_type() && bc.size(0) == T && b0 >= 0 && c0 >= 0 && std::max(b0, c0) + N <= bc.size(1));
+  TORCH_CHECK(state.dim() == 3 && state.size(1) == I && state.size(2) == N, "selective-scan state [slots, inner, state]");
+  TORCH_CHECK(b200::selective_scan_supported((int)N), "selective scan: state sizes 1 .. 256");
+  if (gate.has_value()) {
+    check_rows(*gate, "gate");
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == x.scalar_type() && gate->size(0) == T && gate->size(1) == I);
+  }
+  const c10::cuda::CUDAGuard guard(x.device());
+  Tensor out = torch::empty({T, I}, x.options());
+  if (T == 0) return out;
+  const int ns = b200::selective_scan_slices((int)B, (int)I, (int)N, (int)max_q);
+  Tensor ws;
+  if (ns > 1) { ws = torch::empty({(int64_t)b200::selective_scan_workspace((int)B, (int)I, (int)N, ns)}, dt.options()); ++g_launches; }
+  LAUNCH_OK(b200::selective_scan_launch(x.data_ptr(), x.stride(0), dt.data_ptr<float>(), dt.stride(0), dt_bias.data_ptr<float>(), A_log.data_ptr<float>(), bc.data_ptr(),
+                                        bc.stride(0), (int)b0, (int)c0, D.data_ptr<float>(), gate.has_value() ? gate->data_ptr() : nullptr,
+                                        gate.has_value() ? gate->stride(0) : 0, state.data_ptr<float>(), cu.data_ptr<int>(), ctx.data_ptr<int>(), slots.data_ptr<int>(),
+                                        out.data_ptr(), (int)B, (int)I, (int)N, is_f32(x), (int)max_q, ns, ws.defined() ? ws.data_ptr<float>() : nullptr, cur_stream()));
   return out;
 }
 
@@ -1434,7 +1509,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("hy_sink_softmax", &hy_sink_softmax, py::arg("s"), py::arg("sink"), py::arg("H"), py::arg("ctx0"), py::arg("scale"), py::arg("out_f32"),
         py::arg("window") = 0, py::arg("k0") = 0, py::arg("softcap") = 0.0, py::arg("temp_coef") = 0.0, py::arg("temp_every") = 1.0);
   m.def("hy_scaled_add_norm_", &hy_scaled_add_norm_, py::arg("x"), py::arg("y"), py::arg("ls"), py::arg("w"), py::arg("eps"), py::arg("act_f32"),
-        py::arg("extra") = py::none(), py::arg("gate") = py::none());
+        py::arg("extra") = py::none(), py::arg("gate") = py::none(), py::arg("mult") = 1.0);
   m.def("hy_mlstm_scan", &hy_mlstm_scan);
   m.def("hy_sigmoid_topk", &hy_sigmoid_topk, py::arg("z"), py::arg("E"), py::arg("top"), py::arg("mode") = 0, py::arg("bias") = py::none());
   m.def("hy_clamped_glu", &hy_clamped_glu, py::arg("gate"), py::arg("up"), py::arg("limit"), py::arg("row_of") = py::none(), py::arg("scale") = py::none(),
@@ -1452,10 +1527,17 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("hy_delta_scan", &hy_delta_scan);
   m.def("hy_mingru_scan", &hy_mingru_scan, py::arg("rows"), py::arg("z0"), py::arg("x0"), py::arg("g0"), py::arg("width"), py::arg("state"), py::arg("cu"),
         py::arg("ctx"), py::arg("slots"), py::arg("out_mult"), py::arg("max_q"), py::arg("out") = py::none(), py::arg("col0") = 0);
-  m.def("hy_qk_norm_rope_append", &hy_qk_norm_rope_append);
+  m.def("hy_qk_norm_rope_append", &hy_qk_norm_rope_append, py::arg("rows"), py::arg("q0"), py::arg("k0"), py::arg("v0"), py::arg("heads"), py::arg("dim"),
+        py::arg("qn"), py::arg("kn"), py::arg("eps"), py::arg("inv_freq"), py::arg("kpool"), py::arg("vpool"), py::arg("slot_map"), py::arg("positions"),
+        py::arg("half") = false, py::arg("norm_after") = false, py::arg("rot_mult") = 1.0, py::arg("v_first") = py::none(), py::arg("lam") = 0.0);
   m.def("hy_sink_attention", &hy_sink_attention, py::arg("q"), py::arg("kpool"), py::arg("vpool"), py::arg("sink"), py::arg("block_tables"), py::arg("positions"),
         py::arg("cu"), py::arg("scale"), py::arg("block"), py::arg("window"), py::arg("out_mult"), py::arg("max_ctx"), py::arg("out") = py::none(),
-        py::arg("col0") = 0);
+        py::arg("col0") = 0, py::arg("keep") = 0, py::arg("gate") = py::none());
+  m.def("hy_sink_flash", &hy_sink_flash, py::arg("q"), py::arg("kpool"), py::arg("vpool"), py::arg("sink"), py::arg("block_tables"), py::arg("context_lens"),
+        py::arg("cu"), py::arg("scale"), py::arg("block"), py::arg("window"), py::arg("out_mult"), py::arg("out") = py::none(), py::arg("col0") = 0,
+        py::arg("keep") = 0, py::arg("gate") = py::none());
+  m.def("hy_sink_flash_supported", [](int64_t d, int64_t v) { return b200::sink_flash_supported((int)d, (int)v); });
+  m.def("hy_selective_scan", &hy_selective_scan);
   m.def("hy_group_softmax_topk", &hy_group_softmax_topk);
   m.def("pdl_skip_next", []() { b200::pdl_skip_next(); });
   m.def("sm_arch", []() { return std::string("sm_100a"); });

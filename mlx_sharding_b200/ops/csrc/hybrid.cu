@@ -468,11 +468,11 @@ __global__ void sink_softmax_kernel(const float* __restrict__ s, const float* __
 }
 
 // ---------------------------------------------------------------------------------------------------------- pre-norm residual step
-// x += (y + extra * sigmoid(gate[t])) * ls   (x, y, extra fp32; ls, extra nullable);   xa = (AT)(x * rsqrt(mean(x^2) + eps) * w)
+// x += (y + extra * sigmoid(gate[t])) * ls * mult   (x, y, extra fp32; ls, extra nullable);   xa = (AT)(x * rsqrt(mean(x^2) + eps) * w)
 template <typename AT>
 __global__ void scaled_add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, long long ld_y, const float* __restrict__ ls,
                                        const float* __restrict__ extra, long long ld_e, const float* __restrict__ gate, long long ld_gate,
-                                       const float* __restrict__ w, AT* __restrict__ xa, int n, float eps) {
+                                       const float* __restrict__ w, AT* __restrict__ xa, int n, float eps, float mult) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   const float* yr = y + t * ld_y;
@@ -483,7 +483,7 @@ __global__ void scaled_add_norm_kernel(float* __restrict__ x, const float* __res
     float v = yr[c];
     if (er != nullptr) v += er[c] * sg;
     if (ls != nullptr) v *= ls[c];
-    v += x[t * n + c];
+    v = v * mult + x[t * n + c];
     x[t * n + c] = v;
     ss += v * v;
   }
@@ -641,7 +641,7 @@ __global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z,
 
 // gate rows g and up rows u (F wide each, own row strides) -> g' sigmoid(1.702 g') (u' + 1),  g' = min(s g, limit), u' = clamp(s u, +-limit).  Block i handles row
 // row_of[i] with scale s = scale[i] (both nullable: row i, scale 1): scaling a projection's output equals scaling its input.
-// kind 1: silu(g) u s instead (no clamp; the scale multiplies the product, i.e. the input of the down projection).
+// kind 1: silu(g) u s, kind 2: gelu_tanh(g) u s instead (no clamp; the scale multiplies the product, i.e. the input of the down projection).
 template <typename AT>
 __global__ void clamped_glu_kernel(const AT* __restrict__ gp, long long ld_g, const AT* __restrict__ up, long long ld_u, int F, float limit,
                                    const int* __restrict__ row_of, const float* __restrict__ scale, AT* __restrict__ out, int kind) {
@@ -651,6 +651,7 @@ __global__ void clamped_glu_kernel(const AT* __restrict__ gp, long long ld_g, co
   const AT* urow = up + r * ld_u;
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < F; c += gridDim.y * blockDim.x) {
     if (kind == 1) { stf<AT>(out + r * F + c, silu_f(ldf<AT>(grow + c)) * ldf<AT>(urow + c) * s); continue; }
+    if (kind == 2) { stf<AT>(out + r * F + c, gelu_tanh_f(ldf<AT>(grow + c)) * ldf<AT>(urow + c) * s); continue; }
     const float g = fminf(s * ldf<AT>(grow + c), limit), u = fminf(fmaxf(s * ldf<AT>(urow + c), -limit), limit);
     stf<AT>(out + r * F + c, g * sigmoid_f(1.702f * g) * (u + 1.f));
   }
@@ -826,9 +827,9 @@ cudaError_t latent_attention_launch(const void* q, const void* pool, const float
 }
 
 cudaError_t scaled_add_norm_launch(float* x, const float* y, long long ld_y, const float* ls, const float* extra, long long ld_e,
-                                   const float* gate, long long ld_gate, const float* w, void* xa, bool f32, int n, float eps, int T,
+                                   const float* gate, long long ld_gate, const float* w, void* xa, bool f32, int n, float eps, float mult, int T,
                                    cudaStream_t s) {
-  AT_DISPATCH(f32, (scaled_add_norm_kernel<AT><<<T, 256, 0, s>>>(x, y, ld_y, ls, extra, ld_e, gate, ld_gate, w, (AT*)xa, n, eps)));
+  AT_DISPATCH(f32, (scaled_add_norm_kernel<AT><<<T, 256, 0, s>>>(x, y, ld_y, ls, extra, ld_e, gate, ld_gate, w, (AT*)xa, n, eps, mult)));
   return last();
 }
 

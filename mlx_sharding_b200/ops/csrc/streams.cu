@@ -1,7 +1,7 @@
 // Kernels of stacks that run on several residual streams with dynamic-tanh norms: the stream update fused with the read for the next
-// sublayer, the gated delta rule with one decay per head and key channel, grouped-query attention inside fixed blocks of positions
-// (or a sliding window) with a sink, its prologue (per-head RMS norm of queries and keys, rotation of adjacent pairs, append to the
-// paged pools), minGRU, the group-limited softmax router and the squared ReLU.
+// sublayer, the gated delta rule with one decay per head and key channel, the prologue of grouped-query attention (per-head RMS norm of
+// queries and keys, rotation, value mixing, append to the paged pools; the attention itself is in sinkattn.cu), minGRU, the group-limited
+// softmax router and the squared ReLU.
 //
 // Conventions as in hybrid.cu: a step is a ragged batch (rows cu_seqlens[b] .. cu_seqlens[b+1] belong to sequence b, whose recurrent
 // state lives in slot slots[b]; a sequence whose step starts at position 0 starts from a zero state); activations are AT = bf16
@@ -405,211 +405,87 @@ __global__ void mingru_scan_kernel(const AT* __restrict__ rows, long long ld, in
 }
 
 // ---------------------------------------------------------------------------------------------------------- attention prologue
-// One warp per head of a token (query heads first, then key heads): x / sqrt(mean(x^2) + eps) * w, then adjacent pairs (2i, 2i+1) of the
-// first `rot` entries turn by pos * inv_freq[i].  Queries -> qout fp32 [T, H, D]; keys and the untouched values -> the paged pools.
-template <typename AT>
-__global__ void qk_norm_rope_append_kernel(const AT* __restrict__ rows, long long ld, int q0, int k0, int v0, int H, int G, int D, int V,
-                                           const float* __restrict__ qn, const float* __restrict__ kn, float eps,
-                                           const float* __restrict__ inv_freq, int rot, const int* __restrict__ positions,
-                                           const int* __restrict__ slot_map, int page, float* __restrict__ qout, AT* __restrict__ kpool,
-                                           AT* __restrict__ vpool) {
-  const long long t = blockIdx.x;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const float pos = (float)positions[t];
-  const int slot = slot_map[t], pg = slot / page, off = slot % page;
-  const AT* r = rows + t * ld;
-  for (int hh = warp; hh < H + G; hh += nw) {
-    const bool isq = hh < H;
-    const AT* src = isq ? r + q0 + hh * D : r + k0 + (hh - H) * D;
-    const float* w = isq ? qn : kn;
-    float ss = 0.f;
-    for (int d = lane; d < D; d += 32) { const float v = ldf<AT>(src + d); ss += v * v; }
-    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)D + eps);
-    float* qd = qout + (t * H + hh) * D;
-    AT* kd = kpool + (((long long)pg * G + (hh - H)) * page + off) * D;
-    for (int d0 = 0; d0 < D; d0 += 32) {        // all lanes take part in the shuffle; d even <-> lane even
-      const int d = d0 + lane;
-      float v = d < D ? ldf<AT>(src + d) * inv * w[d] : 0.f;
-      const float other = __shfl_xor_sync(0xffffffffu, v, 1);
-      if (d < rot) {
-        float sn, cs;
-        sincosf(pos * inv_freq[d >> 1], &sn, &cs);
-        v = (d & 1) ? v * cs + other * sn : v * cs - other * sn;
-      }
-      if (d < D) { if (isq) qd[d] = v; else stf<AT>(kd + d, v); }
-    }
-  }
-  for (int i = threadIdx.x; i < G * V; i += blockDim.x) vpool[(((long long)pg * G + i / V) * page + off) * V + i % V] = r[v0 + i];
-}
-
-// ---------------------------------------------------------------------------------------------------------- attention with a sink
-struct SinkAttnArgs {
-  const float* q;                           // fp32 [T, H, D] (normed, rotated)
-  const void* kpool; const void* vpool;     // [pages, G, page, D] / [pages, G, page, V]
-  const float* sink;                        // [H] (nullable)
-  const int* block_tables; int max_blocks;
-  const int* positions; const int* cu; int B;
-  int H, G, D, V, page;
-  int block, window;                        // visible keys j <= p: same block of `block` positions (0: all), p - j < window (0: all)
-  float scale, out_mult;
-  void* out; long long ld_out;              // AT, row t at out + t * ld_out, head h at column h * V
-  int nsplit, chunk;
-  float* part;                              // [T, H, nsplit, V + 2] = (m, l, o[V]) when the keys are split
+struct PrologueArgs {
+  const void* rows; long long ld;           // AT, query heads from column q0 on, keys k0, values v0
+  int q0, k0, v0, H, G, D, V;
+  const float* qn; const float* kn;         // [D] norm weights (nullable)
+  float eps;
+  const float* inv_freq; int rot;           // angles per position of the rot / 2 pairs
+  float rot_mult;                           // factor on cos and sin
+  const int* positions; const int* slot_map;
+  int page;
+  const void* v_first; long long ld_vf;     // AT [T, G V] mixed into the values (nullable)
+  float lam;
+  float* qout; void* kpool; void* vpool;
 };
 
-constexpr int kTile = 32;
-
-__device__ __forceinline__ int first_key(int pos, int block, int window) {
-  int lo = block > 0 ? pos / block * block : 0;
-  if (window > 0) lo = max(lo, pos - window + 1);
-  return lo;
-}
-
-// value column of register i of a lane: VEC (vdim a multiple of 128) 4 lane + 128 (i / 4) + i % 4 — four adjacent columns per 16-byte
-// shared-memory load —, else lane + 32 i
-template <bool VEC>
-__device__ __forceinline__ int sink_vcol(int lane, int i) { return VEC ? 4 * lane + 128 * (i >> 2) + (i & 3) : lane + 32 * i; }
-
-// grid (tokens, G * ceil((H/G) / warps), key splits); one warp per query head, the warps of a CTA share one key / value head whose tile
-// of kTile keys and values is staged in shared memory as floats.  Lane j scores key j of the tile; the running softmax (m, l) and the
-// accumulator live in registers, lane owning the value columns sink_vcol(lane, i).  Key splits count from the first visible key.
-// VEC (dim a multiple of the 16-byte chunk, vdim a multiple of 128): 16-byte shared-memory stores and loads in all phases, key rows
-// padded by 4 floats; else scalar accesses, key rows padded by 1.
-template <typename AT, int NPL, bool VEC>
-__global__ void sink_attention_kernel(SinkAttnArgs a) {
-  extern __shared__ __align__(16) float smem[];
-  const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int D = a.D, V = a.V, ldk = VEC ? D + 4 : D + 1;
-  float* qs = smem;                         // [nw][D]
-  float* ks = qs + nw * D;                  // [tile][D + 1]
-  float* vs = ks + kTile * ldk;             // [tile][V]
-  const int t = blockIdx.x, Rg = a.H / a.G, nb = (Rg + nw - 1) / nw;
-  const int g = blockIdx.y / nb, r = (blockIdx.y % nb) * nw + warp, h = g * Rg + r;
-  const bool valid = r < Rg;
-  const int pos = a.positions[t];
-  const int* bt = a.block_tables + (long long)seq_of(a.cu, a.B, t) * a.max_blocks;
-  for (int i = threadIdx.x; i < nw * D; i += blockDim.x) {
-    const int rr = (blockIdx.y % nb) * nw + i / D;
-    qs[i] = rr < Rg ? a.q[((long long)t * a.H + g * Rg + rr) * D + i % D] * a.scale : 0.f;
+// One warp per head of a token (query heads first, then key heads), the head's entries lane + 32 i in registers: RMS norm (times a weight)
+// and rotation of the first `rot` entries, adjacent pairs (2i, 2i+1) or HALF pairs (i, i + rot / 2), the norm before the rotation or
+// (AFTER) behind it.  The token's cosines and sines are computed once per CTA.  Queries -> qout fp32 [T, H, D]; keys and values (as they
+// are, or (1 - lam) v + lam v_first) -> the paged pools.
+template <typename AT, int NPL, bool HALF, bool AFTER>
+__global__ void qk_norm_rope_append_kernel(PrologueArgs a) {
+  extern __shared__ float cs[];             // [rot / 2] cosines | [rot / 2] sines
+  const long long t = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, D = a.D, H = a.H, G = a.G, V = a.V, hr = a.rot / 2;
+  const float pos = (float)a.positions[t];
+  for (int i = threadIdx.x; i < hr; i += blockDim.x) {
+    float sn, cn;
+    sincosf(pos * a.inv_freq[i], &sn, &cn);
+    cs[i] = cn * a.rot_mult; cs[hr + i] = sn * a.rot_mult;
   }
-  float m = -INFINITY, l = 0.f, o[NPL];
+  __syncthreads();
+  const int slot = a.slot_map[t], pg = slot / a.page, off = slot % a.page;
+  const AT* r = (const AT*)a.rows + t * a.ld;
+  for (int hh = warp; hh < H + G; hh += nw) {
+    const bool isq = hh < H;
+    const AT* src = isq ? r + a.q0 + hh * D : r + a.k0 + (hh - H) * D;
+    const float* w = isq ? a.qn : a.kn;
+    float v[NPL], inv = 1.f;
 #pragma unroll
-  for (int i = 0; i < NPL; ++i) o[i] = 0.f;
-  const float* qh = qs + warp * D;
-  const int lo = first_key(pos, a.block, a.window);
-  const long long jb = (long long)lo + (long long)blockIdx.z * a.chunk;
-  const int jbeg = (int)min(jb, (long long)pos + 1), jend = (int)min((long long)pos + 1, jb + a.chunk);
-  constexpr int E = 16 / (int)sizeof(AT);
-  const bool vec = D % E == 0 && V % E == 0;
-  for (int j0 = jbeg; j0 < jend; j0 += kTile) {
-    __syncthreads();
-    const int nk = min(kTile, jend - j0);
-    for (int jj = warp; jj < nk; jj += nw) {            // each warp fetches whole rows: one block-table lookup per row
-      const int j = j0 + jj;
-      const long long base = ((long long)bt[j / a.page] * a.G + g) * a.page + j % a.page;
-      const AT* ksrc = (const AT*)a.kpool + base * D;
-      const AT* vsrc = (const AT*)a.vpool + base * V;
-      float* kd = ks + jj * ldk;
-      float* vd = vs + jj * V;
-      if (VEC) {
-        for (int c = lane; c < (D + V) / E; c += 32) {
-          float f[E];
-          unpack16<AT>(*reinterpret_cast<const uint4*>(c < D / E ? ksrc + c * E : vsrc + (c - D / E) * E), f);
-          float* dst = c < D / E ? kd + c * E : vd + (c - D / E) * E;
+    for (int i = 0; i < NPL; ++i) v[i] = lane + 32 * i < D ? ldf<AT>(src + lane + 32 * i) : 0.f;
+    auto scale = [&]() {
+      float ss = 0.f;
 #pragma unroll
-          for (int e = 0; e < E; e += 4) *reinterpret_cast<float4*>(dst + e) = make_float4(f[e], f[e + 1], f[e + 2], f[e + 3]);
+      for (int i = 0; i < NPL; ++i) ss += v[i] * v[i];
+      inv = 1.f / sqrtf(warp_sum(ss) / (float)D + a.eps);
+#pragma unroll
+      for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; v[i] *= w != nullptr && d < D ? inv * w[d] : inv; }
+    };
+    if (!AFTER) scale();
+#pragma unroll
+    for (int i = 0; i < NPL; ++i) {
+      const int d = lane + 32 * i;
+      if (32 * i >= a.rot) break;             // uniform over the warp: all lanes take part in the shuffle
+      if (HALF) {
+        if (d < a.rot) {
+          const bool lo = d < hr;
+          const int p = lo ? d + hr : d - hr, k = lo ? d : p;
+          float other = ldf<AT>(src + p);
+          if (!AFTER) other *= w != nullptr ? inv * w[p] : inv;
+          v[i] = lo ? v[i] * cs[k] - other * cs[hr + k] : v[i] * cs[k] + other * cs[hr + k];
         }
-      } else if (vec) {
-        for (int c = lane; c < D / E; c += 32) { float f[E]; unpack16<AT>(*reinterpret_cast<const uint4*>(ksrc + c * E), f);
-#pragma unroll
-          for (int e = 0; e < E; ++e) kd[c * E + e] = f[e]; }
-        for (int c = lane; c < V / E; c += 32) unpack16<AT>(*reinterpret_cast<const uint4*>(vsrc + c * E), vd + c * E);
       } else {
-        for (int d = lane; d < D; d += 32) kd[d] = ldf<AT>(ksrc + d);
-        for (int d = lane; d < V; d += 32) vd[d] = ldf<AT>(vsrc + d);
+        const float other = __shfl_xor_sync(0xffffffffu, v[i], 1);      // d even <-> lane even
+        if (d < a.rot) v[i] = (d & 1) ? v[i] * cs[d >> 1] + other * cs[hr + (d >> 1)] : v[i] * cs[d >> 1] - other * cs[hr + (d >> 1)];
       }
     }
-    __syncthreads();
-    if (!valid) continue;
-    float sc = -INFINITY;
-    if (lane < nk) {
-      const float* kr = ks + lane * ldk;
-      float d = 0.f;
-      if (VEC) {
-        const float4* q4 = reinterpret_cast<const float4*>(qh);
-        const float4* k4 = reinterpret_cast<const float4*>(kr);
-        for (int i = 0; i < (D >> 2); ++i) { const float4 x = q4[i], y = k4[i]; d += x.x * y.x + x.y * y.y + x.z * y.z + x.w * y.w; }
-      } else {
-        for (int i = 0; i < D; ++i) d += qh[i] * kr[i];
-      }
-      sc = d;
-    }
-    const float nm = fmaxf(m, warp_max(sc));
-    const float cf = m == -INFINITY ? 0.f : expf(m - nm);
-    const float pw = lane < nk ? expf(sc - nm) : 0.f;
-    l = l * cf + warp_sum(pw);
-    m = nm;
+    if (AFTER) scale();
+    float* qd = a.qout + (t * H + hh) * D;
+    AT* kd = (AT*)a.kpool + (((long long)pg * G + (hh - H)) * a.page + off) * D;
 #pragma unroll
-    for (int i = 0; i < NPL; ++i) o[i] *= cf;
-    for (int jj = 0; jj < nk; ++jj) {
-      const float w = __shfl_sync(0xffffffffu, pw, jj);
-      const float* vr = vs + jj * V;
-      if (VEC) {
-#pragma unroll
-        for (int i = 0; i < NPL / 4; ++i)
-          if (128 * i < V) {
-            const float4 c = *reinterpret_cast<const float4*>(vr + 4 * lane + 128 * i);
-            o[4 * i] += w * c.x; o[4 * i + 1] += w * c.y; o[4 * i + 2] += w * c.z; o[4 * i + 3] += w * c.w;
-          }
-      } else {
-#pragma unroll
-        for (int i = 0; i < NPL; ++i) {
-          const int d = lane + 32 * i;
-          if (d < V) o[i] += w * vr[d];
-        }
-      }
+    for (int i = 0; i < NPL; ++i) {
+      const int d = lane + 32 * i;
+      if (d < D) { if (isq) qd[d] = v[i]; else stf<AT>(kd + d, v[i]); }
     }
   }
-  if (!valid) return;
-  if (a.nsplit == 1) {
-    // the query's own position is always visible: l > 0.  The sink joins the denominator only: exp(sink - m), no value.
-    if (a.sink != nullptr) l += expf(a.sink[h] - m);
-    const float inv = a.out_mult / l;
-    AT* orow = (AT*)a.out + (long long)t * a.ld_out + (long long)h * V;
-#pragma unroll
-    for (int i = 0; i < NPL; ++i) { const int d = sink_vcol<VEC>(lane, i); if (d < V) stf<AT>(orow + d, o[i] * inv); }
-  } else {
-    float* pp = a.part + (((long long)t * a.H + h) * a.nsplit + blockIdx.z) * (V + 2);
-    if (lane == 0) { pp[0] = m; pp[1] = l; }
-#pragma unroll
-    for (int i = 0; i < NPL; ++i) { const int d = sink_vcol<VEC>(lane, i); if (d < V) pp[2 + d] = o[i]; }
+  AT* vpool = (AT*)a.vpool;
+  const AT* vf = a.v_first != nullptr ? (const AT*)a.v_first + t * a.ld_vf : nullptr;
+  for (int i = threadIdx.x; i < G * V; i += blockDim.x) {
+    AT* dst = vpool + (((long long)pg * G + i / V) * a.page + off) * V + i % V;
+    if (vf == nullptr) *dst = r[a.v0 + i];
+    else stf<AT>(dst, (1.f - a.lam) * ldf<AT>(r + a.v0 + i) + a.lam * ldf<AT>(vf + i));
   }
-}
-
-// merge the key splits of one (token, head): o = sum_z o_z e^(m_z - M) / (sum_z l_z e^(m_z - M) + e^(sink - M)).  One warp each.
-template <typename AT, int NPL>
-__global__ void sink_combine_kernel(const float* __restrict__ part, const float* __restrict__ sink, int H, int V, int nsplit, float out_mult,
-                                    AT* __restrict__ out, long long ld_out) {
-  const long long th = blockIdx.x;
-  const int lane = threadIdx.x, h = (int)(th % H);
-  const float* pp = part + th * nsplit * (V + 2);
-  float M = -INFINITY, den = 0.f, acc[NPL];
-  for (int z = 0; z < nsplit; ++z) M = fmaxf(M, pp[(long long)z * (V + 2)]);
-#pragma unroll
-  for (int i = 0; i < NPL; ++i) acc[i] = 0.f;
-  for (int z = 0; z < nsplit; ++z) {
-    const float* pz = pp + (long long)z * (V + 2);
-    if (pz[0] == -INFINITY) continue;                 // a split beyond this token's keys
-    const float e = expf(pz[0] - M);
-    den += pz[1] * e;
-#pragma unroll
-    for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) acc[i] += pz[2 + d] * e; }
-  }
-  if (sink != nullptr) den += expf(sink[h] - M);
-  const float inv = out_mult / den;
-  AT* orow = out + (th / H) * ld_out + (long long)h * V;
-#pragma unroll
-  for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) stf<AT>(orow + d, acc[i] * inv); }
 }
 
 // ---------------------------------------------------------------------------------------------------------- router
@@ -765,59 +641,34 @@ cudaError_t mingru_scan_launch(const void* rows, long long ld, int z0, int x0, i
   return last();
 }
 
+template <typename AT, int NPL>
+static void prologue_t(const PrologueArgs& a, bool half, bool after, int T, cudaStream_t s) {
+  const int threads = 32 * (a.H + a.G < 8 ? a.H + a.G : 8);
+  const size_t smem = (a.rot < 2 ? 2 : a.rot) * sizeof(float);
+  if (half) {
+    if (after) qk_norm_rope_append_kernel<AT, NPL, true, true><<<T, threads, smem, s>>>(a);
+    else qk_norm_rope_append_kernel<AT, NPL, true, false><<<T, threads, smem, s>>>(a);
+  } else {
+    if (after) qk_norm_rope_append_kernel<AT, NPL, false, true><<<T, threads, smem, s>>>(a);
+    else qk_norm_rope_append_kernel<AT, NPL, false, false><<<T, threads, smem, s>>>(a);
+  }
+}
+
 cudaError_t qk_norm_rope_append_launch(const void* rows, long long ld, int q0, int k0, int v0, int H, int G, int D, int V, const float* qn,
                                        const float* kn, float eps, const float* inv_freq, int rot, const int* positions, const int* slot_map,
-                                       int page, float* qout, void* kpool, void* vpool, bool f32, int T, cudaStream_t s) {
-  if (rot % 2 != 0 || rot > D) return cudaErrorInvalidValue;
-  const int threads = 32 * (H + G < 8 ? H + G : 8);
-  AT_DISPATCH(f32, (qk_norm_rope_append_kernel<AT><<<T, threads, 0, s>>>((const AT*)rows, ld, q0, k0, v0, H, G, D, V, qn, kn, eps, inv_freq, rot, positions,
-                                                                        slot_map, page, qout, (AT*)kpool, (AT*)vpool)));
+                                       int page, float* qout, void* kpool, void* vpool, bool f32, bool half, bool norm_after, float rot_mult,
+                                       const void* v_first, long long ld_vf, float lam, int T, cudaStream_t s) {
+  if (rot % 2 != 0 || rot > D || D > 1024) return cudaErrorInvalidValue;
+  const PrologueArgs a{rows, ld, q0, k0, v0, H, G, D, V, qn, kn, eps, inv_freq, rot, rot_mult, positions, slot_map, page, v_first, ld_vf, lam, qout, kpool, vpool};
+  if (D <= 64) AT_DISPATCH(f32, (prologue_t<AT, 2>(a, half, norm_after, T, s)));
+  else if (D <= 128) AT_DISPATCH(f32, (prologue_t<AT, 4>(a, half, norm_after, T, s)));
+  else if (D <= 256) AT_DISPATCH(f32, (prologue_t<AT, 8>(a, half, norm_after, T, s)));
+  else AT_DISPATCH(f32, (prologue_t<AT, 32>(a, half, norm_after, T, s)));
   return last();
 }
 
 bool delta_scan_wants_prepare(int N, int max_q) { return N <= 256 && max_q >= kDeltaWarpMinTokens; }
 long long delta_scan_prepare_width(int G, int H, int N, int P) { return delta_pre_width(G, H, N, P); }
-
-int sink_attention_warps(int H, int G) {
-  const int rg = H / G;
-  return rg < 8 ? rg : 8;
-}
-
-template <typename AT, int NPL, bool VEC>
-static cudaError_t sink_attention_t(const SinkAttnArgs& a, int T, cudaStream_t s) {
-  const int nw = sink_attention_warps(a.H, a.G), nb = (a.H / a.G + nw - 1) / nw;
-  const size_t smem = ((size_t)nw * a.D + (size_t)kTile * (a.D + (VEC ? 4 : 1)) + (size_t)kTile * a.V) * sizeof(float);
-  auto k = sink_attention_kernel<AT, NPL, VEC>;
-  if (smem > 48 * 1024) { cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); if (e != cudaSuccess) return e; }
-  k<<<dim3(T, a.G * nb, a.nsplit), 32 * nw, smem, s>>>(a);
-  if (a.nsplit > 1) sink_combine_kernel<AT, NPL><<<T * a.H, 32, 0, s>>>(a.part, a.sink, a.H, a.V, a.nsplit, a.out_mult, (AT*)a.out, a.ld_out);
-  return last();
-}
-
-cudaError_t sink_attention_launch(const float* q, const void* kpool, const void* vpool, const float* sink, const int* block_tables, int max_blocks,
-                                  const int* positions, const int* cu, int B, int H, int G, int D, int V, int page, int block, int window,
-                                  float scale, float out_mult, void* out, long long ld_out, bool f32, int T, int nsplit, int chunk, float* part,
-                                  cudaStream_t s) {
-  if (G < 1 || H % G != 0 || V > 512 || (size_t)(8 * D + kTile * (D + 4) + kTile * V) * sizeof(float) > 220 * 1024) return cudaErrorInvalidValue;
-  SinkAttnArgs a{q, kpool, vpool, sink, block_tables, max_blocks, positions, cu, B, H, G, D, V, page, block, window, scale, out_mult, out, ld_out,
-                 nsplit, chunk, part};
-  const int npl = (V + 31) / 32;
-  if (V % 128 == 0 && D % (f32 ? 4 : 8) == 0) {            // 16-byte path: whole chunks of keys, four adjacent value columns per lane
-#define SINK_VEC(N) AT_DISPATCH(f32, return (sink_attention_t<AT, N, true>(a, T, s)))
-    if (npl <= 4) SINK_VEC(4);
-    if (npl <= 8) SINK_VEC(8);
-    SINK_VEC(16);
-#undef SINK_VEC
-  }
-#define SINK_CASE(N) AT_DISPATCH(f32, return (sink_attention_t<AT, N, false>(a, T, s)))
-  if (npl <= 1) SINK_CASE(1);
-  if (npl <= 2) SINK_CASE(2);
-  if (npl <= 4) SINK_CASE(4);
-  if (npl <= 8) SINK_CASE(8);
-  SINK_CASE(16);
-#undef SINK_CASE
-  return cudaErrorInvalidValue;
-}
 
 cudaError_t group_softmax_topk_launch(const float* z, long long ld_z, const float* corr, int E, int top, int ng, int keep, int* idx, float* w, int T,
                                       cudaStream_t s) {

@@ -1,5 +1,5 @@
-// Host launch API of streams.cu (several residual streams with dynamic-tanh norms, gated delta rule, attention with a sink inside
-// blocks of positions, minGRU, group-limited softmax router).  `f32` selects the activation type of the call: float (exact mode) or
+// Host launch API of streams.cu (several residual streams with dynamic-tanh norms, gated delta rule, attention prologue, minGRU,
+// group-limited softmax router).  `f32` selects the activation type of the call: float (exact mode) or
 // bf16 (serving); streams, norm weights, recurrence constants and states are always float.  Nullable pointers are marked.
 #pragma once
 #include <cuda_runtime.h>
@@ -21,15 +21,11 @@ bool delta_scan_wants_prepare(int N, int max_q);
 long long delta_scan_prepare_width(int G, int H, int N, int P);
 cudaError_t mingru_scan_launch(const void* rows, long long ld, int z0, int x0, int g0, int R, float* state, const int* cu, const int* ctx,
                                const int* slots, float out_mult, void* out, long long ld_out, int B, bool f32, int max_q, cudaStream_t s);
+// qn, kn, v_first nullable
 cudaError_t qk_norm_rope_append_launch(const void* rows, long long ld, int q0, int k0, int v0, int H, int G, int D, int V, const float* qn,
                                        const float* kn, float eps, const float* inv_freq, int rot, const int* positions, const int* slot_map,
-                                       int page, float* qout, void* kpool, void* vpool, bool f32, int T, cudaStream_t s);
-int sink_attention_warps(int H, int G);
-// sink nullable; block / window 0 = no such limit; part: [T, H, nsplit, V + 2] floats when nsplit > 1
-cudaError_t sink_attention_launch(const float* q, const void* kpool, const void* vpool, const float* sink, const int* block_tables, int max_blocks,
-                                  const int* positions, const int* cu, int B, int H, int G, int D, int V, int page, int block, int window,
-                                  float scale, float out_mult, void* out, long long ld_out, bool f32, int T, int nsplit, int chunk, float* part,
-                                  cudaStream_t s);
+                                       int page, float* qout, void* kpool, void* vpool, bool f32, bool half, bool norm_after, float rot_mult,
+                                       const void* v_first, long long ld_vf, float lam, int T, cudaStream_t s);
 cudaError_t group_softmax_topk_launch(const float* z, long long ld_z, const float* corr, int E, int top, int ng, int keep, int* idx, float* w, int T,
                                       cudaStream_t s);
 }  // namespace b200

@@ -431,21 +431,21 @@ def gated_rmsnorm(y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: flo
     return v.to(out_dtype)
 
 
-def _rot_half(v: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+def _rot_half(v: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, mult: float = 1.0) -> torch.Tensor:
     half = inv_freq.numel()
     a = pos.float()[:, None] * inv_freq.float()
-    c, s = torch.cos(a), torch.sin(a)
+    c, s = torch.cos(a) * mult, torch.sin(a) * mult
     while c.dim() < v.dim():
         c, s = c.unsqueeze(1), s.unsqueeze(1)
     u1, u2 = v[..., :half], v[..., half:2 * half]
     return torch.cat([u1 * c - u2 * s, u2 * c + u1 * s, v[..., 2 * half:]], -1)
 
 
-def _rot_pairs(v: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+def _rot_pairs(v: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, mult: float = 1.0) -> torch.Tensor:
     """Adjacent pairs ``(2i, 2i+1)`` of the first ``2 * len(inv_freq)`` entries turn by ``pos * inv_freq[i]``."""
     half = inv_freq.numel()
     a = pos.float()[:, None] * inv_freq.float()
-    c, s = torch.cos(a), torch.sin(a)
+    c, s = torch.cos(a) * mult, torch.sin(a) * mult
     while c.dim() < v.dim():
         c, s = c.unsqueeze(1), s.unsqueeze(1)
     u1, u2 = v[..., 0:2 * half:2], v[..., 1:2 * half:2]
@@ -516,14 +516,16 @@ def latent_attention_prefill(q, pool, sink, meta: BatchMeta, scale: float, kv_ra
 
 
 def scaled_add_norm_(x: torch.Tensor, y: torch.Tensor, ls: Optional[torch.Tensor], w: torch.Tensor, eps: float, act_dtype: torch.dtype,
-                     extra: Optional[torch.Tensor] = None, extra_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Pre-norm residual step on the fp32 stream ``x`` (in place): ``x += (y + extra * sigmoid(extra_gate)) * ls`` (``ls``: per-channel
-    layer scale or ``None``; ``extra`` / ``extra_gate``: an always-on branch with one gate logit per row), then returns
-    ``x / sqrt(mean(x^2) + eps) * w`` in the activation dtype: the input of the sublayer that follows."""
+                     extra: Optional[torch.Tensor] = None, extra_gate: Optional[torch.Tensor] = None, mult: float = 1.0) -> torch.Tensor:
+    """Pre-norm residual step on the fp32 stream ``x`` (in place): ``x += (y + extra * sigmoid(extra_gate)) * ls * mult`` (``ls``: per-channel
+    layer scale or ``None``; ``extra`` / ``extra_gate``: an always-on branch with one gate logit per row; ``mult``: one factor for all
+    channels), then returns ``x / sqrt(mean(x^2) + eps) * w`` in the activation dtype: the input of the sublayer that follows."""
     yf = y.float()
     if extra is not None:
         yf = yf + extra.float() * torch.sigmoid(extra_gate.float()).reshape(-1, 1)
-    x += yf * ls.float() if ls is not None else yf
+    if ls is not None:
+        yf = yf * ls.float()
+    x += yf * mult if mult != 1.0 else yf
     return rmsnorm_cast(x, w, eps, act_dtype)
 
 
@@ -791,35 +793,51 @@ def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, dt: torch.Tensor, dt_bias:
     return o.view(T, H * V)
 
 
-def qk_norm_rope_append(rows: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w: torch.Tensor, kn_w: torch.Tensor,
-                        eps: float, inv_freq: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, meta: BatchMeta) -> torch.Tensor:
+def qk_norm_rope_append(rows: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w: Optional[torch.Tensor],
+                        kn_w: Optional[torch.Tensor], eps: float, inv_freq: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, meta: BatchMeta,
+                        half: bool = False, norm_after: bool = False, rot_mult: float = 1.0, v_first: Optional[torch.Tensor] = None,
+                        v_lambda: float = 0.0) -> torch.Tensor:
     """Attention prologue on a fused projection's rows ``[.. q: heads*dim .. k: G*dim .. v: G*dv ..]``: per head ``x / sqrt(mean(x^2) + eps)
-    * w`` on queries and keys (weights ``[dim]`` shared by the heads), then adjacent pairs ``(2i, 2i+1)`` of the first ``2 len(inv_freq)``
-    entries turn by ``position * inv_freq[i]``; keys and (untouched) values go to the pools ``[pages, G, page, d]`` at
-    ``meta.slot_mapping``.  Returns the queries fp32 ``[T, heads, dim]``."""
+    * w`` on queries and keys (weights ``[dim]`` shared by the heads, or ``None``), and rotation of the first ``2 len(inv_freq)`` entries by
+    ``position * inv_freq[i]`` in adjacent pairs ``(2i, 2i+1)`` or (``half``) pairs ``(i, i + len(inv_freq))``, cos and sin times
+    ``rot_mult``; the norm comes before the rotation or (``norm_after``) behind it.  Values: as they are, or ``(1 - v_lambda) v + v_lambda
+    v_first`` with ``v_first`` ``[T, G*dv]``.  Keys and values go to the pools ``[pages, G, page, d]`` at ``meta.slot_mapping``.  Returns
+    the queries fp32 ``[T, heads, dim]``."""
     P, G, page, dk = kpool.shape
     dv = vpool.shape[3]
     T = rows.shape[0]
-    nrm = lambda x, w: x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
-    q = nrm(rows[:, q_col0:q_col0 + heads * dim].float().view(T, heads, dim), qn_w)
-    k = nrm(rows[:, k_col0:k_col0 + G * dk].float().view(T, G, dk), kn_w)
-    if inv_freq is not None and inv_freq.numel():
-        q, k = _rot_pairs(q, meta.positions, inv_freq), _rot_pairs(k, meta.positions, inv_freq)
+
+    def norm(x, w):
+        x = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+        return x if w is None else x * w.float()
+
+    def rotate(x):
+        if inv_freq is None or not inv_freq.numel():
+            return x
+        return (_rot_half if half else _rot_pairs)(x, meta.positions, inv_freq, rot_mult)
+
+    q = rows[:, q_col0:q_col0 + heads * dim].float().view(T, heads, dim)
+    k = rows[:, k_col0:k_col0 + G * dk].float().view(T, G, dk)
+    q, k = (norm(rotate(q), qn_w), norm(rotate(k), kn_w)) if norm_after else (rotate(norm(q, qn_w)), rotate(norm(k, kn_w)))
+    v = rows[:, v_col0:v_col0 + G * dv]
+    if v_first is not None:
+        v = (1.0 - v_lambda) * v.float() + v_lambda * v_first.float()
     slot = meta.slot_mapping.long()
     pg, off = slot // page, slot % page
     kpool[pg, :, off] = k.to(kpool.dtype)
-    vpool[pg, :, off] = rows[:, v_col0:v_col0 + G * dv].reshape(T, G, dv).to(vpool.dtype)
+    vpool[pg, :, off] = v.reshape(T, G, dv).to(vpool.dtype)
     return q.contiguous()
 
 
 def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, sink: Optional[torch.Tensor], meta: BatchMeta, scale: float,
                    block: int = 0, window: int = 0, out_mult: float = 1.0, out_dtype: torch.dtype = torch.float32,
-                   out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
+                   out: Optional[torch.Tensor] = None, out_col0: int = 0, keep_first: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal grouped-query attention over paged keys / values.  ``q`` ``[T, H, d]`` (normed and rotated), pools ``[pages, G, page, d]`` /
     ``[pages, G, page, dv]``; head ``h`` reads key / value head ``h // (H / G)``.  The query at position ``i`` sees keys ``j <= i`` with
     ``floor(j / block) == floor(i / block)`` (``block > 0``: blocks counted from position 0 of the sequence) and ``i - j < window``
-    (``window > 0``).  ``p_j = exp(s_j) / (exp(sink_h) + sum exp(s))`` (``sink=None``: the ordinary softmax).  The result times
-    ``out_mult`` goes to ``out[:, out_col0 : out_col0 + H * dv]`` (a fresh ``[T, H * dv]`` tensor by default), which is returned."""
+    (``window > 0``); the first ``keep_first`` positions of the sequence are visible beside them.  ``p_j = exp(s_j) / (exp(sink_h) + sum
+    exp(s))`` (``sink=None``: the ordinary softmax).  The result times ``out_mult`` and (``gate`` ``[T, H]``: one logit per head) times
+    ``sigmoid(gate)`` goes to ``out[:, out_col0 : out_col0 + H * dv]`` (a fresh ``[T, H * dv]`` tensor by default), which is returned."""
     T, H, D = q.shape
     P, G, page, _ = kpool.shape
     dv, rep = vpool.shape[3], H // G
@@ -834,11 +852,12 @@ def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, si
         V = vpool[pg, :, off].float().repeat_interleave(rep, 1)                           # [n, H, dv]
         sc = torch.einsum("thd,nhd->thn", qf[s:e], K) * scale
         qpos = (c0 + torch.arange(e - s, device=q.device))[:, None]
-        mask = idx[None, :] > qpos
+        hidden = torch.zeros(e - s, n, dtype=torch.bool, device=q.device)
         if block > 0:
-            mask = mask | ((idx[None, :] // block) != (qpos // block))
+            hidden = hidden | ((idx[None, :] // block) != (qpos // block))
         if window > 0:
-            mask = mask | (idx[None, :] <= qpos - window)
+            hidden = hidden | (idx[None, :] <= qpos - window)
+        mask = (idx[None, :] > qpos) | (hidden & (idx[None, :] >= keep_first))
         sc = sc.masked_fill(mask[:, None, :], float("-inf"))
         if sink is None:
             p = torch.softmax(sc, -1)
@@ -846,6 +865,8 @@ def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, si
             sk = sink.float().view(1, H, 1).expand(e - s, H, 1)
             p = torch.softmax(torch.cat([sc, sk], -1), -1)[..., :n]
         res[s:e] = torch.einsum("thn,nhv->thv", p, V)
+    if gate is not None:
+        res = res * torch.sigmoid(gate.float())[:, :, None]
     res = res.view(T, H * dv) * out_mult
     if out is None:
         return res.to(out_dtype)
@@ -854,9 +875,10 @@ def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, si
 
 
 def sink_attention_prefill(q, kpool, vpool, sink, meta: BatchMeta, scale: float, block: int = 0, window: int = 0, out_mult: float = 1.0,
-                           out_dtype: torch.dtype = torch.float32, out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
-    """Single-sequence prefill form of :func:`sink_attention` (the CUDA backend runs it as matrix products); same math here."""
-    return sink_attention(q, kpool, vpool, sink, meta, scale, block, window, out_mult, out_dtype, out, out_col0)
+                           out_dtype: torch.dtype = torch.float32, out: Optional[torch.Tensor] = None, out_col0: int = 0, keep_first: int = 0,
+                           gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Prefill form of :func:`sink_attention` (the CUDA backend runs it on the tensor cores); same math here."""
+    return sink_attention(q, kpool, vpool, sink, meta, scale, block, window, out_mult, out_dtype, out, out_col0, keep_first, gate)
 
 
 def mingru_scan(rows: torch.Tensor, z_col0: int, x_col0: int, g_col0: int, width: int, state: torch.Tensor, meta: BatchMeta,
@@ -916,3 +938,36 @@ def moe_relu2_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, Wu: L
         h = (torch.relu(x[tok].float() @ Wu.weight[e].float().t()) ** 2).to(x.dtype)
         y.index_add_(0, tok, (h.float() @ Wd.weight[e].float().t()) * w[tok, slot].float()[:, None])
     return y
+
+
+# ---- selective scan with one step size per channel, GELU-GLU feed-forward
+def selective_scan(x: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, bc: torch.Tensor, b_col0: int, c_col0: int,
+                   D: torch.Tensor, gate: Optional[torch.Tensor], state: torch.Tensor, meta: BatchMeta) -> torch.Tensor:
+    """Selective state-space recurrence per channel ``c`` and state entry ``n`` (fp32): ``dt = softplus(dt_raw + dt_bias)``,
+    ``S[c, n] <- exp(-exp(A_log[c, n]) dt_c) S[c, n] + dt_c x_c B_n``, ``y_c = sum_n S[c, n] C_n + D_c x_c``; the result is ``y * silu(gate)``
+    (``gate=None``: ``y``).  ``x`` ``[T, inner]`` (after the short convolution), ``dt_raw`` fp32 ``[T, inner]``, ``B`` / ``C`` = columns
+    ``b_col0`` / ``c_col0`` on of ``bc``, ``state`` ``[slots, inner, N]`` fp32.  Returns ``[T, inner]`` in the dtype of ``x``."""
+    T, I = x.shape
+    N = A_log.shape[1]
+    xf = x.float()
+    dt = F.softplus(dt_raw.float() + dt_bias.float(), threshold=30.0)
+    A = -torch.exp(A_log.float())
+    B, Cm = bc[:, b_col0:b_col0 + N].float(), bc[:, c_col0:c_col0 + N].float()
+    y = torch.empty(T, I, dtype=torch.float32, device=x.device)
+    for s, e, c0, slot in _seq_ranges(meta):
+        if e == s:
+            continue
+        S = state[slot].clone() if c0 > 0 else torch.zeros_like(state[slot])
+        for t in range(s, e):
+            S = torch.exp(dt[t][:, None] * A) * S + (dt[t] * xf[t])[:, None] * B[t][None, :]
+            y[t] = S @ Cm[t] + D.float() * xf[t]
+        state[slot] = S
+    if gate is not None:
+        y = y * F.silu(gate.float())
+    return y.to(x.dtype)
+
+
+def gelu_gated_up(x: torch.Tensor, Wg: LinearWeight, Wu: LinearWeight) -> torch.Tensor:
+    """First half of a GELU-GLU feed-forward: ``gelu_tanh(x Wg^T) * (x Wu^T)`` (one fused GEMM on the b200 backend)."""
+    g, u = linear(x, Wg, out_dtype=torch.float32), linear(x, Wu, out_dtype=torch.float32)
+    return (F.gelu(g, approximate="tanh") * u).to(x.dtype)

@@ -39,7 +39,7 @@ def synthetic_model_dir(name: str) -> str:
     mlx-community checkpoint), so ``mlx-sharding-api --model synthetic:llama3-8b`` serves a full-size model without a download."""
     import tempfile
 
-    from ..config import deepseek_v2_lite_config, gemma2_9b_config, gifetar_config, gokapel_config, llama3_8b_config
+    from ..config import deepseek_v2_lite_config, gemma2_9b_config, gifetar_config, gokapel_config, llama3_8b_config, podurax_config
 
     tiny = lambda: dict(model_type="llama", vocab_size=320, hidden_size=64, intermediate_size=128, num_hidden_layers=4,
                         num_attention_heads=4, num_key_value_heads=2, rms_norm_eps=1e-5, rope_theta=10000.0,
@@ -47,8 +47,11 @@ def synthetic_model_dir(name: str) -> str:
     tiny_gifetar = lambda: gifetar_config(width=64, vocab=320, layers=3, heads=4, kv_heads=2, dim=16, vdim=24, experts=4, top=2, expert_ff=32)
     tiny_gokapel = lambda: gokapel_config(width=64, vocab=320, blocks=1, heads=4, kv_heads=2, dim=16, vdim=24, ff=96, experts=4, top=2, expert_ff=32,
                                           block_size=24, gru_width=40)
+    tiny_podurax = lambda: podurax_config(width=64, vocab=320, blocks=1, heads=4, kv_heads=2, dim=16, vdim=24, ff=96, window=24, keep_first=3, inner=80,
+                                          state=8, dt_rank=5)
     canned = {"deepseek-v2-lite": deepseek_v2_lite_config, "llama3-8b": llama3_8b_config, "gemma2-9b": gemma2_9b_config,
-              "tiny-llama": tiny, "gifetar": gifetar_config, "tiny-gifetar": tiny_gifetar, "gokapel": gokapel_config, "tiny-gokapel": tiny_gokapel}
+              "tiny-llama": tiny, "gifetar": gifetar_config, "tiny-gifetar": tiny_gifetar, "gokapel": gokapel_config, "tiny-gokapel": tiny_gokapel,
+              "podurax": podurax_config, "tiny-podurax": tiny_podurax}
     if name not in canned:
         raise FileNotFoundError(f"unknown synthetic model '{name}' (known: {sorted(canned)})")
     d = _SYNTH_DIRS.get(name)
@@ -98,7 +101,7 @@ def key_in_shard(key: str, spec: ShardSpec, tied_embeddings: bool = False, model
     """True if checkpoint tensor ``key`` belongs to stage ``spec`` (half-layer boundaries included)."""
     if "rotary_emb.inv_freq" in key:
         return False
-    if model_type in ("perelorn", "gusolorn", "gifetar", "gokapel"):       # keys: embed, side.embed, l<i>.*, final.norm, head (single-stage model: everything or a layer range)
+    if model_type in ("perelorn", "gusolorn", "gifetar", "gokapel", "podurax"):       # keys: embed, side.embed, l<i>.*, final.norm, head (single-stage model: everything or a layer range)
         m = re.match(r"l(\d+)\.", key)
         if m:
             return spec.owns_layer(int(m.group(1)))
@@ -263,6 +266,9 @@ def random_state_dict(cfg: ModelConfig, spec: Optional[ShardSpec] = None, dtype=
         return
     if cfg.model_type == "gokapel":
         yield from _gokapel_random(cfg, gen, dtype, device, seed)
+        return
+    if cfg.model_type == "podurax":
+        yield from _podurax_random(cfg, gen, dtype, device, seed)
         return
     H = cfg.hidden_size
     q = quantization
@@ -602,3 +608,47 @@ def _gokapel_random(cfg: ModelConfig, gen, dtype, device, seed: int, ranks=(32, 
                 yield p + "mlp.shared.up", lin(Fs, W)
                 yield p + "mlp.shared.down", lin(W, Fs)
     yield from norm("final.norm")
+
+
+def _podurax_random(cfg: ModelConfig, gen, dtype, device, seed: int):
+    """Random-init Podurax tensors (checkpoint names and shapes of that design: RMS norms, selective-scan layers with a short convolution,
+    low-rank step sizes and a decay per channel and state entry, biased attention projections with a value-mixing scalar and a gate per
+    head, gate / up / down matrices, an LM head of its own)."""
+    gen.manual_seed(seed * 1000003 + 53)
+    W = cfg.hidden_size
+    rn = lambda *shape, std=1.0: torch.randn(*shape, generator=gen, device=device, dtype=torch.float32) * std
+    lin = lambda o, i, gain=1.0: (rn(o, i) * gain / (i ** 0.5)).to(dtype)
+    vec = lambda n: (1.0 + 0.1 * rn(n)).to(dtype)
+    small = lambda n, std=0.2: (std * rn(n)).to(dtype)
+    yield "embed", rn(cfg.vocab_size, W).to(dtype)
+    for i, L in enumerate(cfg.layer_specs):
+        p, m, mlp = f"l{i}.", L["mixer"], L["mlp"]
+        yield p + "norm1", vec(W)
+        if L["type"] == "mamba1":
+            I, N, R, K = (int(m[k]) for k in ("inner", "state", "dt_rank", "conv"))
+            yield p + "mix.in", lin(2 * I, W)
+            yield p + "mix.conv", (0.5 * rn(I, K)).to(dtype)
+            yield p + "mix.conv.b", small(I)
+            yield p + "mix.x", lin(R + 2 * N, I)
+            yield p + "mix.dt", lin(I, R)
+            yield p + "mix.dt.b", (rn(I) - 2.0).to(dtype)
+            yield p + "mix.A_log", torch.log(torch.rand(I, N, generator=gen, device=device) * N + 0.05).to(dtype)
+            yield p + "mix.D", vec(I)
+            yield p + "mix.o", lin(W, I)
+        else:
+            H, G, D, V = (int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * V)):
+                yield p + "mix." + n, lin(rows, W)
+                yield p + "mix." + n + ".b", small(rows)
+            if m.get("v_mix"):
+                yield p + "mix.vmix", (0.4 + 0.1 * rn(1))[0].to(dtype)
+            yield p + "mix.g", lin(H, W)
+            yield p + "mix.o", lin(W, H * V)
+        if mlp:
+            F = int(mlp["ff"])
+            yield p + "norm2", vec(W)
+            yield p + "mlp.gate", lin(F, W)
+            yield p + "mlp.up", lin(F, W)
+            yield p + "mlp.down", lin(W, F)
+    yield "final.norm", vec(W)
+    yield "head", lin(cfg.vocab_size, W)
