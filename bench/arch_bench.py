@@ -1,4 +1,8 @@
-"""Hybrid designs beside the framework's closest existing model.  ``--arch gokapel``: Gokapel beside Gusolorn (the other stack of recurrent
+"""Hybrid designs beside the framework's closest existing model.  ``--arch podurax``: Podurax beside Gokapel (the other stack of recurrent
+layers and attention with a sink over its own key / value pools on an fp32 residual) at equal width, depth, heads and feed-forward, and each
+of its kernels beside the like kernel (selective scan with a step size per channel / Perelorn's selective scan with one per head, attention
+in a window beside kept first tokens with a gate / Gokapel's inside blocks and Llama's paged and flash attention, prologue with value mixing /
+Gokapel's, scaled residual add + norm / stream step with dynamic tanh, GELU-GLU product / clamped-GLU product).  ``--arch gokapel``: Gokapel beside Gusolorn (the other stack of recurrent
 layers, attention over paged rows, dense and routed feed-forwards on an fp32 residual) at equal width, depth, heads and experts, and each of
 its kernels beside the like kernel (gated delta rule / mLSTM scan, block-local attention with a sink / windowed latent attention and
 differential attention, stream step with dynamic tanh / scaled residual add + norm, query/key norm + rotation + append / latent prologue,
@@ -28,7 +32,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
-from mlx_sharding_b200.config import deepseek_v2_lite_config, gifetar_config, gokapel_config, gusolorn_config, perelorn_config  # noqa: E402
+from mlx_sharding_b200.config import deepseek_v2_lite_config, gifetar_config, gokapel_config, gusolorn_config, perelorn_config, podurax_config  # noqa: E402
 from mlx_sharding_b200.ops.meta import BatchMeta  # noqa: E402
 from mlx_sharding_b200.parallel.pipeline import StageExecutor  # noqa: E402
 from mlx_sharding_b200.utils.loader import random_model  # noqa: E402
@@ -463,7 +467,113 @@ def gokapel_main(sizes=(1024, 2048)):
         print(json.dumps(dict(bench="arch-kernel", roofline=f"{hbm} GB/s {tag}", **row)), flush=True)
 
 
+def podurax_kernel_table(width, dev, hbm):
+    """Podurax's kernels alone at one layer's shapes beside the like kernels; bytes = what the kernel must move.  Decode = 64 sequences at
+    context 2048, prefill = one 2048-token prompt; windows (and Gokapel's blocks) of 1024 positions, 16 kept first tokens."""
+    from mlx_sharding_b200.ops import b200 as O
+    from mlx_sharding_b200.ops.weights import LinearWeight
+
+    rows = []
+    H, G, D, V, W, WIN, KEEP = 16, 4, 128, 128, width, 1024, 16
+    I, N, R = 2 * W, 16, W // 16
+    bf = torch.bfloat16
+
+    def add(name, ms, nbytes, like=None, flops=None):
+        r = dict(kernel=name, ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), frac_hbm=round(nbytes / ms / 1e6 / hbm, 3))
+        if flops:
+            r["tflops"] = round(flops / ms / 1e9, 1)
+        if like:
+            r["like_kernel"] = like
+        rows.append(r)
+
+    for phase, B, q, ctx0 in (("decode", 64, 1, 2047), ("prefill", 1, 2048, 0)):
+        meta, _ = step_meta(B, q, ctx0, dev, True)
+        T, npg = B * q, 1 + B * ((ctx0 + q + PS - 1) // PS)
+        # ---- selective scans: state read and written once per step (decode)
+        st = torch.zeros(B + 1, I, N, device=dev)
+        u = torch.randn(T, 2 * I, device=dev).to(bf)
+        xc, dt, bc = u[:, :I].contiguous(), torch.randn(T, I, device=dev), torch.randn(T, R + 2 * N, device=dev).to(bf)
+        dtb, alog, Dv = torch.randn(I, device=dev) - 3.0, torch.log(torch.rand(I, N, device=dev) * N + 0.05), torch.ones(I, device=dev)
+        sbytes = (2 * B * I * N * 4 if q == 1 else 0) + T * I * (2 + 4 + 2 + 2) + T * 2 * N * 2 + I * N * 4
+        ms = timed(lambda: O.selective_scan(xc, dt, dtb, alog, bc, R, R + N, Dv, u[:, I:], st, meta))
+        add(f"selective_scan {phase}", ms, sbytes)
+        H2, P2, N2 = 2 * W // 64, 64, 128
+        xbc, st2 = torch.randn(T, H2 * P2 + 2 * N2, device=dev).to(bf), torch.zeros(B + 1, H2, N2, P2, device=dev)
+        dt2, db2, al2, D2 = torch.randn(T, H2, device=dev).to(bf), torch.zeros(H2, device=dev), torch.zeros(H2, device=dev), torch.ones(H2, device=dev)
+        ms = timed(lambda: O.ssm_scan(xbc, dt2, db2, al2, D2, st2, meta, H2, P2, N2, 1))
+        add(f"ssm_scan (Perelorn) {phase}", ms, (2 * B * H2 * N2 * P2 * 4 if q == 1 else 0) + T * (H2 * P2 + 2 * N2 + H2) * 2 + T * H2 * P2 * 4,
+            like=f"selective_scan {phase}")
+        cw, cb, cst = torch.randn(I, 4, device=dev), torch.zeros(I, device=dev), torch.zeros(B + 1, 3, I, device=dev).to(bf)
+        ms = timed(lambda: O.causal_conv_silu(u[:, :I], cw, cb, cst, meta))
+        add(f"causal_conv_silu (shared) {phase}", ms, T * I * 4 + (2 * B * 3 * I * 2 if q == 1 else 0))
+        # ---- attention
+        kp, vp = torch.randn(npg, G, PS, D, device=dev).to(bf), torch.randn(npg, G, PS, V, device=dev).to(bf)
+        rows_ = torch.randn(T, H * D + G * D + G * V + H, device=dev).to(bf)
+        vf, gate = torch.randn(T, G * V, device=dev).to(bf), rows_[:, H * D + G * (D + V):]
+        inv = (10000.0 ** (-2.0 * torch.arange(D // 4, dtype=torch.float64) / (D // 2))).float().to(dev)
+        sink, qn = torch.zeros(H, device=dev), torch.ones(D, device=dev)
+        prol = lambda: O.qk_norm_rope_append(rows_, 0, H * D, H * D + G * D, H, D, None, None, 1e-6, inv, kp, vp, meta, half=True, norm_after=True,
+                                             rot_mult=1.1, v_first=vf, v_lambda=0.4)
+        qf = prol()
+        pbytes = T * (H * D + G * D + G * V) * 2 + T * H * D * 4 + T * G * (D + V) * 2
+        add(f"qk_norm_rope_append(value mixing) {phase}", timed(prol), pbytes + T * G * V * 2)
+        ms = timed(lambda: O.qk_norm_rope_append(rows_, 0, H * D, H * D + G * D, H, D, qn, qn, 1e-6, inv, kp, vp, meta))
+        add(f"qk_norm_rope_append (Gokapel) {phase}", ms, pbytes, like=f"qk_norm_rope_append(value mixing) {phase}")
+        n_of = lambda p: min(p + 1, WIN) + min(KEEP, max(0, p - WIN + 1))
+        pairs = B * n_of(ctx0) if q == 1 else sum(n_of(p) for p in range(q))
+        abytes = (B * n_of(ctx0) * G * (D + V) * 2 if q == 1 else q * G * (D + V) * 2) + T * H * (D * 4 + V * 2)
+        ms = timed(lambda: O.sink_attention(qf, kp, vp, sink, meta, D ** -0.5, 0, WIN, 1.0, bf, keep_first=KEEP, gate=gate))
+        name = f"sink_attention(window {WIN}, keep {KEEP}, gate) {phase}"
+        add(name, ms, abytes, flops=2 * H * (D + V) * pairs)
+        bpairs = B * ((ctx0 % WIN) + 1) if q == 1 else sum((p % WIN) + 1 for p in range(q))
+        ms = timed(lambda: O.sink_attention(qf, kp, vp, sink, meta, D ** -0.5, WIN, 0, 1.0, bf))
+        add(f"sink_attention(block {WIN}) (Gokapel) {phase}", ms, (B * WIN * G * (D + V) * 2 if q == 1 else q * G * (D + V) * 2) + T * H * (D * 4 + V * 2), like=name,
+            flops=2 * H * (D + V) * bpairs)
+        qb = qf.to(bf)
+        lpairs = B * (ctx0 + 1) if q == 1 else q * (q + 1) // 2
+        ms = timed(lambda: O.paged_attention(qb, kp, vp, meta, D ** -0.5))
+        add(f"paged / flash attention, all keys (Llama) {phase}", ms, (B * (ctx0 + 1) * G * (D + V) * 2 if q == 1 else q * G * (D + V) * 2) + T * H * (D + V) * 2, like=name,
+            flops=2 * H * (D + V) * lpairs)
+        dq, dkp = torch.randn(T, H * 2 * 64, device=dev).to(bf), torch.randn(npg, G, PS, 128, device=dev).to(bf)
+        ms = timed(lambda: O.diff_attention(dq, dkp, vp, meta, H, 0.125, 30.0, 0.1, 1024.0, 0.8, 1e-5, 0.2))
+        add(f"diff_attention, all keys (Gifetar) {phase}", ms, (B * (ctx0 + 1) * G * (128 + V) * 2 if q == 1 else q * G * (128 + V) * 2) + T * H * (128 + V) * 2, like=name)
+        # ---- residual step and feed-forward
+        x, y, nw = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev), torch.ones(W, device=dev)
+        add(f"scaled_add_norm_(mult) {phase}", timed(lambda: O.scaled_add_norm_(x, y, None, nw, 1e-6, bf, mult=0.5)), T * W * (4 * 3 + 2))
+        xs, two = torch.randn(T, 2, W, device=dev), torch.eye(2, device=dev)
+        ms = timed(lambda: O.hyper_step_(xs, y, None, None, None, two, two[0].contiguous(), 0.5, two[0].contiguous(), 0.7, nw, nw, bf))
+        add(f"hyper_step_(2 streams) (Gokapel) {phase}", ms, T * W * (4 * 5 + 2), like=f"scaled_add_norm_(mult) {phase}")
+        F = 4 * W
+        wg, wu = (LinearWeight(weight=(torch.randn(F, W, device=dev) * W ** -0.5).to(bf)) for _ in range(2))
+        h = torch.randn(T, W, device=dev).to(bf)
+        fb, ff = 2 * F * W * 2 + T * (W + F) * 2, 4 * T * F * W
+        add(f"gelu_gated_up {phase}", timed(lambda: O.gelu_gated_up(h, wg, wu)), fb, flops=ff)
+        add(f"clamped_gated_up (Gusolorn) {phase}", timed(lambda: O.clamped_gated_up(h, wg, wu, 7.0)), fb, like=f"gelu_gated_up {phase}", flops=ff)
+        for nm, n_, k_ in (("in projection", 2 * I, W), ("x projection", R + 2 * N, I), ("step-size projection", I, R), ("out projection", W, I)):
+            w_, x_ = LinearWeight(weight=(torch.randn(n_, k_, device=dev) * k_ ** -0.5).to(bf)), torch.randn(T, k_, device=dev).to(bf)
+            add(f"linear_any {nm} {n_}x{k_} {phase}", timed(lambda: O.linear_any(x_, w_, bf)), n_ * k_ * 2 + T * (n_ + k_) * 2, flops=2 * T * n_ * k_)
+    return rows
+
+
+def podurax_main(sizes=(1024, 2048)):
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm, tag = peaks()
+    for width in sizes:
+        for name, cfg in (("podurax", podurax_config(width=width, vocab=32000, blocks=2, heads=16, kv_heads=4, ff=4 * width)),
+                          ("gokapel", gokapel_config(width=width, vocab=32000, blocks=2, heads=16, kv_heads=4, ff=4 * width, experts=16, top=2, expert_ff=width // 2))):
+            m = random_model(cfg, dtype=torch.bfloat16, device=dev, seed=1)
+            r = model_runs(name, m, 32, 1024, 2048, dev, True)
+            print(json.dumps(dict(bench="arch", model=name, width=width, layers=len(cfg["layers"]), **{k: (round(v, 3) if isinstance(v, float) else v) for k, v in r.items()})), flush=True)
+            del m
+            torch.cuda.empty_cache()
+    for row in podurax_kernel_table(sizes[-1], dev, hbm):
+        print(json.dumps(dict(bench="arch-kernel", roofline=f"{hbm} GB/s {tag}", **row)), flush=True)
+
+
 def main(sizes=(1024, 2048), arch="perelorn"):
+    if arch == "podurax":
+        return podurax_main(sizes)
     if arch == "gokapel":
         return gokapel_main(sizes)
     if arch == "gusolorn":

@@ -52,6 +52,10 @@ struct SinkForm {                            // what the SINK form adds (unused 
   float out_mult;
 };
 
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(smem)));
+}
+
 template <int DK, int DV, bool SINK>
 __global__ void __launch_bounds__(kThreads)
 flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long long q_ld_h,
@@ -98,19 +102,24 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int r_lo = lane >> 2, c2 = (lane & 3) * 2;
 
-  auto load_tile = [&](int j, int buf) {
-    __nv_bfloat16* dK = sK + buf * kBN * KS;
-    __nv_bfloat16* dV = sV + buf * kBN * VS;
+  // two threads per key row, 16-byte chunks alternating between them; the row's page is looked up one tile before its copy is issued
+  const int lr = threadIdx.x >> 1, lc = threadIdx.x & 1;
+  auto row_of = [&](int j) {
+    const int pos = min(j * kBN + lr, kv_end - 1);         // behind the end: the last key, masked later
+    return ((size_t)bt[pos / page] * kv_heads + hk) * page + (pos % page);
+  };
+  auto load_tile = [&](size_t row, int buf) {
     const int KC = D / 8, VC = V / 8;
-    for (int i = threadIdx.x; i < kBN * (KC + VC); i += kThreads) {
-      const int r = i / (KC + VC), c = i % (KC + VC);
-      int pos = j * kBN + r;
-      if (pos >= kv_end) pos = kv_end - 1;  // clamp: masked later
-      const size_t pg = bt[pos / page];
-      const size_t row = (pg * kv_heads + hk) * page + (pos % page);
-      if (c < KC) cp_async16(dK + r * KS + c * 8, kpool + row * D + c * 8);
-      else cp_async16(dV + r * VS + (c - KC) * 8, vpool + row * V + (c - KC) * 8);
-    }
+    __nv_bfloat16* dK = sK + (buf * kBN + lr) * KS;
+    __nv_bfloat16* dV = sV + (buf * kBN + lr) * VS;
+    const __nv_bfloat16* gK = kpool + row * D;
+    const __nv_bfloat16* gV = vpool + row * V;
+#pragma unroll
+    for (int c = 0; c < DK / 16; ++c)
+      if (!SINK || 2 * c + lc < KC) cp_async16(dK + (2 * c + lc) * 8, gK + (2 * c + lc) * 8);
+#pragma unroll
+    for (int c = 0; c < DV / 16; ++c)
+      if (!SINK || 2 * c + lc < VC) cp_async16(dV + (2 * c + lc) * 8, gV + (2 * c + lc) * 8);
     cp_async_commit();
   };
 
@@ -156,53 +165,69 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   const int qpos_a = pos0 + warp * 16 + r_lo, qpos_b = qpos_a + 8;
 
   const int lo_a = SINK ? first_key(qpos_a) : 0, lo_b = SINK ? first_key(qpos_b) : 0;
-  load_tile(tile_at(0), 0);
+  load_tile(row_of(tile_at(0)), 0);
+  size_t next_row = ntiles > 1 ? row_of(tile_at(1)) : 0;
+  const int last_lo = SINK ? first_key(pos0 + rows - 1) : 0;
   for (int j = 0; j < ntiles; ++j) {
     const int buf = j & 1;
-    if (j + 1 < ntiles) { load_tile(tile_at(j + 1), buf ^ 1); cp_async_wait<1>(); }
-    else cp_async_wait<0>();
+    if (j + 1 < ntiles) {
+      load_tile(next_row, buf ^ 1);
+      if (j + 2 < ntiles) next_row = row_of(tile_at(j + 2));
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
     __syncthreads();
     const __nv_bfloat16* tK = sK + buf * kBN * KS;
     const __nv_bfloat16* tV = sV + buf * kBN * VS;
     // ---- S = Q K^T  (16 x 64 per warp)
     float s[kBN / 8][4];
 #pragma unroll
-    for (int nt = 0; nt < kBN / 8; ++nt) {
-      s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
-      const __nv_bfloat16* kr = tK + (nt * 8 + r_lo) * KS + c2;
+    for (int nt = 0; nt < kBN / 8; ++nt) s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f;
+    {
+      // lanes 0-7: keys nt*8 .. +7 at column ks*16, 8-15: the same keys at column +8, 16-31: the next eight keys
+      const __nv_bfloat16* kr = tK + ((lane & 7) + ((lane >> 4) << 3)) * KS + ((lane >> 3) & 1) * 8;
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ++ks) {
-        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(kr + ks * 16);
-        const uint32_t b1 = *reinterpret_cast<const uint32_t*>(kr + ks * 16 + 8);
-        mma_bf16(s[nt], qa[ks], b0, b1);
+#pragma unroll
+        for (int nt = 0; nt < kBN / 8; nt += 2) {
+          uint32_t kb[4];
+          ldmatrix_x4(kb, kr + nt * 8 * KS + ks * 16);
+          mma_bf16(s[nt], qa[ks], kb[0], kb[1]);
+          mma_bf16(s[nt + 1], qa[ks], kb[2], kb[3]);
+        }
       }
     }
-    // ---- scale, causal mask, online softmax (base 2)
+    // ---- mask (tiles that every row of the CTA sees as a whole need none), online softmax (base 2) on the raw scores
     const int kbase = tile_at(j) * kBN;
     float mx_a = m_a, mx_b = m_b;
+    if (kbase + kBN - 1 > pos0 || (SINK && kbase < last_lo && kbase + kBN > x.keep)) {
+#pragma unroll
+      for (int nt = 0; nt < kBN / 8; ++nt) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int kpos = kbase + nt * 8 + c2 + e;
+          if (!(kpos <= qpos_a && (!SINK || kpos >= lo_a || kpos < x.keep))) s[nt][e] = -INFINITY;
+          if (!(kpos <= qpos_b && (!SINK || kpos >= lo_b || kpos < x.keep))) s[nt][2 + e] = -INFINITY;
+        }
+      }
+    }
 #pragma unroll
     for (int nt = 0; nt < kBN / 8; ++nt) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int kpos = kbase + nt * 8 + c2 + e;
-        const bool va = kpos <= qpos_a && (!SINK || kpos >= lo_a || kpos < x.keep), vb = kpos <= qpos_b && (!SINK || kpos >= lo_b || kpos < x.keep);
-        s[nt][e] = va ? s[nt][e] * scale_log2 : -INFINITY;
-        s[nt][2 + e] = vb ? s[nt][2 + e] * scale_log2 : -INFINITY;
-        mx_a = fmaxf(mx_a, s[nt][e]);
-        mx_b = fmaxf(mx_b, s[nt][2 + e]);
-      }
+      mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
+      mx_b = fmaxf(mx_b, fmaxf(s[nt][2], s[nt][3]));
     }
     mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1)); mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
     mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1)); mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 2));
-    const float ca = (mx_a == -INFINITY) ? 1.f : exp2f(m_a - mx_a);
-    const float cb = (mx_b == -INFINITY) ? 1.f : exp2f(m_b - mx_b);
-    const float ba = (mx_a == -INFINITY) ? 0.f : mx_a, bb = (mx_b == -INFINITY) ? 0.f : mx_b;
+    const float ca = (mx_a == -INFINITY) ? 1.f : exp2f((m_a - mx_a) * scale_log2);
+    const float cb = (mx_b == -INFINITY) ? 1.f : exp2f((m_b - mx_b) * scale_log2);
+    const float ba = (mx_a == -INFINITY) ? 0.f : -mx_a * scale_log2, bb = (mx_b == -INFINITY) ? 0.f : -mx_b * scale_log2;
     float sa = 0.f, sb = 0.f;
     uint32_t pa[kBN / 16][4];
 #pragma unroll
     for (int nt = 0; nt < kBN / 8; ++nt) {
-      const float p0 = exp2f(s[nt][0] - ba), p1 = exp2f(s[nt][1] - ba);
-      const float p2 = exp2f(s[nt][2] - bb), p3 = exp2f(s[nt][3] - bb);
+      const float p0 = exp2f(fmaf(s[nt][0], scale_log2, ba)), p1 = exp2f(fmaf(s[nt][1], scale_log2, ba));
+      const float p2 = exp2f(fmaf(s[nt][2], scale_log2, bb)), p3 = exp2f(fmaf(s[nt][3], scale_log2, bb));
       sa += p0 + p1; sb += p2 + p3;
       pa[nt >> 1][(nt & 1) * 2 + 0] = pack_bf16(p0, p1);
       pa[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16(p2, p3);
@@ -231,7 +256,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   const int ra = warp * 16 + r_lo, rb = ra + 8;
   float fa = 1.f, fb = 1.f;
   if constexpr (SINK) {
-    if (x.sink != nullptr) { const float sk = x.sink[hq] * 1.4426950408889634f; l_a += exp2f(sk - m_a); l_b += exp2f(sk - m_b); }
+    if (x.sink != nullptr) { const float sk = x.sink[hq] * 1.4426950408889634f; l_a += exp2f(fmaf(-m_a, scale_log2, sk)); l_b += exp2f(fmaf(-m_b, scale_log2, sk)); }
     fa = fb = x.out_mult;
     if (x.gate != nullptr) {
       auto sig = [&](int r) { return 1.f / (1.f + expf(-__bfloat162float(x.gate[(size_t)(tok0 + r) * x.ld_gate + hq]))); };

@@ -27,19 +27,70 @@ struct SelScanArgs {
 // floats of workspace per sequence (a multiple of 4: the states are read 16 bytes at a time)
 __host__ __device__ inline long long ws_stride(int I, int N, int NS) { return ((long long)NS * I * N + (long long)(NS - 1) * I + 3) / 4 * 4; }
 
-constexpr int kScanThreads = 128;
-constexpr int kScanTokens = 16;             // tokens staged in shared memory at a time
+constexpr int kLanes = 128;                 // compute threads of a CTA (and as many helpers)
 
-// decay factors: the exact path calls expf; bf16 serving folds log2(e) into the rate and uses the hardware's base-2 exponential
+// One step S <- exp(rate dt) S + add.  bf16 serving folds log2(e) into the rate and uses the hardware's base-2 exponential.  Exact mode adds
+// S (exp(rate dt) - 1) for slow decays: a factor close to 1 would carry its last-bit error, which has a sign of its own, through every token
+// of a long memory; the difference to 1 is exact to its own last bit.
 template <typename AT> __device__ __forceinline__ float rate_of(float a_log);
 template <> __device__ __forceinline__ float rate_of<float>(float a_log) { return -expf(a_log); }
 template <> __device__ __forceinline__ float rate_of<__nv_bfloat16>(float a_log) { return -expf(a_log) * 1.4426950408889634f; }
-template <typename AT> __device__ __forceinline__ float decay_of(float rate, float dt);
-template <> __device__ __forceinline__ float decay_of<float>(float rate, float dt) { return expf(rate * dt); }
-template <> __device__ __forceinline__ float decay_of<__nv_bfloat16>(float rate, float dt) {
+template <typename AT> __device__ __forceinline__ float advance(float S, float rate, float dt, float x, float B);
+template <> __device__ __forceinline__ float advance<float>(float S, float rate, float dt, float x, float B) {
+  const float e = rate * dt;
+  return e > -0.5f ? fmaf(S, expm1f(e), fmaf(x, B, S)) : fmaf(S, expf(e), x * B);
+}
+__device__ __forceinline__ float exp2_hw(float v) {
   float r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(rate * dt));
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
   return r;
+}
+template <> __device__ __forceinline__ float advance<__nv_bfloat16>(float S, float rate, float dt, float x, float B) {
+  return fmaf(exp2_hw(rate * dt), S, x * B);
+}
+
+// two floats in one 64-bit register: packed multiply and multiply-add
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r)) : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
+  return r;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(r))
+      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)), "l"(reinterpret_cast<unsigned long long&>(c)));
+  return r;
+}
+
+// one token on SN adjacent state entries: advances S, returns the lane's part of S . C (FOLD: no output)
+template <typename AT, int SN, bool FOLD>
+__device__ __forceinline__ float token(float* S, const float* A, float2 ddx, const float* B, const float* C) {
+  if constexpr (sizeof(AT) == 2) {
+    const float2 d2 = make_float2(ddx.x, ddx.x), x2 = make_float2(ddx.y, ddx.y);
+    float2 y = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < SN; i += 4) {
+      const float4 b = *reinterpret_cast<const float4*>(B + i);
+      const float4 c = FOLD ? b : *reinterpret_cast<const float4*>(C + i);
+#pragma unroll
+      for (int k = 0; k < 4; k += 2) {
+        const float2 r = mul2(make_float2(A[i + k], A[i + k + 1]), d2);
+        const float2 xb = mul2(x2, k == 0 ? make_float2(b.x, b.y) : make_float2(b.z, b.w));
+        const float2 s = fma2(make_float2(exp2_hw(r.x), exp2_hw(r.y)), make_float2(S[i + k], S[i + k + 1]), xb);
+        S[i + k] = s.x; S[i + k + 1] = s.y;
+        if (!FOLD) y = fma2(s, k == 0 ? make_float2(c.x, c.y) : make_float2(c.z, c.w), y);
+      }
+    }
+    return y.x + y.y;
+  } else {
+    float y = 0.f;
+#pragma unroll
+    for (int i = 0; i < SN; ++i) {
+      S[i] = advance<AT>(S[i], A[i], ddx.x, ddx.y, B[i]);
+      if (!FOLD) y = fmaf(S[i], C[i], y);
+    }
+    return y;
+  }
 }
 
 template <int SN> __device__ __forceinline__ void load_states(const float* p, int n0, int N, bool vec, float* S) {
@@ -65,53 +116,131 @@ template <int SN> __device__ __forceinline__ void store_states(float* p, int n0,
   }
 }
 
-// L lanes share a channel, lane l holding the state entries SN l .. SN l + SN - 1 in registers; a CTA runs kScanThreads / L channels of one
-// sequence (and of one time slice).  The operands of kTok tokens are staged in shared memory as floats (step sizes through the softplus
-// once per channel); the outputs go back through shared memory so that gate and store are coalesced.
+// the barrier both sides of a CTA arrive at (named: the two sides sit in different branches)
+__device__ __forceinline__ void round_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(2 * kLanes) : "memory"); }
+
+// L lanes share a channel, lane l holding the state entries SN l .. SN l + SN - 1 in registers; a CTA runs 128 / L channels of one
+// sequence (and of one time slice) with 128 compute threads, which touch shared memory only, and 128 helpers, which stage the operands of
+// TOK tokens ahead (step sizes through the softplus once per channel) and finish the outputs of TOK tokens behind (D x, gate, store); both
+// sides work on two buffers with one barrier per TOK tokens, and the helpers' global loads are issued one round before they are used.
+// Tokens behind the end are staged as zero step sizes, which leave the state as it is.
 //
-// The recurrence is linear in S with a diagonal decay, so a long portion is cut into NS slices of tokens.  FOLD: the slice's end state from
-// a zero start and its sum of step sizes (the product of its decays is exp(-A sum dt)) -> workspace; slice 0 also copies the state at the
-// step's start there.  Main form: the start of a slice is folded from the slices before it, then its tokens run with outputs; the slice
-// with the sequence's last token writes the state back.                    grid (ceil(I / channels), B, NS)
-template <typename AT, int L, int SN, bool FOLD>
-__global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(SelScanArgs a, int kTok) {
-  constexpr int CPB = kScanThreads / L, NP = L * SN;
-  extern __shared__ __align__(16) float smem[];
-  float* Bs = smem;                         // [tok][NP]
-  float* Cs = Bs + kTok * NP;               // [tok][NP]
-  float* ds = Cs + kTok * NP;               // [tok][CPB]
-  float* xs = ds + kTok * CPB;              // [tok][CPB]
-  float* ys = xs + kTok * CPB;              // [tok][CPB]
-  const int b = blockIdx.y, sl = blockIdx.z, I = a.I, N = a.N, NS = a.NS;
-  const int c_0 = blockIdx.x * CPB, ch = threadIdx.x / L, l = threadIdx.x % L, c = c_0 + ch, n0 = l * SN;
+// The recurrence is linear in S with a diagonal decay, so a long portion on few channels is cut into NS slices of tokens.  FOLD: the
+// slice's end state from a zero start and its sum of step sizes (the product of its decays is exp(-A sum dt)) -> workspace; slice 0 also
+// copies the state at the step's start there.  Main form: the start of a slice is folded from the slices before it, then its tokens run
+// with outputs; the slice with the sequence's last token writes the state back.                  grid (ceil(I / channels), B, NS)
+template <typename AT, int L, int SN, int TOK, bool FOLD>
+__global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs a) {
+  constexpr int CPB = kLanes / L, NP = L * SN, EPT = (TOK * CPB + kLanes - 1) / kLanes, BPT = (TOK * NP + kLanes - 1) / kLanes;
+  __shared__ __align__(16) float Bs[2][TOK * NP];
+  __shared__ __align__(16) float Cs[FOLD ? 1 : 2][FOLD ? 4 : TOK * NP];
+  __shared__ __align__(16) float2 ds[2][TOK * CPB];         // (dt, dt x)
+  __shared__ __align__(16) float ys[FOLD ? 1 : 2][FOLD ? 4 : TOK * CPB];
+  const int b = blockIdx.y, sl = blockIdx.z, I = a.I, N = a.N, NS = a.NS, c_0 = blockIdx.x * CPB;
   const int s = a.cu[b], q = a.cu[b + 1] - s;
   if (q == 0) return;
   const int len = (q + NS - 1) / NS, j_0 = sl * len, j_1 = min(q, j_0 + len);
   if (j_0 >= j_1) return;
+  const int tiles = (j_1 - j_0 + TOK - 1) / TOK;
+  const long long IN = (long long)I * N;
+  float* ws = a.ws + b * ws_stride(I, N, NS);
+  if (threadIdx.x >= kLanes) {
+    // ---- helpers
+    if (FOLD && j_1 == q) return;             // nothing follows this slice (the compute threads leave as well, before any barrier)
+    const int tid = threadIdx.x - kLanes;
+    const AT* X = reinterpret_cast<const AT*>(a.x);
+    const AT* BC = reinterpret_cast<const AT*>(a.bc);
+    const AT* Z = reinterpret_cast<const AT*>(a.gate);
+    float rd[EPT], rx[EPT], rb[BPT], rc[BPT], ex[EPT], ez[EPT], bias[EPT], Dk[EPT];
+#pragma unroll
+    for (int i = 0; i < EPT; ++i) {
+      const int k = c_0 + (tid + i * kLanes) % CPB;
+      bias[i] = k < I ? a.dt_bias[k] : 0.f;
+      Dk[i] = !FOLD && k < I ? a.D[k] : 0.f;
+    }
+    auto fetch = [&](int tile) {              // operands of a tile -> registers
+#pragma unroll
+      for (int i = 0; i < EPT; ++i) {
+        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
+        const bool ok = e < TOK * CPB && j < j_1 && k < I;
+        rd[i] = ok ? a.dt[(long long)(s + j) * a.ld_dt + k] : -INFINITY;
+        rx[i] = ok ? ldf<AT>(X + (long long)(s + j) * a.ld_x + k) : 0.f;
+      }
+#pragma unroll
+      for (int i = 0; i < BPT; ++i) {
+        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / NP, n = e % NP;
+        const bool ok = e < TOK * NP && j < j_1 && n < N;
+        const AT* row = BC + (long long)(s + j) * a.ld_bc + n;
+        rb[i] = ok ? ldf<AT>(row + a.b0) : 0.f;
+        if (!FOLD) rc[i] = ok ? ldf<AT>(row + a.c0) : 0.f;
+      }
+    };
+    auto stage = [&](int buf) {
+#pragma unroll
+      for (int i = 0; i < EPT; ++i) {
+        const int e = tid + i * kLanes;
+        const float d = softplus_f(rd[i] + bias[i]);            // -inf: 0
+        if (TOK * CPB % kLanes == 0 || e < TOK * CPB) ds[buf][e] = make_float2(d, d * rx[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < BPT; ++i) {
+        const int e = tid + i * kLanes;
+        if (TOK * NP % kLanes == 0 || e < TOK * NP) { Bs[buf][e] = rb[i]; if (!FOLD) Cs[buf][e] = rc[i]; }
+      }
+    };
+    auto fetch_out = [&](int tile) {          // x and gate of a tile whose outputs are finished next round
+#pragma unroll
+      for (int i = 0; i < EPT; ++i) {
+        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
+        const bool ok = e < TOK * CPB && j < j_1 && k < I;
+        ex[i] = ok ? ldf<AT>(X + (long long)(s + j) * a.ld_x + k) : 0.f;
+        ez[i] = ok && Z != nullptr ? ldf<AT>(Z + (long long)(s + j) * a.ld_g + k) : 0.f;
+      }
+    };
+    auto finish = [&](int tile) {
+#pragma unroll
+      for (int i = 0; i < EPT; ++i) {
+        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
+        if (e >= TOK * CPB || j >= j_1 || k >= I) continue;
+        float y = ys[tile & 1][e] + Dk[i] * ex[i];
+        if (Z != nullptr) y *= silu_f(ez[i]);
+        stf<AT>((AT*)a.out + (long long)(s + j) * I + k, y);
+      }
+    };
+    fetch(0);
+    stage(0);
+    fetch(1);
+    round_barrier();
+    for (int k = 0; k < tiles; ++k) {         // round k: tile k is computed
+      if (k + 1 < tiles) stage((k + 1) & 1);
+      if (!FOLD && k > 0) finish(k - 1);
+      if (k + 2 < tiles) fetch(k + 2);
+      if (!FOLD) fetch_out(k);
+      round_barrier();
+    }
+    if (!FOLD) finish(tiles - 1);
+    return;
+  }
+  // ---- compute threads
+  const int ch = threadIdx.x / L, l = threadIdx.x % L, c = c_0 + ch, n0 = l * SN;
   const bool fresh = a.ctx[b] - q == 0, live = c < I, vec = N % 4 == 0;
   const int cc = live ? c : 0;
   float S[SN], A[SN];
   float* gS = a.state + ((long long)a.slots[b] * I + cc) * N;
-  const long long IN = (long long)I * N;
-  float* ws = a.ws + b * ws_stride(I, N, NS);
   float* wS = ws + (long long)cc * N;       // + i * IN: start state (i = 0), end state of slice i - 1
   float* wd = ws + NS * IN + cc;            // + i * I: sum of the step sizes of slice i
-  if (NS == 1 || FOLD) {
-    if (fresh) {
+  if (fresh && (NS == 1 || FOLD)) {
 #pragma unroll
-      for (int i = 0; i < SN; ++i) S[i] = 0.f;
-    } else {
-      load_states<SN>(gS, n0, N, vec, S);
-    }
+    for (int i = 0; i < SN; ++i) S[i] = 0.f;
   } else {
-    load_states<SN>(wS, n0, N, vec, S);
+    load_states<SN>(NS == 1 || FOLD ? gS : wS, n0, N, vec, S);
   }
   load_states<SN>(a.A_log + (long long)cc * N, n0, N, vec, A);
 #pragma unroll
   for (int i = 0; i < SN; ++i) A[i] = n0 + i < N ? rate_of<AT>(A[i]) : 0.f;
   if (FOLD) {
     if (sl == 0 && live) store_states<SN>(wS, n0, N, vec, S);
-    if (j_1 == q) return;                   // nothing follows this slice
+    if (j_1 == q) return;
 #pragma unroll
     for (int i = 0; i < SN; ++i) S[i] = 0.f;
   } else {
@@ -120,68 +249,47 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(SelScanArg
       load_states<SN>(wS + (k + 1) * IN, n0, N, vec, E);
       const float d = wd[(long long)k * I];
 #pragma unroll
-      for (int i = 0; i < SN; ++i) S[i] = decay_of<AT>(A[i], d) * S[i] + E[i];
+      for (int i = 0; i < SN; ++i) S[i] = advance<AT>(S[i], A[i], d, 1.f, E[i]);
     }
   }
   float sum_dt = 0.f;
-  const AT* X = reinterpret_cast<const AT*>(a.x);
-  const AT* BC = reinterpret_cast<const AT*>(a.bc);
-  for (int jb = j_0; jb < j_1; jb += kTok) {
-    const int nt = min(kTok, j_1 - jb);
-    const long long t0 = s + jb;
-    __syncthreads();                        // the last tokens' operands and outputs are no longer read
-#pragma unroll 4
-    for (int e = threadIdx.x; e < nt * CPB; e += kScanThreads) {
-      const int jj = e / CPB, k = c_0 + e % CPB;
-      float d = 0.f, xv = 0.f;
-      if (k < I) {
-        d = softplus_f(a.dt[(t0 + jj) * a.ld_dt + k] + a.dt_bias[k]);
-        xv = ldf<AT>(X + (t0 + jj) * a.ld_x + k);
-      }
-      ds[e] = d; xs[e] = xv;
-    }
+  round_barrier();
+  for (int k = 0; k < tiles; ++k) {
+    const int buf = k & 1;
+    const float2* dk = ds[buf] + ch;
+    const float* Bk = Bs[buf] + n0;
+    const float* Ck = FOLD ? Bk : Cs[FOLD ? 0 : buf] + n0;
 #pragma unroll 2
-    for (int e = threadIdx.x; e < nt * NP; e += kScanThreads) {
-      const int jj = e / NP, n = e % NP;
-      const AT* row = BC + (t0 + jj) * a.ld_bc;
-      Bs[e] = n < N ? ldf<AT>(row + a.b0 + n) : 0.f;
-      if (!FOLD) Cs[e] = n < N ? ldf<AT>(row + a.c0 + n) : 0.f;
-    }
-    __syncthreads();
-#pragma unroll 4
-    for (int jj = 0; jj < nt; ++jj) {
-      const float d = ds[jj * CPB + ch], dx = d * xs[jj * CPB + ch];
-      float y = 0.f;
+    for (int j = 0; j < TOK; j += 4) {
+      float y[4];
 #pragma unroll
-      for (int i = 0; i < SN; i += 4) {
-        const float4 B4 = *reinterpret_cast<const float4*>(Bs + jj * NP + n0 + i);
-        S[i] = decay_of<AT>(A[i], d) * S[i] + dx * B4.x;
-        S[i + 1] = decay_of<AT>(A[i + 1], d) * S[i + 1] + dx * B4.y;
-        S[i + 2] = decay_of<AT>(A[i + 2], d) * S[i + 2] + dx * B4.z;
-        S[i + 3] = decay_of<AT>(A[i + 3], d) * S[i + 3] + dx * B4.w;
-        if (!FOLD) {
-          const float4 C4 = *reinterpret_cast<const float4*>(Cs + jj * NP + n0 + i);
-          y += S[i] * C4.x + S[i + 1] * C4.y + S[i + 2] * C4.z + S[i + 3] * C4.w;
+      for (int t = 0; t < 4; ++t) {
+        const float2 d = dk[(j + t) * CPB];
+        y[t] = token<AT, SN, FOLD>(S, A, d, Bk + (j + t) * NP, Ck + (j + t) * NP);
+        if (FOLD) sum_dt += d.x;
+      }
+      if (FOLD) continue;
+      // sums over the L lanes of a channel, four tokens at once: after the first two levels lane l holds token l % 4
+      float* yk = ys[FOLD ? 0 : buf] + j * CPB + ch;
+      if (L == 1) {
+#pragma unroll
+        for (int t = 0; t < 4; ++t) yk[t * CPB] = y[t];
+      } else {
+        const bool odd = l & 1;
+        const float u0 = (odd ? y[1] : y[0]) + __shfl_xor_sync(0xffffffffu, odd ? y[0] : y[1], 1);
+        const float u1 = (odd ? y[3] : y[2]) + __shfl_xor_sync(0xffffffffu, odd ? y[2] : y[3], 1);
+        if (L == 2) {
+          yk[(odd ? 1 : 0) * CPB] = u0; yk[(odd ? 3 : 2) * CPB] = u1;
+        } else {
+          const bool hi = l & 2;
+          float v = (hi ? u1 : u0) + __shfl_xor_sync(0xffffffffu, hi ? u0 : u1, 2);
+#pragma unroll
+          for (int o = 4; o < L; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+          if (L == 4 || l < 4) yk[(l & 3) * CPB] = v;
         }
       }
-      if (FOLD) {
-        sum_dt += d;
-      } else {
-#pragma unroll
-        for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-        if (l == 0) ys[jj * CPB + ch] = y;
-      }
     }
-    if (FOLD) continue;
-    __syncthreads();
-#pragma unroll 4
-    for (int e = threadIdx.x; e < nt * CPB; e += kScanThreads) {
-      const int jj = e / CPB, k = c_0 + e % CPB;
-      if (k >= I) continue;
-      float y = ys[e] + a.D[k] * xs[e];
-      if (a.gate != nullptr) y *= silu_f(ldf<AT>((const AT*)a.gate + (t0 + jj) * a.ld_g + k));
-      stf<AT>((AT*)a.out + (t0 + jj) * I + k, y);
-    }
+    round_barrier();
   }
   if (!live) return;
   if (FOLD) {
@@ -189,6 +297,71 @@ __global__ void __launch_bounds__(kScanThreads) selective_scan_kernel(SelScanArg
     if (l == 0) wd[(long long)sl * I] = sum_dt;
   } else if (j_1 == q) {
     store_states<SN>(gS, n0, N, vec, S);
+  }
+}
+
+// One token per sequence (decode): no staging, every operand straight into registers, kStepSeqs sequences per thread so that their state
+// loads are in flight together and the rates are computed once.                        grid (ceil(I / channels), ceil(B / kStepSeqs))
+constexpr int kStepSeqs = 4;
+
+template <typename AT, int L, int SN>
+__global__ void __launch_bounds__(kLanes) selective_step_kernel(SelScanArgs a, int B) {
+  constexpr int CPB = kLanes / L;
+  const int I = a.I, N = a.N, l = threadIdx.x % L, c = blockIdx.x * CPB + threadIdx.x / L, n0 = l * SN;
+  const bool live = c < I, vec = N % 4 == 0;
+  const int cc = live ? c : 0;
+  float S[kStepSeqs][SN], Bv[kStepSeqs][SN], Cv[kStepSeqs][SN], A[SN], d[kStepSeqs], x[kStepSeqs], z[kStepSeqs];
+  float* gS[kStepSeqs];
+  bool on[kStepSeqs];
+  const AT* X = reinterpret_cast<const AT*>(a.x);
+  const AT* BC = reinterpret_cast<const AT*>(a.bc);
+  const AT* Z = reinterpret_cast<const AT*>(a.gate);
+#pragma unroll
+  for (int i = 0; i < kStepSeqs; ++i) {
+    const int b = blockIdx.y * kStepSeqs + i;
+    const long long t = b < B ? a.cu[b] : 0;
+    on[i] = b < B && a.cu[b + 1] > a.cu[b];
+    gS[i] = a.state + ((long long)(on[i] ? a.slots[b] : 0) * I + cc) * N;
+    if (!on[i]) continue;
+    if (a.ctx[b] == 1) {                      // the sequence's first token
+#pragma unroll
+      for (int k = 0; k < SN; ++k) S[i][k] = 0.f;
+    } else {
+      load_states<SN>(gS[i], n0, N, vec, S[i]);
+    }
+    d[i] = a.dt[t * a.ld_dt + cc];
+    x[i] = ldf<AT>(X + t * a.ld_x + cc);
+    z[i] = Z != nullptr ? ldf<AT>(Z + t * a.ld_g + cc) : 0.f;
+    const AT* row = BC + t * a.ld_bc;
+#pragma unroll
+    for (int k = 0; k < SN; ++k) {
+      Bv[i][k] = n0 + k < N ? ldf<AT>(row + a.b0 + n0 + k) : 0.f;
+      Cv[i][k] = n0 + k < N ? ldf<AT>(row + a.c0 + n0 + k) : 0.f;
+    }
+  }
+  load_states<SN>(a.A_log + (long long)cc * N, n0, N, vec, A);
+  const float bias = a.dt_bias[cc], Dk = a.D[cc];
+#pragma unroll
+  for (int k = 0; k < SN; ++k) A[k] = n0 + k < N ? rate_of<AT>(A[k]) : 0.f;
+#pragma unroll
+  for (int i = 0; i < kStepSeqs; ++i) {
+    if (!on[i]) continue;                     // uniform over the CTA
+    const float dt = softplus_f(d[i] + bias);
+    float y = 0.f;
+#pragma unroll
+    for (int k = 0; k < SN; ++k) {
+      S[i][k] = advance<AT>(S[i][k], A[k], dt, dt * x[i], Bv[i][k]);
+      y = fmaf(S[i][k], Cv[i][k], y);
+    }
+#pragma unroll
+    for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (!live) continue;
+    store_states<SN>(gS[i], n0, N, vec, S[i]);
+    if (l == 0) {
+      y += Dk * x[i];
+      if (Z != nullptr) y *= silu_f(z[i]);
+      stf<AT>((AT*)a.out + (long long)a.cu[blockIdx.y * kStepSeqs + i] * I + c, y);
+    }
   }
 }
 
@@ -200,16 +373,31 @@ ScanShape scan_shape(int N) {
   return r;
 }
 
+template <typename AT, int L, int SN>
+cudaError_t scan_t(const SelScanArgs& a, int B, int max_q, cudaStream_t s) {
+  constexpr int CPB = kLanes / L, TOK = L == 1 ? 8 : L * SN <= 64 ? 16 : L * SN <= 128 ? 8 : 4;
+  const int nc = (a.I + CPB - 1) / CPB;
+  if (max_q <= 1) {
+    selective_step_kernel<AT, L, SN><<<dim3(nc, (B + kStepSeqs - 1) / kStepSeqs), kLanes, 0, s>>>(a, B);
+    return last();
+  }
+  const dim3 grid(nc, B, a.NS);
+  if (a.NS > 1) selective_scan_kernel<AT, L, SN, TOK, true><<<grid, 2 * kLanes, 0, s>>>(a);
+  selective_scan_kernel<AT, L, SN, TOK, false><<<grid, 2 * kLanes, 0, s>>>(a);
+  return last();
+}
+
 }  // namespace
 
 bool selective_scan_supported(int N) { return N >= 1 && N <= 256; }
 
+// Two passes over NS slices take about 2 / NS of the time of one pass while there are idle SMs: worth it from four slices on.
 int selective_scan_slices(int B, int I, int N, int max_q) {
-  const int cpb = kScanThreads / scan_shape(N).L;
+  const int cpb = kLanes / scan_shape(N).L;
   const long long ctas = (long long)B * ((I + cpb - 1) / cpb);
   int ns = 1;
-  while (ns < 32 && ctas * ns < 592 && max_q >= 128 * ns) ns *= 2;       // slices of at least 64 tokens
-  return ns;
+  while (ns < 32 && ctas * ns * 2 <= 296 && max_q >= 128 * ns) ns *= 2;       // slices of at least 64 tokens
+  return ns >= 4 ? ns : 1;
 }
 
 long long selective_scan_workspace(int B, int I, int N, int slices) {
@@ -221,19 +409,10 @@ cudaError_t selective_scan_launch(const void* x, long long ld_x, const float* dt
                                   const int* ctx, const int* slots, void* out, int B, int I, int N, bool f32, int max_q, int slices, float* ws,
                                   cudaStream_t s) {
   if (!selective_scan_supported(N) || slices < 1 || (slices > 1 && ws == nullptr)) return cudaErrorInvalidValue;
-  SelScanArgs a{x, ld_x, dt, ld_dt, dt_bias, A_log, bc, ld_bc, b0, c0, D, gate, ld_g, state, cu, ctx, slots, out, I, N, slices, ws};
+  const SelScanArgs a{x, ld_x, dt, ld_dt, dt_bias, A_log, bc, ld_bc, b0, c0, D, gate, ld_g, state, cu, ctx, slots, out, I, N, slices, ws};
   const ScanShape sh = scan_shape(N);
-  const int cpb = kScanThreads / sh.L, tok = max_q < 1 ? 1 : (max_q < kScanTokens ? max_q : kScanTokens);
-  const size_t smem = (size_t)tok * (2 * sh.L * sh.SN + 3 * cpb) * sizeof(float);
-  const dim3 grid((I + cpb - 1) / cpb, B, slices);
-  auto go = [&](auto fold, auto run) -> cudaError_t {
-    if (slices > 1) fold<<<grid, kScanThreads, smem, s>>>(a, tok);
-    run<<<grid, kScanThreads, smem, s>>>(a, tok);
-    return last();
-  };
-#define SCAN_CASE(LL, NN) \
-  if (sh.L == LL && sh.SN == NN) { AT_DISPATCH(f32, return go(selective_scan_kernel<AT, LL, NN, true>, selective_scan_kernel<AT, LL, NN, false>)); }
-  SCAN_CASE(1, 4) SCAN_CASE(2, 4) SCAN_CASE(4, 4) SCAN_CASE(8, 4) SCAN_CASE(16, 4) SCAN_CASE(32, 4) SCAN_CASE(32, 8)
+#define SCAN_CASE(LL, NN) if (sh.L == LL && sh.SN == NN) AT_DISPATCH(f32, return (scan_t<AT, LL, NN>(a, B, max_q, s)))
+  SCAN_CASE(1, 4); SCAN_CASE(2, 4); SCAN_CASE(4, 4); SCAN_CASE(8, 4); SCAN_CASE(16, 4); SCAN_CASE(32, 4); SCAN_CASE(32, 8);
 #undef SCAN_CASE
   return cudaErrorInvalidValue;
 }
