@@ -6,6 +6,8 @@
 // (exact mode); step sizes, decays and the state are fp32 in both.
 #include "selscan.h"
 #include "hybrid_common.cuh"
+#include <string.h>
+#include <type_traits>
 
 namespace b200 {
 namespace {
@@ -27,7 +29,8 @@ struct SelScanArgs {
 // floats of workspace per sequence (a multiple of 4: the states are read 16 bytes at a time)
 __host__ __device__ inline long long ws_stride(int I, int N, int NS) { return ((long long)NS * I * N + (long long)(NS - 1) * I + 3) / 4 * 4; }
 
-constexpr int kLanes = 128;                 // compute threads of a CTA (and as many helpers)
+constexpr int kCompute = 256, kHelpers = 256;       // threads of a CTA of the scan
+constexpr int kStepThreads = 128;
 
 // One step S <- exp(rate dt) S + add.  bf16 serving folds log2(e) into the rate and uses the hardware's base-2 exponential.  Exact mode adds
 // S (exp(rate dt) - 1) for slow decays: a factor close to 1 would carry its last-bit error, which has a sign of its own, through every token
@@ -47,6 +50,26 @@ __device__ __forceinline__ float exp2_hw(float v) {
 }
 template <> __device__ __forceinline__ float advance<__nv_bfloat16>(float S, float rate, float dt, float x, float B) {
   return fmaf(exp2_hw(rate * dt), S, x * B);
+}
+
+// Step size and gate without the branches of the library's log1p and division (a helper's instructions are a dependent chain).
+// softplus(v) = max(v, 0) + log1p(e), e = exp(-|v|) <= 1; log1p(e) = 2 atanh(s) with s = e / (2 + e) <= 1/3, its power series in s up to
+// s^13 (the next term is below 2^-26 of the sum).
+template <typename AT> __device__ __forceinline__ float step_of(float v);
+template <> __device__ __forceinline__ float step_of<float>(float v) { return softplus_f(v); }
+template <> __device__ __forceinline__ float step_of<__nv_bfloat16>(float v) {
+  const float e = exp2_hw(-1.4426950408889634f * fabsf(v)), s = __fdividef(e, 2.f + e), z = s * s;
+  float p = fmaf(z, 1.f / 13.f, 1.f / 11.f);
+  p = fmaf(z, p, 1.f / 9.f);
+  p = fmaf(z, p, 1.f / 7.f);
+  p = fmaf(z, p, 1.f / 5.f);
+  p = fmaf(z, p, 1.f / 3.f);
+  return fmaxf(v, 0.f) + 2.f * fmaf(s * z, p, s);
+}
+template <typename AT> __device__ __forceinline__ float gated(float y, float z);
+template <> __device__ __forceinline__ float gated<float>(float y, float z) { return y * silu_f(z); }
+template <> __device__ __forceinline__ float gated<__nv_bfloat16>(float y, float z) {
+  return y * __fdividef(z, 1.f + exp2_hw(fminf(-1.4426950408889634f * z, 126.f)));
 }
 
 // two floats in one 64-bit register: packed multiply and multiply-add
@@ -69,17 +92,12 @@ __device__ __forceinline__ float token(float* S, const float* A, float2 ddx, con
     const float2 d2 = make_float2(ddx.x, ddx.x), x2 = make_float2(ddx.y, ddx.y);
     float2 y = make_float2(0.f, 0.f);
 #pragma unroll
-    for (int i = 0; i < SN; i += 4) {
-      const float4 b = *reinterpret_cast<const float4*>(B + i);
-      const float4 c = FOLD ? b : *reinterpret_cast<const float4*>(C + i);
-#pragma unroll
-      for (int k = 0; k < 4; k += 2) {
-        const float2 r = mul2(make_float2(A[i + k], A[i + k + 1]), d2);
-        const float2 xb = mul2(x2, k == 0 ? make_float2(b.x, b.y) : make_float2(b.z, b.w));
-        const float2 s = fma2(make_float2(exp2_hw(r.x), exp2_hw(r.y)), make_float2(S[i + k], S[i + k + 1]), xb);
-        S[i + k] = s.x; S[i + k + 1] = s.y;
-        if (!FOLD) y = fma2(s, k == 0 ? make_float2(c.x, c.y) : make_float2(c.z, c.w), y);
-      }
+    for (int i = 0; i < SN; i += 2) {
+      const float2 r = mul2(make_float2(A[i], A[i + 1]), d2);
+      const float2 xb = mul2(x2, *reinterpret_cast<const float2*>(B + i));
+      const float2 s = fma2(make_float2(exp2_hw(r.x), exp2_hw(r.y)), make_float2(S[i], S[i + 1]), xb);
+      S[i] = s.x; S[i + 1] = s.y;
+      if (!FOLD) y = fma2(s, *reinterpret_cast<const float2*>(C + i), y);
     }
     return y.x + y.y;
   } else {
@@ -93,12 +111,16 @@ __device__ __forceinline__ float token(float* S, const float* A, float2 ddx, con
   }
 }
 
+// SN adjacent state entries from n0 on (zeros behind N); vec: rows of a multiple of SN floats (of 4 beyond that)
 template <int SN> __device__ __forceinline__ void load_states(const float* p, int n0, int N, bool vec, float* S) {
+  using V = std::conditional_t<SN == 2, float2, float4>;
+  constexpr int E = sizeof(V) / 4;
   if (vec) {
 #pragma unroll
-    for (int i = 0; i < SN; i += 4) {
-      const float4 v = n0 + i < N ? *reinterpret_cast<const float4*>(p + n0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-      S[i] = v.x; S[i + 1] = v.y; S[i + 2] = v.z; S[i + 3] = v.w;
+    for (int i = 0; i < SN; i += E) {
+      V v{};
+      if (n0 + i < N) v = *reinterpret_cast<const V*>(p + n0 + i);
+      memcpy(S + i, &v, sizeof(V));
     }
   } else {
 #pragma unroll
@@ -106,10 +128,12 @@ template <int SN> __device__ __forceinline__ void load_states(const float* p, in
   }
 }
 template <int SN> __device__ __forceinline__ void store_states(float* p, int n0, int N, bool vec, const float* S) {
+  using V = std::conditional_t<SN == 2, float2, float4>;
+  constexpr int E = sizeof(V) / 4;
   if (vec) {
 #pragma unroll
-    for (int i = 0; i < SN; i += 4)
-      if (n0 + i < N) *reinterpret_cast<float4*>(p + n0 + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+    for (int i = 0; i < SN; i += E)
+      if (n0 + i < N) { V v; memcpy(&v, S + i, sizeof(V)); *reinterpret_cast<V*>(p + n0 + i) = v; }
   } else {
 #pragma unroll
     for (int i = 0; i < SN; ++i) if (n0 + i < N) p[n0 + i] = S[i];
@@ -117,10 +141,10 @@ template <int SN> __device__ __forceinline__ void store_states(float* p, int n0,
 }
 
 // the barrier both sides of a CTA arrive at (named: the two sides sit in different branches)
-__device__ __forceinline__ void round_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(2 * kLanes) : "memory"); }
+__device__ __forceinline__ void round_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(kCompute + kHelpers) : "memory"); }
 
-// L lanes share a channel, lane l holding the state entries SN l .. SN l + SN - 1 in registers; a CTA runs 128 / L channels of one
-// sequence (and of one time slice) with 128 compute threads, which touch shared memory only, and 128 helpers, which stage the operands of
+// L lanes share a channel, lane l holding the state entries SN l .. SN l + SN - 1 in registers; a CTA runs 256 / L channels of one
+// sequence (and of one time slice) with 256 compute threads, which touch shared memory only, and 256 helpers, which stage the operands of
 // TOK tokens ahead (step sizes through the softplus once per channel) and finish the outputs of TOK tokens behind (D x, gate, store); both
 // sides work on two buffers with one barrier per TOK tokens, and the helpers' global loads are issued one round before they are used.
 // Tokens behind the end are staged as zero step sizes, which leave the state as it is.
@@ -130,8 +154,8 @@ __device__ __forceinline__ void round_barrier() { asm volatile("bar.sync 1, %0;"
 // copies the state at the step's start there.  Main form: the start of a slice is folded from the slices before it, then its tokens run
 // with outputs; the slice with the sequence's last token writes the state back.                  grid (ceil(I / channels), B, NS)
 template <typename AT, int L, int SN, int TOK, bool FOLD>
-__global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs a) {
-  constexpr int CPB = kLanes / L, NP = L * SN, EPT = (TOK * CPB + kLanes - 1) / kLanes, BPT = (TOK * NP + kLanes - 1) / kLanes;
+__global__ void __launch_bounds__(kCompute + kHelpers, 2) selective_scan_kernel(SelScanArgs a) {
+  constexpr int CPB = kCompute / L, NP = L * SN, EPT = (TOK * CPB + kHelpers - 1) / kHelpers, BPT = (TOK * NP + kHelpers - 1) / kHelpers;
   __shared__ __align__(16) float Bs[2][TOK * NP];
   __shared__ __align__(16) float Cs[FOLD ? 1 : 2][FOLD ? 4 : TOK * NP];
   __shared__ __align__(16) float2 ds[2][TOK * CPB];         // (dt, dt x)
@@ -144,66 +168,71 @@ __global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs 
   const int tiles = (j_1 - j_0 + TOK - 1) / TOK;
   const long long IN = (long long)I * N;
   float* ws = a.ws + b * ws_stride(I, N, NS);
-  if (threadIdx.x >= kLanes) {
+  if (threadIdx.x >= kCompute) {
     // ---- helpers
     if (FOLD && j_1 == q) return;             // nothing follows this slice (the compute threads leave as well, before any barrier)
-    const int tid = threadIdx.x - kLanes;
+    const int tid = threadIdx.x - kCompute;
     const AT* X = reinterpret_cast<const AT*>(a.x);
     const AT* BC = reinterpret_cast<const AT*>(a.bc);
     const AT* Z = reinterpret_cast<const AT*>(a.gate);
-    float rd[EPT], rx[EPT], rb[BPT], rc[BPT], ex[EPT], ez[EPT], bias[EPT], Dk[EPT];
+    // operands in flight, as they are stored: addresses behind the end are clamped and the values dropped when they are used, so that no
+    // load waits for another's conversion
+    float rd[EPT], bias[EPT], Dk[EPT];
+    AT rx[EPT], rb[BPT], rc[BPT], ex[EPT], ez[EPT];
 #pragma unroll
     for (int i = 0; i < EPT; ++i) {
-      const int k = c_0 + (tid + i * kLanes) % CPB;
+      const int k = c_0 + (tid + i * kHelpers) % CPB;
       bias[i] = k < I ? a.dt_bias[k] : 0.f;
       Dk[i] = !FOLD && k < I ? a.D[k] : 0.f;
     }
-    auto fetch = [&](int tile) {              // operands of a tile -> registers
+    auto fetch = [&](int tile) {    // operands of a tile -> registers
 #pragma unroll
       for (int i = 0; i < EPT; ++i) {
-        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
-        const bool ok = e < TOK * CPB && j < j_1 && k < I;
-        rd[i] = ok ? a.dt[(long long)(s + j) * a.ld_dt + k] : -INFINITY;
-        rx[i] = ok ? ldf<AT>(X + (long long)(s + j) * a.ld_x + k) : 0.f;
+        const int e = tid + i * kHelpers, j = min(j_0 + tile * TOK + e / CPB, j_1 - 1), k = min(c_0 + e % CPB, I - 1);
+        rd[i] = a.dt[(long long)(s + j) * a.ld_dt + k];
+        rx[i] = X[(long long)(s + j) * a.ld_x + k];
       }
 #pragma unroll
       for (int i = 0; i < BPT; ++i) {
-        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / NP, n = e % NP;
-        const bool ok = e < TOK * NP && j < j_1 && n < N;
+        const int e = tid + i * kHelpers, j = min(j_0 + tile * TOK + e / NP, j_1 - 1), n = min(e % NP, N - 1);
         const AT* row = BC + (long long)(s + j) * a.ld_bc + n;
-        rb[i] = ok ? ldf<AT>(row + a.b0) : 0.f;
-        if (!FOLD) rc[i] = ok ? ldf<AT>(row + a.c0) : 0.f;
+        rb[i] = row[a.b0];
+        if (!FOLD) rc[i] = row[a.c0];
       }
     };
-    auto stage = [&](int buf) {
+    auto stage = [&](int tile) {
 #pragma unroll
       for (int i = 0; i < EPT; ++i) {
-        const int e = tid + i * kLanes;
-        const float d = softplus_f(rd[i] + bias[i]);            // -inf: 0
-        if (TOK * CPB % kLanes == 0 || e < TOK * CPB) ds[buf][e] = make_float2(d, d * rx[i]);
+        const int e = tid + i * kHelpers;
+        const bool ok = j_0 + tile * TOK + e / CPB < j_1 && c_0 + e % CPB < I;
+        const float d = ok ? step_of<AT>(rd[i] + bias[i]) : 0.f;
+        if (TOK * CPB % kHelpers == 0 || e < TOK * CPB) ds[tile & 1][e] = make_float2(d, d * ldf<AT>(&rx[i]));
       }
 #pragma unroll
       for (int i = 0; i < BPT; ++i) {
-        const int e = tid + i * kLanes;
-        if (TOK * NP % kLanes == 0 || e < TOK * NP) { Bs[buf][e] = rb[i]; if (!FOLD) Cs[buf][e] = rc[i]; }
+        const int e = tid + i * kHelpers;
+        const bool ok = e % NP < N;
+        if (TOK * NP % kHelpers == 0 || e < TOK * NP) {
+          Bs[tile & 1][e] = ok ? ldf<AT>(&rb[i]) : 0.f;
+          if (!FOLD) Cs[tile & 1][e] = ok ? ldf<AT>(&rc[i]) : 0.f;
+        }
       }
     };
-    auto fetch_out = [&](int tile) {          // x and gate of a tile whose outputs are finished next round
+    auto fetch_out = [&](int tile) {        // x and gate of a tile whose outputs are finished later
 #pragma unroll
       for (int i = 0; i < EPT; ++i) {
-        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
-        const bool ok = e < TOK * CPB && j < j_1 && k < I;
-        ex[i] = ok ? ldf<AT>(X + (long long)(s + j) * a.ld_x + k) : 0.f;
-        ez[i] = ok && Z != nullptr ? ldf<AT>(Z + (long long)(s + j) * a.ld_g + k) : 0.f;
+        const int e = tid + i * kHelpers, j = min(j_0 + tile * TOK + e / CPB, j_1 - 1), k = min(c_0 + e % CPB, I - 1);
+        ex[i] = X[(long long)(s + j) * a.ld_x + k];
+        if (Z != nullptr) ez[i] = Z[(long long)(s + j) * a.ld_g + k];
       }
     };
     auto finish = [&](int tile) {
 #pragma unroll
       for (int i = 0; i < EPT; ++i) {
-        const int e = tid + i * kLanes, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
+        const int e = tid + i * kHelpers, j = j_0 + tile * TOK + e / CPB, k = c_0 + e % CPB;
         if (e >= TOK * CPB || j >= j_1 || k >= I) continue;
-        float y = ys[tile & 1][e] + Dk[i] * ex[i];
-        if (Z != nullptr) y *= silu_f(ez[i]);
+        float y = ys[tile & 1][e] + Dk[i] * ldf<AT>(&ex[i]);
+        if (Z != nullptr) y = gated<AT>(y, ldf<AT>(&ez[i]));
         stf<AT>((AT*)a.out + (long long)(s + j) * I + k, y);
       }
     };
@@ -212,10 +241,12 @@ __global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs 
     fetch(1);
     round_barrier();
     for (int k = 0; k < tiles; ++k) {         // round k: tile k is computed
-      if (k + 1 < tiles) stage((k + 1) & 1);
-      if (!FOLD && k > 0) finish(k - 1);
+      if (k + 1 < tiles) stage(k + 1);
       if (k + 2 < tiles) fetch(k + 2);
-      if (!FOLD) fetch_out(k);
+      if (!FOLD) {
+        if (k > 0) finish(k - 1);
+        fetch_out(k);
+      }
       round_barrier();
     }
     if (!FOLD) finish(tiles - 1);
@@ -223,7 +254,7 @@ __global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs 
   }
   // ---- compute threads
   const int ch = threadIdx.x / L, l = threadIdx.x % L, c = c_0 + ch, n0 = l * SN;
-  const bool fresh = a.ctx[b] - q == 0, live = c < I, vec = N % 4 == 0;
+  const bool fresh = a.ctx[b] - q == 0, live = c < I, vec = N % (SN == 2 ? 2 : 4) == 0;
   const int cc = live ? c : 0;
   float S[SN], A[SN];
   float* gS = a.state + ((long long)a.slots[b] * I + cc) * N;
@@ -305,39 +336,36 @@ __global__ void __launch_bounds__(2 * kLanes) selective_scan_kernel(SelScanArgs 
 constexpr int kStepSeqs = 4;
 
 template <typename AT, int L, int SN>
-__global__ void __launch_bounds__(kLanes) selective_step_kernel(SelScanArgs a, int B) {
-  constexpr int CPB = kLanes / L;
+__global__ void __launch_bounds__(kStepThreads) selective_step_kernel(SelScanArgs a, int B) {
+  constexpr int CPB = kStepThreads / L;
   const int I = a.I, N = a.N, l = threadIdx.x % L, c = blockIdx.x * CPB + threadIdx.x / L, n0 = l * SN;
-  const bool live = c < I, vec = N % 4 == 0;
+  const bool live = c < I, vec = N % (SN == 2 ? 2 : 4) == 0;
   const int cc = live ? c : 0;
-  float S[kStepSeqs][SN], Bv[kStepSeqs][SN], Cv[kStepSeqs][SN], A[SN], d[kStepSeqs], x[kStepSeqs], z[kStepSeqs];
+  float S[kStepSeqs][SN], A[SN], d[kStepSeqs];
+  AT Bv[kStepSeqs][SN], Cv[kStepSeqs][SN], x[kStepSeqs], z[kStepSeqs];         // as they are stored: no load waits for another's conversion
   float* gS[kStepSeqs];
-  bool on[kStepSeqs];
+  bool on[kStepSeqs], fresh[kStepSeqs];
+  long long row[kStepSeqs];
   const AT* X = reinterpret_cast<const AT*>(a.x);
   const AT* BC = reinterpret_cast<const AT*>(a.bc);
   const AT* Z = reinterpret_cast<const AT*>(a.gate);
 #pragma unroll
+  for (int i = 0; i < kStepSeqs; ++i) {       // behind the end: the last sequence, never stored
+    const int b = min(blockIdx.y * kStepSeqs + i, B - 1), t0 = a.cu[b], t1 = a.cu[b + 1];
+    on[i] = blockIdx.y * kStepSeqs + i < B && t1 > t0;
+    row[i] = min(t0, a.cu[B] - 1);
+    fresh[i] = a.ctx[b] == 1;                 // the sequence's first token
+    gS[i] = a.state + ((long long)a.slots[b] * I + cc) * N;
+  }
+#pragma unroll
   for (int i = 0; i < kStepSeqs; ++i) {
-    const int b = blockIdx.y * kStepSeqs + i;
-    const long long t = b < B ? a.cu[b] : 0;
-    on[i] = b < B && a.cu[b + 1] > a.cu[b];
-    gS[i] = a.state + ((long long)(on[i] ? a.slots[b] : 0) * I + cc) * N;
-    if (!on[i]) continue;
-    if (a.ctx[b] == 1) {                      // the sequence's first token
+    load_states<SN>(gS[i], n0, N, vec, S[i]);
+    d[i] = a.dt[row[i] * a.ld_dt + cc];
+    x[i] = X[row[i] * a.ld_x + cc];
+    if (Z != nullptr) z[i] = Z[row[i] * a.ld_g + cc];
+    const AT* p = BC + row[i] * a.ld_bc;
 #pragma unroll
-      for (int k = 0; k < SN; ++k) S[i][k] = 0.f;
-    } else {
-      load_states<SN>(gS[i], n0, N, vec, S[i]);
-    }
-    d[i] = a.dt[t * a.ld_dt + cc];
-    x[i] = ldf<AT>(X + t * a.ld_x + cc);
-    z[i] = Z != nullptr ? ldf<AT>(Z + t * a.ld_g + cc) : 0.f;
-    const AT* row = BC + t * a.ld_bc;
-#pragma unroll
-    for (int k = 0; k < SN; ++k) {
-      Bv[i][k] = n0 + k < N ? ldf<AT>(row + a.b0 + n0 + k) : 0.f;
-      Cv[i][k] = n0 + k < N ? ldf<AT>(row + a.c0 + n0 + k) : 0.f;
-    }
+    for (int k = 0; k < SN; ++k) { const int n = min(n0 + k, N - 1); Bv[i][k] = p[a.b0 + n]; Cv[i][k] = p[a.c0 + n]; }
   }
   load_states<SN>(a.A_log + (long long)cc * N, n0, N, vec, A);
   const float bias = a.dt_bias[cc], Dk = a.D[cc];
@@ -346,44 +374,48 @@ __global__ void __launch_bounds__(kLanes) selective_step_kernel(SelScanArgs a, i
 #pragma unroll
   for (int i = 0; i < kStepSeqs; ++i) {
     if (!on[i]) continue;                     // uniform over the CTA
-    const float dt = softplus_f(d[i] + bias);
+    const float dt = step_of<AT>(d[i] + bias), xv = ldf<AT>(&x[i]);
     float y = 0.f;
 #pragma unroll
     for (int k = 0; k < SN; ++k) {
-      S[i][k] = advance<AT>(S[i][k], A[k], dt, dt * x[i], Bv[i][k]);
-      y = fmaf(S[i][k], Cv[i][k], y);
+      S[i][k] = advance<AT>(fresh[i] ? 0.f : S[i][k], A[k], dt, dt * xv, n0 + k < N ? ldf<AT>(&Bv[i][k]) : 0.f);
+      y = fmaf(S[i][k], n0 + k < N ? ldf<AT>(&Cv[i][k]) : 0.f, y);
     }
 #pragma unroll
     for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
     if (!live) continue;
     store_states<SN>(gS[i], n0, N, vec, S[i]);
     if (l == 0) {
-      y += Dk * x[i];
-      if (Z != nullptr) y *= silu_f(z[i]);
-      stf<AT>((AT*)a.out + (long long)a.cu[blockIdx.y * kStepSeqs + i] * I + c, y);
+      y += Dk * xv;
+      if (Z != nullptr) y = gated<AT>(y, ldf<AT>(&z[i]));
+      stf<AT>((AT*)a.out + row[i] * I + c, y);
     }
   }
 }
 
+// lanes per channel and state entries per lane: of the scan (two entries per lane while a warp covers the state: a token's instructions
+// are a dependent chain, more warps hide it) and of the step kernel (16 bytes of state per load)
 struct ScanShape { int L, SN; };
-ScanShape scan_shape(int N) {
-  ScanShape r{1, 4};
+ScanShape scan_shape(int N, int SN) {
+  ScanShape r{1, SN};
   while (r.L < 32 && r.L * r.SN < N) r.L *= 2;
-  if (r.L * r.SN < N) r.SN = 8;
+  while (r.L * r.SN < N) r.SN *= 2;
   return r;
 }
 
 template <typename AT, int L, int SN>
-cudaError_t scan_t(const SelScanArgs& a, int B, int max_q, cudaStream_t s) {
-  constexpr int CPB = kLanes / L, TOK = L == 1 ? 8 : L * SN <= 64 ? 16 : L * SN <= 128 ? 8 : 4;
-  const int nc = (a.I + CPB - 1) / CPB;
-  if (max_q <= 1) {
-    selective_step_kernel<AT, L, SN><<<dim3(nc, (B + kStepSeqs - 1) / kStepSeqs), kLanes, 0, s>>>(a, B);
-    return last();
-  }
-  const dim3 grid(nc, B, a.NS);
-  if (a.NS > 1) selective_scan_kernel<AT, L, SN, TOK, true><<<grid, 2 * kLanes, 0, s>>>(a);
-  selective_scan_kernel<AT, L, SN, TOK, false><<<grid, 2 * kLanes, 0, s>>>(a);
+cudaError_t scan_t(const SelScanArgs& a, int B, cudaStream_t s) {
+  constexpr int CPB = kCompute / L, TOK = L <= 2 ? 4 : L == 4 ? 8 : L == 8 ? 32 : L * SN <= 64 ? 16 : L * SN <= 128 ? 8 : 4;
+  const dim3 grid((a.I + CPB - 1) / CPB, B, a.NS);
+  if (a.NS > 1) selective_scan_kernel<AT, L, SN, TOK, true><<<grid, kCompute + kHelpers, 0, s>>>(a);
+  selective_scan_kernel<AT, L, SN, TOK, false><<<grid, kCompute + kHelpers, 0, s>>>(a);
+  return last();
+}
+
+template <typename AT, int L, int SN>
+cudaError_t step_t(const SelScanArgs& a, int B, cudaStream_t s) {
+  constexpr int CPB = kStepThreads / L;
+  selective_step_kernel<AT, L, SN><<<dim3((a.I + CPB - 1) / CPB, (B + kStepSeqs - 1) / kStepSeqs), kStepThreads, 0, s>>>(a, B);
   return last();
 }
 
@@ -393,7 +425,7 @@ bool selective_scan_supported(int N) { return N >= 1 && N <= 256; }
 
 // Two passes over NS slices take about 2 / NS of the time of one pass while there are idle SMs: worth it from four slices on.
 int selective_scan_slices(int B, int I, int N, int max_q) {
-  const int cpb = kLanes / scan_shape(N).L;
+  const int cpb = kCompute / scan_shape(N, 2).L;
   const long long ctas = (long long)B * ((I + cpb - 1) / cpb);
   int ns = 1;
   while (ns < 32 && ctas * ns * 2 <= 296 && max_q >= 128 * ns) ns *= 2;       // slices of at least 64 tokens
@@ -410,9 +442,16 @@ cudaError_t selective_scan_launch(const void* x, long long ld_x, const float* dt
                                   cudaStream_t s) {
   if (!selective_scan_supported(N) || slices < 1 || (slices > 1 && ws == nullptr)) return cudaErrorInvalidValue;
   const SelScanArgs a{x, ld_x, dt, ld_dt, dt_bias, A_log, bc, ld_bc, b0, c0, D, gate, ld_g, state, cu, ctx, slots, out, I, N, slices, ws};
-  const ScanShape sh = scan_shape(N);
-#define SCAN_CASE(LL, NN) if (sh.L == LL && sh.SN == NN) AT_DISPATCH(f32, return (scan_t<AT, LL, NN>(a, B, max_q, s)))
-  SCAN_CASE(1, 4); SCAN_CASE(2, 4); SCAN_CASE(4, 4); SCAN_CASE(8, 4); SCAN_CASE(16, 4); SCAN_CASE(32, 4); SCAN_CASE(32, 8);
+#define SCAN_CASE(F, LL, NN) if (sh.L == LL && sh.SN == NN) AT_DISPATCH(f32, return (F<AT, LL, NN>(a, B, s)))
+  if (max_q <= 1) {
+    const ScanShape sh = scan_shape(N, 4);
+    SCAN_CASE(step_t, 1, 4); SCAN_CASE(step_t, 2, 4); SCAN_CASE(step_t, 4, 4); SCAN_CASE(step_t, 8, 4); SCAN_CASE(step_t, 16, 4); SCAN_CASE(step_t, 32, 4);
+    SCAN_CASE(step_t, 32, 8);
+  } else {
+    const ScanShape sh = scan_shape(N, 2);
+    SCAN_CASE(scan_t, 1, 2); SCAN_CASE(scan_t, 2, 2); SCAN_CASE(scan_t, 4, 2); SCAN_CASE(scan_t, 8, 2); SCAN_CASE(scan_t, 16, 2); SCAN_CASE(scan_t, 32, 2);
+    SCAN_CASE(scan_t, 32, 4); SCAN_CASE(scan_t, 32, 8);
+  }
 #undef SCAN_CASE
   return cudaErrorInvalidValue;
 }
