@@ -542,7 +542,7 @@ def gated_rmsnorm(y, gate, w, eps: float, groups: int, mode: str, out_dtype):
 
 
 def causal_conv_silu(u, w, b, conv_state, meta: BatchMeta):
-    return C().hy_causal_conv_silu(u, w, b, conv_state, meta.cu_seqlens, meta.context_lens, _slots(meta))
+    return C().hy_causal_conv_silu(u, w, b, conv_state, meta.cu_seqlens, meta.context_lens, _slots(meta), int(meta.max_q_len))
 
 
 def ssm_scan(xbc, dt_raw, dt_bias, A_log, D, state, meta: BatchMeta, heads: int, vdim: int, nstate: int, groups: int):

@@ -13,8 +13,9 @@
 // kernel is the planned replacement; the GEMMs that dominate prefill FLOPs already run on tcgen05.
 //
 // SINK form (attention of sinkattn.cu for long portions): keys visible inside blocks of positions or a sliding window beside kept first
-// tokens (only tiles with visible keys are walked), a sink that joins the softmax denominator, a gate per head, fp32 queries, and run-time
-// head sizes up to DK / DV (multiples of 8; the missing key columns are zeros).
+// tokens (only tiles with visible keys are walked), a sink that joins the softmax denominator, a gate per head, and run-time head sizes up to
+// DK / DV (multiples of 8; the missing key columns are zeros).  The queries are fp32: each enters the product as the sum of two bf16 numbers,
+// so that the scores are those of the fp32 queries, as in the other forms.
 #include "kernels.h"
 #include "launch.h"
 #include "ptx.cuh"
@@ -124,23 +125,25 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   };
 
   // ---- Q fragments (A operand), straight from global memory
-  uint32_t qa[DK / 16][4];
+  uint32_t qa[DK / 16][4], ql[SINK ? DK / 16 : 1][4];          // ql: what the rounding of fp32 queries to bf16 leaves (SINK)
   {
     const int ra = warp * 16 + r_lo, rb = ra + 8;
     if constexpr (SINK) {
       const float* fa = x.q32 + ((size_t)(tok0 + ra) * q_heads + hq) * D;
       const float* fb = fa + (size_t)8 * q_heads * D;
-      auto pair = [&](const float* p, bool ok, int c) {          // d is a multiple of 8: a pair is inside or outside as a whole
-        if (!ok || c >= D) return 0u;
+      auto pair = [&](const float* p, bool ok, int c, uint32_t& hi, uint32_t& lo) {      // d is a multiple of 8: a pair is inside or outside as a whole
+        hi = lo = 0u;
+        if (!ok || c >= D) return;
         const float2 f = *reinterpret_cast<const float2*>(p + c);
-        return pack_bf16(f.x, f.y);
+        hi = pack_bf16(f.x, f.y);
+        lo = pack_bf16(f.x - __uint_as_float(hi << 16), f.y - __uint_as_float(hi & 0xffff0000u));
       };
 #pragma unroll
       for (int ks = 0; ks < DK / 16; ++ks) {
-        qa[ks][0] = pair(fa, ra < rows, ks * 16 + c2);
-        qa[ks][1] = pair(fb, rb < rows, ks * 16 + c2);
-        qa[ks][2] = pair(fa, ra < rows, ks * 16 + 8 + c2);
-        qa[ks][3] = pair(fb, rb < rows, ks * 16 + 8 + c2);
+        pair(fa, ra < rows, ks * 16 + c2, qa[ks][0], ql[ks][0]);
+        pair(fb, rb < rows, ks * 16 + c2, qa[ks][1], ql[ks][1]);
+        pair(fa, ra < rows, ks * 16 + 8 + c2, qa[ks][2], ql[ks][2]);
+        pair(fb, rb < rows, ks * 16 + 8 + c2, qa[ks][3], ql[ks][3]);
       }
       if (D < DK) {                            // key columns behind d: zeros in both buffers (the copies never touch them)
         const int pad = DK - D;
@@ -195,6 +198,10 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
           ldmatrix_x4(kb, kr + nt * 8 * KS + ks * 16);
           mma_bf16(s[nt], qa[ks], kb[0], kb[1]);
           mma_bf16(s[nt + 1], qa[ks], kb[2], kb[3]);
+          if constexpr (SINK) {
+            mma_bf16(s[nt], ql[ks], kb[0], kb[1]);
+            mma_bf16(s[nt + 1], ql[ks], kb[2], kb[3]);
+          }
         }
       }
     }

@@ -875,17 +875,18 @@ Tensor hy_gated_rmsnorm(const Tensor& y, const Tensor& g, const Tensor& w, doubl
 }
 
 Tensor hy_causal_conv_silu(const Tensor& u, const Tensor& w, const Tensor& bias, Tensor cstate, const Tensor& cu, const Tensor& ctx,
-                           const Tensor& slots) {
+                           const Tensor& slots, int64_t max_q) {
   check_act(u, "u"); check_rows(u, "u"); check_f32c(w, "w"); check_f32c(bias, "bias"); check_i32(cu, "cu_seqlens"); check_i32(ctx, "context_lens");
   check_i32(slots, "state_slots");
   const int64_t T = u.size(0), C = u.size(1), K = w.size(1), B = slots.numel();
   TORCH_CHECK(w.size(0) == C && bias.numel() == C && cstate.is_contiguous() && cstate.scalar_type() == u.scalar_type() && cu.numel() == B + 1);
   TORCH_CHECK(K == 1 || (cstate.dim() == 3 && cstate.size(1) == K - 1 && cstate.size(2) == C), "conv state must be [slots, taps - 1, channels]");
-  TORCH_CHECK(K <= 17, "short convolution: at most 17 taps");
+  TORCH_CHECK(K >= 1 && K <= 17, "short convolution: at most 17 taps");
   const c10::cuda::CUDAGuard guard(u.device());
   Tensor out = torch::empty({T, C}, u.options());
+  if (T == 0) return out;
   LAUNCH_OK(b200::causal_conv_silu_launch(u.data_ptr(), u.stride(0), w.data_ptr<float>(), bias.data_ptr<float>(), cstate.data_ptr(), cu.data_ptr<int>(),
-                                          ctx.data_ptr<int>(), slots.data_ptr<int>(), (int)B, (int)C, (int)K, out.data_ptr(), is_f32(u), (int)T, cur_stream()));
+                                          ctx.data_ptr<int>(), slots.data_ptr<int>(), (int)B, (int)C, (int)K, out.data_ptr(), is_f32(u), (int)max_q, (int)T, cur_stream()));
   return out;
 }
 

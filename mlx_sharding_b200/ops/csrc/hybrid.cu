@@ -95,25 +95,75 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ y, const AT* __re
 
 // ---------------------------------------------------------------------------------------------------------- short convolution
 // out[t, c] = silu(b[c] + sum_k w[c, k] * in(t - (K-1) + k, c)); inputs before this step come from the sequence's conv state
-// ([slots, K-1, C], the last K-1 inputs), inputs before position 0 are zero.          grid (T, ceil(C / blockDim))
-template <typename AT>
+// ([slots, K-1, C], the last K-1 inputs), inputs before position 0 are zero.  A thread walks kConvRows rows of one channel with the last
+// K-1 inputs in registers (KT = K - 1 as a constant; the rows' loads are issued together).     grid (ceil(C / blockDim), ceil(T / kConvRows))
+constexpr int kConvRows = 8;
+
+template <typename AT, int KT>
 __global__ void causal_conv_silu_kernel(const AT* __restrict__ u, long long ld_u, const float* __restrict__ w, const float* __restrict__ bias,
                                         const AT* __restrict__ cstate, const int* __restrict__ cu, const int* __restrict__ ctx,
-                                        const int* __restrict__ slots, int B, int C, int K, AT* __restrict__ out) {
-  const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
+                                        const int* __restrict__ slots, int B, int C, int T, AT* __restrict__ out) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, t0 = blockIdx.y * kConvRows, t1 = min(T, t0 + kConvRows);
   if (c >= C) return;
-  const int b = seq_of(cu, B, t);
-  const int j = t - cu[b], c0 = ctx[b] - (cu[b + 1] - cu[b]);
-  const AT* st = cstate + (long long)slots[b] * (K - 1) * C;
-  float acc = bias[c];
-  for (int k = 0; k < K; ++k) {
-    const int jj = j - (K - 1) + k;          // row of this step (>= 0) or history (< 0)
-    float v = 0.f;
-    if (jj >= 0) v = ldf<AT>(u + (long long)(t - j + jj) * ld_u + c);
-    else if (c0 > 0) v = ldf<AT>(st + (long long)(K - 1 + jj) * C + c);
-    acc += w[c * K + k] * v;
+  AT raw[kConvRows];
+#pragma unroll
+  for (int i = 0; i < kConvRows; ++i) raw[i] = u[(long long)min(t0 + i, T - 1) * ld_u + c];
+  float wr[KT + 1], win[KT + 1];
+#pragma unroll
+  for (int k = 0; k <= KT; ++k) wr[k] = w[(long long)c * (KT + 1) + k];
+  const float b0 = bias[c];
+  int b = seq_of(cu, B, t0);
+  auto enter = [&](int t) {                  // the KT inputs in front of row t of sequence b
+    const int j = t - cu[b], c0 = ctx[b] - (cu[b + 1] - cu[b]);
+#pragma unroll
+    for (int k = 0; k < KT; ++k) {
+      const int jj = j - KT + k;             // row of this step (>= 0) or history (< 0)
+      win[k] = jj >= 0 ? ldf<AT>(u + (long long)(t - j + jj) * ld_u + c) : c0 > 0 ? ldf<AT>(cstate + ((long long)slots[b] * KT + KT + jj) * C + c) : 0.f;
+    }
+  };
+  int end = cu[b + 1];
+  enter(t0);
+#pragma unroll
+  for (int i = 0; i < kConvRows; ++i) {
+    const int t = t0 + i;
+    if (t >= t1) break;
+    if (t == end) {                          // the next sequence that has rows
+      do ++b; while (cu[b + 1] == t);
+      end = cu[b + 1];
+      enter(t);
+    }
+    win[KT] = ldf<AT>(&raw[i]);
+    float acc = b0;
+#pragma unroll
+    for (int k = 0; k <= KT; ++k) acc = fmaf(wr[k], win[k], acc);
+    stf<AT>(out + (long long)t * C + c, silu_f(acc));
+#pragma unroll
+    for (int k = 0; k < KT; ++k) win[k] = win[k + 1];
   }
-  stf<AT>(out + (long long)t * C + c, silu_f(rnd<AT>(acc)));
+}
+
+// One token per sequence: convolution and state shift in one pass.  A thread owns one (sequence, channel) column.
+//                                                                                       grid (ceil(C / blockDim), B)
+template <typename AT, int KT>
+__global__ void conv_step_kernel(const AT* __restrict__ u, long long ld_u, const float* __restrict__ w, const float* __restrict__ bias, AT* __restrict__ cstate,
+                                 const int* __restrict__ cu, const int* __restrict__ ctx, const int* __restrict__ slots, int C, AT* __restrict__ out) {
+  const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y, t = cu[b];
+  if (c >= C || cu[b + 1] == t) return;
+  const bool fresh = ctx[b] == 1;
+  AT* st = cstate + (long long)slots[b] * KT * C + c;
+  AT h[KT + 1];
+#pragma unroll
+  for (int k = 0; k < KT; ++k) h[k] = st[(long long)k * C];
+  h[KT] = u[t * ld_u + c];
+  float acc = bias[c];
+#pragma unroll
+  for (int k = 0; k <= KT; ++k) {
+    if (fresh && k < KT) stf<AT>(&h[k], 0.f);
+    acc = fmaf(w[(long long)c * (KT + 1) + k], ldf<AT>(&h[k]), acc);
+  }
+  stf<AT>(out + (long long)t * C + c, silu_f(acc));
+#pragma unroll
+  for (int k = 0; k < KT; ++k) st[(long long)k * C] = h[k + 1];
 }
 
 // new state = last K-1 inputs of the sequence; each thread owns one (sequence, channel) column: reads, then writes
@@ -733,15 +783,28 @@ cudaError_t gated_rmsnorm_launch(const float* y, const void* g, long long ld_g, 
   return last();
 }
 
-cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
-                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int T, cudaStream_t s) {
-  if (K - 1 > 16) return cudaErrorInvalidValue;
-  dim3 grid(T, (C + 255) / 256), gridu(B, (C + 255) / 256);
-  AT_DISPATCH(f32, (causal_conv_silu_kernel<AT><<<grid, 256, 0, s>>>((const AT*)u, ld_u, w, bias, (const AT*)cstate, cu, ctx, slots, B, C, K,
-                                                                    (AT*)out)));
-  if (K > 1)
-    AT_DISPATCH(f32, (conv_state_update_kernel<AT><<<gridu, 256, 0, s>>>((const AT*)u, ld_u, (AT*)cstate, cu, ctx, slots, C, K)));
+template <typename AT, int KT>
+static cudaError_t conv_t(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu, const int* ctx, const int* slots, int B, int C,
+                          void* out, int max_q, int T, cudaStream_t s) {
+  const int nc = (C + 127) / 128;
+  if (max_q <= 1) {
+    conv_step_kernel<AT, KT><<<dim3(nc, B), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (AT*)cstate, cu, ctx, slots, C, (AT*)out);
+    return last();
+  }
+  causal_conv_silu_kernel<AT, KT><<<dim3(nc, (T + kConvRows - 1) / kConvRows), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (const AT*)cstate, cu, ctx, slots, B, C, T, (AT*)out);
+  if (KT > 0) conv_state_update_kernel<AT><<<dim3(B, (C + 255) / 256), 256, 0, s>>>((const AT*)u, ld_u, (AT*)cstate, cu, ctx, slots, C, KT + 1);
   return last();
+}
+
+cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
+                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int max_q, int T, cudaStream_t s) {
+#define CONV_CASE(KK) case KK: AT_DISPATCH(f32, return (conv_t<AT, KK - 1>(u, ld_u, w, bias, cstate, cu, ctx, slots, B, C, out, max_q, T, s))); break;
+  switch (K) {
+    CONV_CASE(1) CONV_CASE(2) CONV_CASE(3) CONV_CASE(4) CONV_CASE(5) CONV_CASE(6) CONV_CASE(7) CONV_CASE(8) CONV_CASE(9) CONV_CASE(10) CONV_CASE(11) CONV_CASE(12)
+    CONV_CASE(13) CONV_CASE(14) CONV_CASE(15) CONV_CASE(16) CONV_CASE(17)
+  }
+#undef CONV_CASE
+  return cudaErrorInvalidValue;
 }
 
 template <typename AT, int MODE>

@@ -15,7 +15,7 @@ cudaError_t rmsnorm_cast_launch(const float* x, long long ld_x, const float* w, 
 cudaError_t gated_rmsnorm_launch(const float* y, const void* g, long long ld_g, const float* w, void* out, bool f32, int C, int groups,
                                  int mode, float eps, int T, cudaStream_t s);
 cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
-                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int T, cudaStream_t s);
+                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int max_q, int T, cudaStream_t s);
 cudaError_t ssm_scan_launch(const void* xbc, long long ld_x, const void* dt, long long ld_dt, const float* dt_bias, const float* A_log,
                             const float* D, float* state, const int* cu, const int* ctx, const int* slots, float* out, int B, int H, int N,
                             int P, int G, bool f32, int max_q, cudaStream_t s);
