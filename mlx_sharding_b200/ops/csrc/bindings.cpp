@@ -1327,6 +1327,8 @@ b200::SinkAttnArgs sink_args(const Tensor& q, const Tensor& kpool, const Tensor&
   a.q = q.data_ptr<float>(); a.kpool = kpool.data_ptr(); a.vpool = vpool.data_ptr();
   a.block_tables = block_tables.data_ptr<int>(); a.max_blocks = (int)block_tables.size(1); a.cu = cu.data_ptr<int>(); a.B = (int)(cu.numel() - 1);
   a.H = (int)H; a.G = (int)G; a.D = (int)q.size(2); a.V = (int)V; a.page = (int)kpool.size(2);
+  a.page_shift = -1;
+  for (int i = 0; i < 31; ++i) if ((1 << i) == a.page) a.page_shift = i;
   a.block = (int)block; a.window = (int)window; a.keep = (int)keep; a.scale = (float)scale; a.out_mult = (float)out_mult;
   a.out = static_cast<char*>(out.data_ptr()) + col0 * out.element_size(); a.ld_out = out.stride(0);
   a.nsplit = 1; a.chunk = 1 << 30;
@@ -1352,8 +1354,10 @@ Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpo
   // few query rows over long spans (decode): split the keys over CTAs so the grid fills the GPU; a second kernel merges the parts
   const int nw = b200::sink_attention_heads_per_cta(a.H, a.G, a.D, a.V);
   const int64_t ctas = T * G * ((H / G + nw - 1) / nw), unit = b200::sink_attention_chunk_unit();
-  if (ctas < 6 * sm_count() && span > 256) {
-    int64_t nsplit = std::min<int64_t>({(6 * sm_count() + ctas - 1) / ctas, (span + 127) / 128, (int64_t)32});
+  // (four CTAs of four warps are resident per SM: one wave of them)
+  const int64_t wave = 4 * sm_count();
+  if (2 * ctas <= wave && span > 256) {
+    int64_t nsplit = std::min<int64_t>({wave / ctas, (span + 127) / 128, (int64_t)32});
     const int64_t chunk = ((span + nsplit - 1) / nsplit + unit - 1) / unit * unit;
     nsplit = (span + chunk - 1) / chunk;
     if (nsplit > 1) { a.nsplit = (int)nsplit; a.chunk = (int)chunk; }

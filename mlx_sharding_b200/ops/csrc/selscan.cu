@@ -72,19 +72,6 @@ template <> __device__ __forceinline__ float gated<__nv_bfloat16>(float y, float
   return y * __fdividef(z, 1.f + exp2_hw(fminf(-1.4426950408889634f * z, 126.f)));
 }
 
-// two floats in one 64-bit register: packed multiply and multiply-add
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-  float2 r;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(r)) : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)));
-  return r;
-}
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-  float2 r;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(r))
-      : "l"(reinterpret_cast<unsigned long long&>(a)), "l"(reinterpret_cast<unsigned long long&>(b)), "l"(reinterpret_cast<unsigned long long&>(c)));
-  return r;
-}
-
 // one token on SN adjacent state entries: advances S, returns the lane's part of S . C (FOLD: no output)
 template <typename AT, int SN, bool FOLD>
 __device__ __forceinline__ float token(float* S, const float* A, float2 ddx, const float* B, const float* C) {

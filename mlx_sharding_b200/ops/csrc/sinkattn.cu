@@ -29,31 +29,75 @@ template <typename AT> __device__ __forceinline__ float head_factor(const SinkAt
 }
 
 // ---------------------------------------------------------------------------------------------------------- vector form
-// E activations (16 bytes of bf16, 32 of float) as raw registers
-template <typename AT> struct Chunk8;
-template <> struct Chunk8<__nv_bfloat16> {
-  uint4 a;
-  __device__ __forceinline__ void load(const __nv_bfloat16* p) { a = __ldg(reinterpret_cast<const uint4*>(p)); }
-  __device__ __forceinline__ void zero() { a = make_uint4(0u, 0u, 0u, 0u); }
-  __device__ __forceinline__ void get(float* f) const { unpack16<__nv_bfloat16>(a, f); }
-};
-template <> struct Chunk8<float> {
-  uint4 a, b;
-  __device__ __forceinline__ void load(const float* p) {
-    a = __ldg(reinterpret_cast<const uint4*>(p)); b = __ldg(reinterpret_cast<const uint4*>(p) + 1);
-  }
-  __device__ __forceinline__ void zero() { a = b = make_uint4(0u, 0u, 0u, 0u); }
-  __device__ __forceinline__ void get(float* f) const { unpack16<float>(a, f); unpack16<float>(b, f + 4); }
-};
+// 2^v: the library's for exact mode, the hardware's for bf16 serving (results that the inputs' rounding drowns)
+template <typename AT> __device__ __forceinline__ float exp2_of(float v);
+template <> __device__ __forceinline__ float exp2_of<float>(float v) { return exp2f(v); }
+template <> __device__ __forceinline__ float exp2_of<__nv_bfloat16>(float v) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+  return r;
+}
+
+// 8 adjacent activations (16 bytes of bf16, 32 of float): asynchronous copy into this thread's slot of shared memory, and out of it
+template <typename AT> constexpr int kChunkBytes = 8 * (int)sizeof(AT);
+template <typename AT> __device__ __forceinline__ void chunk_copy(unsigned dst, const AT* src) {
+#pragma unroll
+  for (int i = 0; i < kChunkBytes<AT>; i += 16)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst + i), "l"((const char*)src + i) : "memory");
+}
+__device__ __forceinline__ void chunk_get(const __nv_bfloat16* p, float2* f) {
+  const uint4 a = *reinterpret_cast<const uint4*>(p);
+  const unsigned w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) f[i] = make_float2(__uint_as_float(w[i] << 16), __uint_as_float(w[i] & 0xffff0000u));
+}
+__device__ __forceinline__ void chunk_get(const float* p, float2* f) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = make_float2(a.x, a.y); f[1] = make_float2(a.z, a.w); f[2] = make_float2(b.x, b.y); f[3] = make_float2(b.z, b.w);
+}
 
 constexpr int kRowWarps = 4;
 
+// Sums of NV values over LK lanes, every lane gets all of them: each level sends half of the values that are left one way and keeps the other
+// half (NV - 1 shuffles in all instead of NV log2 LK), then the totals are handed round.
+template <int NV, int LK> __device__ __forceinline__ void sum_over_lanes(float (&v)[NV], int lane) {
+  int left = NV;
+#pragma unroll
+  for (int w = 1; w < LK; w <<= 1) {
+    if (left > 1) {
+      left >>= 1;
+      const bool up = lane & w;
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i)
+        if (i < left) {
+          const float send = up ? v[i] : v[i + left], keep = up ? v[i + left] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], w);
+    }
+  }
+  float r[NV];
+#pragma unroll
+  for (int x = 0; x < NV; ++x) {
+    int src = 0, n = NV;
+#pragma unroll
+    for (int w = 1; w < LK; w <<= 1)
+      if (n > 1) { n >>= 1; if (x & n) src |= w; }
+    r[x] = __shfl_sync(0xffffffffu, v[x % left], src, LK);
+  }
+#pragma unroll
+  for (int x = 0; x < NV; ++x) v[x] = r[x];
+}
+
 // grid (tokens, G * ceil((H/G) / RG), key splits), 4 warps.  LK lanes share a key: each holds 8 adjacent entries of the key and of the value
-// (dim and vdim multiples of 8, at most 8 LK), so a warp reads 32 / LK keys at a time straight from the pages with 16-byte loads, U of them
-// per lane group in flight, and uses them for RG query heads.  Every lane group runs an online softmax (base 2) of its own over its keys;
+// (dim and vdim multiples of 8, at most 8 LK), so a warp takes 32 / LK keys at a time, U of them per lane group and step, straight from the
+// pages by asynchronous copies of S - 1 steps ahead — every thread reads back only what it copied itself, so no barrier is involved — and
+// uses them for RG query heads.  Every lane group runs an online softmax (base 2) of its own over its keys;
 // the groups are merged at the end, over the lanes of a warp by shuffles and over the warps in shared memory.
-template <typename AT, int LK, int RG, int U>
-__global__ void __launch_bounds__(32 * kRowWarps) sink_rows_kernel(SinkAttnArgs a) {
+template <typename AT, int LK, int RG, int U, int S>
+__global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_kernel(SinkAttnArgs a) {
+  extern __shared__ __align__(16) unsigned char ring[];      // [S][U][key, value][thread] chunks
   constexpr int KPW = 32 / LK, STEP = kRowWarps * KPW;
   __shared__ float so[kRowWarps][RG][8 * LK];
   __shared__ float sm[kRowWarps][RG], sl[kRowWarps][RG];
@@ -62,77 +106,112 @@ __global__ void __launch_bounds__(32 * kRowWarps) sink_rows_kernel(SinkAttnArgs 
   const int g = blockIdx.y / nb, r0 = (blockIdx.y % nb) * RG, pos = a.positions[t];
   const int* bt = a.block_tables + (long long)seq_of(a.cu, a.B, t) * a.max_blocks;
   const bool dk = d0 < D, dv = d0 < V;
-  float q[RG][8], o[RG][8], m[RG], l[RG];
+  float2 q[RG][4], o[RG][4];
+  float m[RG], l[RG];
 #pragma unroll
   for (int r = 0; r < RG; ++r) {
     m[r] = -INFINITY; l[r] = 0.f;
 #pragma unroll
-    for (int e = 0; e < 8; ++e) { q[r][e] = 0.f; o[r][e] = 0.f; }
+    for (int e = 0; e < 4; ++e) q[r][e] = o[r][e] = make_float2(0.f, 0.f);
     if (dk && r0 + r < Rg) {
-      const float4* qp = reinterpret_cast<const float4*>(a.q + ((long long)t * a.H + g * Rg + r0 + r) * D + d0);
-      const float4 x = qp[0], y = qp[1];
+      const float2* qp = reinterpret_cast<const float2*>(a.q + ((long long)t * a.H + g * Rg + r0 + r) * D + d0);
       const float f = a.scale * kLog2e;
-      q[r][0] = x.x * f; q[r][1] = x.y * f; q[r][2] = x.z * f; q[r][3] = x.w * f;
-      q[r][4] = y.x * f; q[r][5] = y.y * f; q[r][6] = y.z * f; q[r][7] = y.w * f;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) q[r][e] = mul2(qp[e], make_float2(f, f));
     }
   }
   const Visible vis(a, pos);
   const long long ib = (long long)blockIdx.z * a.chunk;
   const int ibeg = (int)min(ib, (long long)vis.n), iend = (int)min((long long)vis.n, ib + a.chunk);
-  const AT* kpool = (const AT*)a.kpool;
-  const AT* vpool = (const AT*)a.vpool;
-  for (int i0 = ibeg + warp * KPW + grp; i0 - grp < iend; i0 += STEP * U) {       // the bound is uniform over the warp
-    Chunk8<AT> kc[U], vc[U];
+  const AT* kpool = (const AT*)a.kpool + d0;
+  const AT* vpool = (const AT*)a.vpool + d0;
+  AT* slot = reinterpret_cast<AT*>(ring) + threadIdx.x * 8;
+  constexpr int kSlots = 32 * kRowWarps * 8;                  // elements between the chunks of one thread
+  const unsigned slot_addr = (unsigned)__cvta_generic_to_shared(slot);
+  const int first = ibeg + warp * KPW + grp, steps = max(0, (iend - (first - grp) + STEP * U - 1) / (STEP * U));      // uniform over the warp
+  int pg[U], off[U];
+  auto pages = [&](int k) {                   // pages of step k (behind the end: of the last key, masked later)
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      const int i = i0 + u * STEP, j = vis.key_at(min(i, iend - 1));
-      const long long row = ((long long)bt[j / a.page] * G + g) * a.page + j % a.page;
-      if (dk) kc[u].load(kpool + row * D + d0); else kc[u].zero();
-      if (dv) vc[u].load(vpool + row * V + d0); else vc[u].zero();
+      const int j = vis.key_at(min(first + (k * U + u) * STEP, iend - 1)), p = a.page_shift >= 0 ? j >> a.page_shift : j / a.page;
+      pg[u] = bt[p];
+      off[u] = j - p * a.page;
     }
-    float s[U][RG];
+  };
+  auto copy = [&](int stage) {
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      float f[8];
-      kc[u].get(f);
+      const long long row = (long long)(pg[u] * G + g) * a.page + off[u];
+      const unsigned dst = slot_addr + (stage * U + u) * 2 * kSlots * (int)sizeof(AT);
+      if (dk) chunk_copy<AT>(dst, kpool + row * D);
+      if (dv) chunk_copy<AT>(dst + kSlots * (int)sizeof(AT), vpool + row * V);
+    }
+  };
+  if (!dk || !dv) {                           // entries behind dim / vdim: zeros
+    for (int c = 0; c < S * U; ++c)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        if (!dk) stf<AT>(slot + 2 * c * kSlots + e, 0.f);
+        if (!dv) stf<AT>(slot + (2 * c + 1) * kSlots + e, 0.f);
+      }
+  }
+  if (steps > 0) pages(0);
+#pragma unroll
+  for (int k = 0; k < S - 1; ++k) {
+    if (k < steps) { copy(k); if (k + 1 < steps) pages(k + 1); }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  int stage = 0;
+  for (int k = 0; k < steps; ++k) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(S - 2) : "memory");
+    const AT* cur = slot + stage * U * 2 * kSlots;
+    stage = stage + 1 == S ? 0 : stage + 1;
+    const int i0 = first + k * U * STEP;
+    float s[U * RG];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      float2 f[4];
+      chunk_get(cur + 2 * u * kSlots, f);
 #pragma unroll
       for (int r = 0; r < RG; ++r) {
-        float d = 0.f;
+        float2 d = mul2(q[r][0], f[0]);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) d += q[r][e] * f[e];
-        s[u][r] = d;
+        for (int e = 1; e < 4; ++e) d = fma2(q[r][e], f[e], d);
+        s[u * RG + r] = d.x + d.y;
       }
     }
+    sum_over_lanes<U * RG, LK>(s, lane);
 #pragma unroll
     for (int u = 0; u < U; ++u)
+      if (i0 + u * STEP >= iend) {
 #pragma unroll
-      for (int r = 0; r < RG; ++r) {
-#pragma unroll
-        for (int w = LK / 2; w > 0; w >>= 1) s[u][r] += __shfl_xor_sync(0xffffffffu, s[u][r], w);
-        if (i0 + u * STEP >= iend) s[u][r] = -INFINITY;
+        for (int r = 0; r < RG; ++r) s[u * RG + r] = -INFINITY;
       }
 #pragma unroll
     for (int r = 0; r < RG; ++r) {
       float nm = m[r];
 #pragma unroll
-      for (int u = 0; u < U; ++u) nm = fmaxf(nm, s[u][r]);
-      const float base = nm == -INFINITY ? 0.f : nm, cf = exp2f(m[r] - base);       // m = -inf (nothing yet): the factor is 0
+      for (int u = 0; u < U; ++u) nm = fmaxf(nm, s[u * RG + r]);
+      const float base = nm == -INFINITY ? 0.f : nm, cf = exp2_of<AT>(m[r] - base);       // m = -inf (nothing yet): the factor is 0
       m[r] = nm;
       l[r] *= cf;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[r][e] *= cf;
+      for (int e = 0; e < 4; ++e) o[r][e] = mul2(o[r][e], make_float2(cf, cf));
 #pragma unroll
-      for (int u = 0; u < U; ++u) { s[u][r] = exp2f(s[u][r] - base); l[r] += s[u][r]; }
+      for (int u = 0; u < U; ++u) { s[u * RG + r] = exp2_of<AT>(s[u * RG + r] - base); l[r] += s[u * RG + r]; }
     }
 #pragma unroll
     for (int u = 0; u < U; ++u) {
-      float f[8];
-      vc[u].get(f);
+      float2 f[4];
+      chunk_get(cur + (2 * u + 1) * kSlots, f);
 #pragma unroll
       for (int r = 0; r < RG; ++r)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) o[r][e] += s[u][r] * f[e];
+        for (int e = 0; e < 4; ++e) o[r][e] = fma2(make_float2(s[u * RG + r], s[u * RG + r]), f[e], o[r][e]);
     }
+    // the stage read last round is free
+    if (k + S - 1 < steps) { copy(stage == 0 ? S - 2 : stage == 1 ? S - 1 : stage - 2); if (k + S < steps) pages(k + S); }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   }
   // merge the lane groups of the warp, then the warps
 #pragma unroll
@@ -143,11 +222,14 @@ __global__ void __launch_bounds__(32 * kRowWarps) sink_rows_kernel(SinkAttnArgs 
       const float nm = fmaxf(m[r], om), base = nm == -INFINITY ? 0.f : nm, c0 = exp2f(m[r] - base), c1 = exp2f(om - base);
       m[r] = nm; l[r] = l[r] * c0 + ol * c1;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) o[r][e] = o[r][e] * c0 + __shfl_xor_sync(0xffffffffu, o[r][e], w) * c1;
+      for (int e = 0; e < 4; ++e) {
+        o[r][e].x = o[r][e].x * c0 + __shfl_xor_sync(0xffffffffu, o[r][e].x, w) * c1;
+        o[r][e].y = o[r][e].y * c0 + __shfl_xor_sync(0xffffffffu, o[r][e].y, w) * c1;
+      }
     }
     if (grp == 0) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) so[warp][r][d0 + e] = o[r][e];
+      for (int e = 0; e < 4; ++e) { so[warp][r][d0 + 2 * e] = o[r][e].x; so[warp][r][d0 + 2 * e + 1] = o[r][e].y; }
     }
     if (lane == 0) { sm[warp][r] = m[r]; sl[warp][r] = l[r]; }
   }
@@ -302,11 +384,16 @@ template <typename AT, int LK>
 cudaError_t rows_form(const SinkAttnArgs& a, int T, cudaStream_t s) {
   const int Rg = a.H / a.G, hp = heads_of(Rg);
   const dim3 grid(T, a.G * ((Rg + hp - 1) / hp), a.nsplit);
-  constexpr int U = sizeof(AT) == 2 ? 4 : 2;
-  if (hp == 1) sink_rows_kernel<AT, LK, 1, U><<<grid, 32 * kRowWarps, 0, s>>>(a);
-  else if (hp == 2) sink_rows_kernel<AT, LK, 2, U><<<grid, 32 * kRowWarps, 0, s>>>(a);
-  else sink_rows_kernel<AT, LK, 4, U><<<grid, 32 * kRowWarps, 0, s>>>(a);
-  return last();
+  constexpr int U = 2, S = sizeof(AT) == 2 ? 4 : 3, smem = S * U * 2 * 32 * kRowWarps * kChunkBytes<AT>;
+  auto go = [&](auto k) -> cudaError_t {
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);      // static and dynamic together may pass 48 KB
+    if (e != cudaSuccess) return e;
+    k<<<grid, 32 * kRowWarps, smem, s>>>(a);
+    return last();
+  };
+  if (hp == 1) return go(sink_rows_kernel<AT, LK, 1, U, S>);
+  if (hp == 2) return go(sink_rows_kernel<AT, LK, 2, U, S>);
+  return go(sink_rows_kernel<AT, LK, 4, U, S>);
 }
 
 template <typename AT, int NPL>

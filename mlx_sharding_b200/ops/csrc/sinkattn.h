@@ -11,6 +11,7 @@ struct SinkAttnArgs {
   const int* block_tables; int max_blocks;
   const int* positions; const int* cu; int B;
   int H, G, D, V, page;
+  int page_shift;                           // log2(page), -1 when page is no power of two
   // visible keys j <= p: same block of `block` positions (0: all) and p - j < window (0: all), or j < keep
   int block, window, keep;
   float scale, out_mult;
