@@ -541,6 +541,55 @@ __global__ void scaled_add_norm_kernel(float* __restrict__ x, const float* __res
   for (int c = threadIdx.x; c < n; c += blockDim.x) stf<AT>(xa + t * n + c, x[t * n + c] * r * w[c]);   // own writes: same thread, same c
 }
 
+// The same with the row in registers: NV groups of four channels per thread, every load of the row in flight at once (n a multiple of 4,
+// 16-byte aligned rows, at most 4 NV blockDim channels).
+template <typename AT, int NV>
+__global__ void scaled_add_norm_vec_kernel(float* __restrict__ x, const float* __restrict__ y, long long ld_y, const float* __restrict__ ls,
+                                           const float* __restrict__ extra, long long ld_e, const float* __restrict__ gate, long long ld_gate,
+                                           const float* __restrict__ w, AT* __restrict__ xa, int n, float eps, float mult) {
+  __shared__ float red[32];
+  const long long t = blockIdx.x;
+  float4* xr = reinterpret_cast<float4*>(x + t * n);
+  const float4* yr = reinterpret_cast<const float4*>(y + t * ld_y);
+  const float4* er = extra != nullptr ? reinterpret_cast<const float4*>(extra + t * ld_e) : nullptr;
+  const float4* lr = reinterpret_cast<const float4*>(ls);
+  const float4* wr = reinterpret_cast<const float4*>(w);
+  const int n4 = n / 4;
+  float4 xv[NV], yv[NV], wv[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = min(threadIdx.x + i * blockDim.x, n4 - 1);
+    xv[i] = xr[c]; yv[i] = yr[c]; wv[i] = wr[c];
+  }
+  const float sg = extra != nullptr ? sigmoid_f(gate[t * ld_gate]) : 0.f;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c >= n4) continue;
+    float4 v = yv[i];
+    if (er != nullptr) { const float4 e = er[c]; v.x += e.x * sg; v.y += e.y * sg; v.z += e.z * sg; v.w += e.w * sg; }
+    if (ls != nullptr) { const float4 l = lr[c]; v.x *= l.x; v.y *= l.y; v.z *= l.z; v.w *= l.w; }
+    v.x = v.x * mult + xv[i].x; v.y = v.y * mult + xv[i].y; v.z = v.z * mult + xv[i].z; v.w = v.w * mult + xv[i].w;
+    xr[c] = v;
+    xv[i] = v;
+    ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+  }
+  const float r = rsqrtf(block_sum(ss, red) / (float)n + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = threadIdx.x + i * blockDim.x;
+    if (c >= n4) continue;
+    const float4 v = make_float4(xv[i].x * r * wv[i].x, xv[i].y * r * wv[i].y, xv[i].z * r * wv[i].z, xv[i].w * r * wv[i].w);
+    if constexpr (sizeof(AT) == 4) {
+      reinterpret_cast<float4*>(xa + t * n)[c] = v;
+    } else {
+      __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      reinterpret_cast<uint2*>(xa + t * n)[c] = make_uint2(reinterpret_cast<unsigned&>(lo), reinterpret_cast<unsigned&>(hi));
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------- mLSTM scan
 // Matrix memory with exponential gating, stabilised by a running maximum m (all fp32):
 //   i = cap tanh((gi + bi) / cap), f = logsigmoid(cap tanh((gf + bf) / cap)), m' = max(f + m, i), a = e^(f + m - m'), b = e^(i - m')
@@ -892,6 +941,16 @@ cudaError_t latent_attention_launch(const void* q, const void* pool, const float
 cudaError_t scaled_add_norm_launch(float* x, const float* y, long long ld_y, const float* ls, const float* extra, long long ld_e,
                                    const float* gate, long long ld_gate, const float* w, void* xa, bool f32, int n, float eps, float mult, int T,
                                    cudaStream_t s) {
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (n % 4 == 0 && n <= 16384 && ld_y % 4 == 0 && ld_e % 4 == 0 && al16(x) && al16(y) && al16(ls) && al16(extra) && al16(w) && al16(xa)) {
+    if (n <= 4096) {
+      const int th = n <= 512 ? 128 : n <= 1024 ? 256 : n <= 2048 ? 512 : 1024;
+      AT_DISPATCH(f32, (scaled_add_norm_vec_kernel<AT, 1><<<T, th, 0, s>>>(x, y, ld_y, ls, extra, ld_e, gate, ld_gate, w, (AT*)xa, n, eps, mult)));
+    } else {
+      AT_DISPATCH(f32, (scaled_add_norm_vec_kernel<AT, 4><<<T, n <= 8192 ? 512 : 1024, 0, s>>>(x, y, ld_y, ls, extra, ld_e, gate, ld_gate, w, (AT*)xa, n, eps, mult)));
+    }
+    return last();
+  }
   AT_DISPATCH(f32, (scaled_add_norm_kernel<AT><<<T, 256, 0, s>>>(x, y, ld_y, ls, extra, ld_e, gate, ld_gate, w, (AT*)xa, n, eps, mult)));
   return last();
 }
