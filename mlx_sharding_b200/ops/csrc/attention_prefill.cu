@@ -50,7 +50,7 @@ struct SinkForm {                            // what the SINK form adds (unused 
   const float* q32;                          // [T, heads, d]
   const float* sink; const __nv_bfloat16* gate; long long ld_gate;
   int d, v, block, window, keep;
-  float out_mult;
+  float scale, out_mult;                     // scale multiplies the queries (scale_log2 is log2(e) alone)
 };
 
 __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem) {
@@ -134,7 +134,8 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
       auto pair = [&](const float* p, bool ok, int c, uint32_t& hi, uint32_t& lo) {      // d is a multiple of 8: a pair is inside or outside as a whole
         hi = lo = 0u;
         if (!ok || c >= D) return;
-        const float2 f = *reinterpret_cast<const float2*>(p + c);
+        float2 f = *reinterpret_cast<const float2*>(p + c);
+        f.x *= x.scale; f.y *= x.scale;
         hi = pack_bf16(f.x, f.y);
         lo = pack_bf16(f.x - __uint_as_float(hi << 16), f.y - __uint_as_float(hi & 0xffff0000u));
       };
@@ -310,9 +311,9 @@ cudaError_t launch_sink(const SinkAttnArgs& a, const int* context_lens, int max_
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  const SinkForm x{a.q, a.sink, static_cast<const __nv_bfloat16*>(a.gate), a.ld_gate, a.D, a.V, a.block, a.window, a.keep, a.out_mult};
+  const SinkForm x{a.q, a.sink, static_cast<const __nv_bfloat16*>(a.gate), a.ld_gate, a.D, a.V, a.block, a.window, a.keep, a.scale, a.out_mult};
   kern<<<dim3(max_tiles, a.H), kThreads, smem, s>>>(nullptr, 0, 0, static_cast<const __nv_bfloat16*>(a.kpool), static_cast<const __nv_bfloat16*>(a.vpool),
-                                                    a.block_tables, a.max_blocks, a.cu, context_lens, a.B, a.H, a.G, a.page, a.scale * 1.4426950408889634f,
+                                                    a.block_tables, a.max_blocks, a.cu, context_lens, a.B, a.H, a.G, a.page, 1.4426950408889634f,
                                                     static_cast<__nv_bfloat16*>(a.out), a.ld_out, x);
   return cudaGetLastError();
 }
