@@ -244,7 +244,7 @@ def attention_reference(q, k, v, ctx0, n, scale, size, keep, gate):
 
 @pytest.mark.parametrize("device,dtype,tol", DEVICES)
 @pytest.mark.parametrize("H,G,D,V,rot,size,keep,portions,page", [
-    (4, 2, 8, 16, 4, 10, 3, [13, 14, 1, 2], 8), (3, 1, 10, 20, 6, 9, 0, [20, 3], 8), (8, 8, 64, 48, 16, 40, 5, [70, 1, 33, 16], 16), (2, 1, 6, 5, 0, 0, 0, [11, 5], 4),
+    (4, 2, 8, 16, 4, 10, 3, [13, 14, 1, 2], 8), (3, 1, 10, 20, 6, 9, 0, [20, 3], 8), (6, 6, 56, 40, 24, 40, 5, [70, 1, 33, 16], 16), (2, 1, 6, 5, 0, 0, 0, [11, 5], 4),
     (10, 2, 128, 128, 64, 100, 17, [150, 66, 1], 64), (6, 2, 24, 136, 8, 50, 7, [60, 20], 16), (6, 1, 72, 104, 72, 33, 70, [120, 40, 1], 16),
     (4, 4, 192, 96, 32, 64, 64, [100, 64, 3], 64), (3, 3, 200, 16, 8, 20, 2, [40, 1], 16)])
 def test_attention_alone(H, G, D, V, rot, size, keep, portions, page, device, dtype, tol):
