@@ -21,7 +21,7 @@ MODEL_REMAPPING = {
     "mistral": "llama",  # reference utils.py:15
 }
 
-SUPPORTED_ARCHS = ("llama", "gemma2", "deepseek_v2", "perelorn", "gusolorn", "gifetar", "gokapel", "podurax")
+SUPPORTED_ARCHS = ("llama", "gemma2", "deepseek_v2", "perelorn", "gusolorn", "gifetar", "gokapel", "podurax", "lomusun")
 
 
 @dataclass(frozen=True)
@@ -174,6 +174,8 @@ class ModelConfig:
             d = _gokapel_flat(d)
         elif "model_type" not in d and str(d.get("architecture", "")).lower() == "podurax":
             d = _podurax_flat(d)
+        elif "model_type" not in d and str(d.get("architecture", "")).lower() == "lomusun":
+            d = _lomusun_flat(d)
         mt = d.get("model_type", "llama")
         if mt == "phi-msft":
             raise ValueError(
@@ -513,6 +515,61 @@ def podurax_config(width=2048, vocab=32000, blocks=2, heads=16, kv_heads=4, dim=
     for _ in range(blocks):
         layers += [one("mamba1", scan), one("attention", att), one("attention", att), one("mamba1", scan)]
     d = dict(architecture="Podurax", embedding=dict(scale=1.0), layers=layers, norm=dict(eps=1e-6), residual_mult=0.5, vocab=vocab, width=width)
+    d.update(overrides)
+    return d
+
+
+def _lomusun_flat(d: Dict[str, Any]) -> Dict[str, Any]:
+    """Lomusun's nested config.json (``layers`` = list of {type, mixer, mlp}; ``norm.eps``; ``max_positions``; ``vocab``; ``width``) -> the flat
+    fields of :class:`ModelConfig`.  Mixers: ``parallel`` (left = attention: heads, kv_heads, dim, vdim, scale, optional mask.size; right =
+    gated delta rule: heads, kv_heads, dim, vdim, conv; left_scale, right_scale) and ``attention`` (heads, kv_heads, dim, vdim, scale, conv,
+    bias_max, optional mask.size, optional kv_from = layer whose cached keys and values it reads).  Feed-forward: ``moe`` (router.{experts,
+    top, scale}, expert.{ff, limit}) or none.  Every size is read from the file."""
+    layers = [dict(type=str(L["type"]), mixer=dict(L["mixer"]), mlp=(dict(L["mlp"]) if L.get("mlp") else None)) for L in d["layers"]]
+    for i, L in enumerate(layers):
+        m = L["mixer"]
+        if L["type"] not in ("parallel", "attention"):
+            raise ValueError(f"Lomusun: unknown mixer type '{L['type']}'")
+        if L["mlp"] is not None and L["mlp"].get("kind", "moe") != "moe":
+            raise ValueError(f"Lomusun: unknown feed-forward kind '{L['mlp'].get('kind')}'")
+        for a in ((m["left"], m["right"]) if L["type"] == "parallel" else (m,)):
+            if min(int(a[k]) for k in ("heads", "kv_heads", "dim", "vdim")) < 1 or int(a["heads"]) % int(a["kv_heads"]) != 0:
+                raise ValueError(f"Lomusun layer {i}: heads must be a multiple of kv_heads, all sizes positive")
+            if a.get("mask") and int(a["mask"]["size"]) < 1:
+                raise ValueError(f"Lomusun layer {i}: mask.size must be positive")
+        if int((m["right"] if L["type"] == "parallel" else m)["conv"]) < 1:
+            raise ValueError(f"Lomusun layer {i}: conv must be positive")
+        if L["mlp"] is not None and not (1 <= int(L["mlp"]["router"]["top"]) <= int(L["mlp"]["router"]["experts"])):
+            raise ValueError(f"Lomusun layer {i}: router.top must lie in 1 .. router.experts")
+        src = m.get("kv_from") if L["type"] == "attention" else None
+        if src is not None:
+            s = layers[int(src)] if 0 <= int(src) < i else None
+            if s is None or s["type"] != "attention" or s["mixer"].get("kv_from") is not None:
+                raise ValueError(f"Lomusun layer {i}: kv_from must name an earlier attention layer with keys and values of its own")
+            if any(int(s["mixer"][k]) != int(m[k]) for k in ("kv_heads", "dim", "vdim")):
+                raise ValueError(f"Lomusun layer {i}: kv_from layer has other key / value sizes")
+    out = {k: v for k, v in d.items() if k not in ("architecture", "layers", "norm", "vocab", "width", "max_positions")}
+    ff = [L["mlp"]["expert"]["ff"] for L in layers if L["mlp"]]
+    out.update(model_type="lomusun", hidden_size=int(d["width"]), vocab_size=int(d["vocab"]), num_hidden_layers=len(layers),
+               rms_norm_eps=float(d["norm"]["eps"]), layer_specs=layers, intermediate_size=int(max(ff)) if ff else 0,
+               max_position_embeddings=int(d["max_positions"]), tie_word_embeddings=True,
+               num_attention_heads=max(int((L["mixer"]["left"] if L["type"] == "parallel" else L["mixer"])["heads"]) for L in layers))
+    return out
+
+
+def lomusun_config(width=2048, vocab=32000, blocks=2, heads=16, kv_heads=4, dim=128, vdim=128, experts=16, top=2, expert_ff=1024, window=1024,
+                   max_positions=8192, **overrides) -> Dict[str, Any]:
+    """A Lomusun config.json with layer sizes that resemble a real model: ``blocks`` x (attention beside a gated delta rule, attention,
+    attention on the keys and values of the layer before, attention beside a gated delta rule), each with a mixture of experts."""
+    par = dict(left=dict(dim=dim, heads=heads, kv_heads=kv_heads, mask=dict(size=window), scale=dim ** -0.5, vdim=vdim), left_scale=0.7,
+               right=dict(conv=4, dim=dim, heads=heads, kv_heads=heads, vdim=vdim), right_scale=0.6)
+    att = dict(bias_max=window // 2, conv=3, dim=dim, heads=heads, kv_heads=kv_heads, mask=dict(size=window), scale=dim ** -0.5, vdim=vdim)
+    moe = dict(kind="moe", router=dict(experts=experts, top=top, scale=1.5), expert=dict(ff=expert_ff, limit=7.0))
+    one = lambda t, m: dict(type=t, mixer=dict(m), mlp=dict(moe))
+    layers = []
+    for b in range(blocks):
+        layers += [one("parallel", par), one("attention", att), one("attention", dict(att, kv_from=4 * b + 1)), one("parallel", par)]
+    d = dict(architecture="Lomusun", layers=layers, max_positions=max_positions, norm=dict(eps=1e-6), vocab=vocab, width=width)
     d.update(overrides)
     return d
 

@@ -125,7 +125,9 @@ class LLMEngine:
         self.num_groups = num_groups or max(1, getattr(pipeline, "num_stages", 1))
         self.max_seqs = max_seqs_per_group
         self.max_prefill_tokens = max_prefill_tokens
-        self.max_model_len = max_model_len
+        # a model with a table of learned positions has no more than those
+        limit = getattr(pipeline, "max_positions", 0)
+        self.max_model_len = min(max_model_len, limit) if limit else max_model_len
         # mixed_batches: a prefill step also carries the next decode token of every running sequence of the group (one ragged
         # batch), so streams in flight keep their inter-token latency while new prompts are being prefilled
         self.mixed_batches = mixed_batches

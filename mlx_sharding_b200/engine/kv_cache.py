@@ -185,12 +185,14 @@ class HybridCache(PagedKVCache):
     slots* for recurrent layers (``state[li]`` = dict name -> ``[num_slots, ...]`` tensor).  ``layout`` lists the local layers:
     ``("paged", row_width, dtype)``, ``("paged_kv", kv_heads, d_k, d_v, dtype[, {name: (shape, dtype)}])`` (separate key and value pools ``[pages, kv_heads, page,
     d]``, the geometry of :class:`PagedKVCache`, with sizes of the layer's own; the optional dict adds state tensors for a recurrence
-    that runs beside the attention in the same layer), ``("state", {name: (shape, dtype)})`` or ``("alias", j)`` (the layer keeps nothing of its own and
-    reads local layer ``j``'s pool, which comes earlier in the list: cross-layer sharing of cached rows).  Pages and slots are managed on the host by
+    that runs beside the attention in the same layer), ``("state", {name: (shape, dtype)})`` or ``("alias", j[, {state}])`` (the layer keeps no rows of its own
+    and reads local layer ``j``'s pools, which come earlier in the list: cross-layer sharing of cached rows; the optional dict as above).  Pages and slots are managed on the host by
     :class:`SequenceTable`; the step metadata carries block tables and slot ids."""
 
     def __init__(self, layout, num_pages: int, page_size: int, num_slots: int, device="cpu"):
-        if not any(ent[0] == "state" or (ent[0] == "paged_kv" and len(ent) > 5 and ent[5]) for ent in layout):
+        extra_of = lambda ent: {"paged_kv": ent[5:6], "alias": ent[2:3]}.get(ent[0], ())          # state tensors beside (aliased) pools
+        slots_of = lambda ent: {n: torch.zeros(num_slots, *shape, dtype=dt, device=device) for n, (shape, dt) in ent[0].items()} if ent and ent[0] else None
+        if not any(ent[0] == "state" or any(extra_of(ent)) for ent in layout):
             num_slots = 0                  # no recurrent layer: sequences hold pages only, the engine hands out no slots
         self.num_layers, self.num_pages, self.page_size, self.num_slots = len(layout), num_pages, page_size, num_slots
         self.kv_heads, self.d_k, self.d_v = 1, 0, 0
@@ -201,7 +203,7 @@ class HybridCache(PagedKVCache):
                     raise ValueError("cache layout: an alias must name an earlier paged layer")
                 self.k.append(self.k[ent[1]])
                 self.v.append(self.v[ent[1]])
-                self.state.append(None)
+                self.state.append(slots_of(extra_of(ent)))
             elif ent[0] == "paged":
                 self.k.append(torch.zeros(num_pages, 1, page_size, ent[1], dtype=ent[2], device=device))
                 self.v.append(torch.empty(0, dtype=ent[2], device=device))
@@ -211,8 +213,7 @@ class HybridCache(PagedKVCache):
                 self.k.append(torch.zeros(num_pages, heads, page_size, dk, dtype=dt, device=device))
                 self.v.append(torch.zeros(num_pages, heads, page_size, dv, dtype=dt, device=device))
                 # a layer that runs attention BESIDE a recurrence keeps both: pools and, as an optional sixth entry, state tensors
-                extra = ent[5] if len(ent) > 5 else None
-                self.state.append({n: torch.zeros(num_slots, *shape, dtype=sdt, device=device) for n, (shape, sdt) in extra.items()} if extra else None)
+                self.state.append(slots_of(extra_of(ent)))
             else:
                 self.k.append(None)
                 self.v.append(None)

@@ -37,6 +37,11 @@ class TraceSession:
         if not entries:
             return torch.empty(0, 0)
         t = self.table
+        limit = getattr(self.stage.model, "max_positions", 0)
+        for e in entries:
+            n = (t.length[self.ids[e["id"]]] if e["id"] in self.ids else 0) + len(e["tokens"])
+            if limit and n > limit:
+                raise ValueError(f"request {e['id']}: {n} tokens, the model has {limit} positions")
         sids, q_lens, ctx0, toks, rows, base = [], [], [], [], [], 0
         for e in entries:
             if e["id"] not in self.ids:

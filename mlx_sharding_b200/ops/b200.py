@@ -537,12 +537,18 @@ def rmsnorm_cast(x, w, eps: float, out_dtype):
     return C().hy_rmsnorm_cast(x, w, float(eps), _is32(out_dtype))
 
 
-def gated_rmsnorm(y, gate, w, eps: float, groups: int, mode: str, out_dtype):
-    return C().hy_gated_rmsnorm(y, gate, w, float(eps), int(groups), {"silu_pre": 0, "sigmoid_post": 1}[mode], _is32(out_dtype))
+def gated_rmsnorm(y, gate, w, eps: float, groups: int, mode: str, out_dtype, out=None, out_col0: int = 0):
+    return C().hy_gated_rmsnorm(y, gate, w, float(eps), int(groups), {"silu_pre": 0, "sigmoid_post": 1, "silu_post": 2}[mode], _is32(out_dtype), out, int(out_col0))
 
 
 def causal_conv_silu(u, w, b, conv_state, meta: BatchMeta):
     return C().hy_causal_conv_silu(u, w, b, conv_state, meta.cu_seqlens, meta.context_lens, _slots(meta), int(meta.max_q_len))
+
+
+def conv_qkv_append(u, w, conv_state, heads: int, dim: int, kpool, vpool, meta: BatchMeta):
+    """Convolution, fp32 queries and the append of keys and values in one kernel (plus the state update of portions)."""
+    return C().hy_conv_qkv_append(u, w, conv_state, int(heads), int(dim), kpool, vpool, meta.slot_mapping, meta.cu_seqlens, meta.context_lens, _slots(meta),
+                                  int(meta.max_q_len))
 
 
 def ssm_scan(xbc, dt_raw, dt_bias, A_log, D, state, meta: BatchMeta, heads: int, vdim: int, nstate: int, groups: int):
@@ -620,8 +626,8 @@ def router_logits(x, w):
     return torch.nn.functional.linear(x.float(), w)
 
 
-def sigmoid_topk(z, num_experts: int, top: int):
-    idx, w = C().hy_sigmoid_topk(z, int(num_experts), int(top))
+def sigmoid_topk(z, num_experts: int, top: int, correction=None, normalise: bool = False, scale: float = 1.0):
+    idx, w = C().hy_sigmoid_topk(z, int(num_experts), int(top), 0, correction, bool(normalise), float(scale))
     return idx, w
 
 
@@ -652,8 +658,8 @@ def clamped_gated_up(x, Wg: LinearWeight, Wu: LinearWeight, limit: float):
     return C().hy_clamped_glu(lin(x, Wg.weight), lin(x, Wu.weight), float(limit), None, None)
 
 
-def moe_clamped_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float):
-    return _moe_experts(x, idx, w, Wg, Wu, Wd, float(limit), 0)
+def moe_clamped_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, on_input: bool = True):
+    return _moe_experts(x, idx, w, Wg, Wu, Wd, float(limit), 0, on_input)
 
 
 def moe_glu_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight):
@@ -666,8 +672,8 @@ def silu_glu(g, u, out_dtype=None, row_scale=None):
     return C().hy_clamped_glu(g, u, 0.0, None, row_scale, 1)
 
 
-def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, kind: int):
-    """``kind`` 0: routed clamped-GLU experts with the router weight on the expert's input.  ``kind`` 1: SiLU-GLU experts, weight on the output.  bf16 banks whose sizes fit the grouped tcgen05 GEMM
+def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, kind: int, on_input: bool = False):
+    """``kind`` 0: routed clamped-GLU experts, ``kind`` 1: SiLU-GLU experts; the router weight scales the expert's input (``on_input``) or its output.  bf16 banks whose sizes fit the grouped tcgen05 GEMM
     (expert rows multiples of 128, inner sizes multiples of 8): counting-sort permutation that scales each gathered row by its pair's
     weight -> grouped two-weight GEMM with the clamped GLU in its epilogue -> grouped down GEMM (fp32) -> sum per token.  Exact mode
     (fp32) and other sizes apply the weight to the gate / up products (linear in the input) and run either one weight-row read per
@@ -677,7 +683,7 @@ def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight
     wg, wu, wd = Wg.weight, Wu.weight, Wd.weight
     E, F, K = wg.shape
     wflat = w.reshape(-1).contiguous()
-    in_scale, out_wts = (wflat, None) if kind == 0 else (None, wflat)
+    in_scale, out_wts = (wflat, None) if on_input else (None, wflat)
     if _tc_ok(x) and wg.dtype == torch.bfloat16 and F % 128 == 0 and K % 128 == 0:
         offs, pair_row, xp = c.moe_permute(idx, x, E, in_scale)
         if kind == 0:
@@ -789,8 +795,8 @@ def relu2_(x):
     return C().hy_relu2_(x)
 
 
-def stream_embed(table, ids, scale: float, streams: int):
-    return C().hy_stream_embed(table, ids, float(scale), int(streams))
+def stream_embed(table, ids, scale: float, streams: int, pos_table=None, positions=None):
+    return C().hy_stream_embed(table, ids, float(scale), int(streams), pos_table, positions)
 
 
 def dyt_cast(x, alpha: float, w, b, out_dtype):
@@ -802,35 +808,46 @@ def hyper_step_(xs, y, y2, gate, ls, mix, out_w, mult: float, in_w, alpha: float
     return C().hy_hyper_step_(xs, y, y2, gate, ls, mix, out_w, float(mult), in_w, float(alpha), w, b, _is32(act_dtype))
 
 
+HEAD_DELTA_MAX_DIM = 512         # key sizes of the kernels with one decay per head; larger ones repeat the decay over the key channels
+
+
 def delta_scan(qkv, beta, dt, dt_bias, A_log, state, meta: BatchMeta, heads: int, kv_heads: int, dim: int, vdim: int, q_scale: float,
                unit_eps: float = 1e-6):
+    if dt_bias.numel() == heads and dim > 1:        # one decay per head (``ops/csrc/headdelta.cu``)
+        if dim <= HEAD_DELTA_MAX_DIM:
+            return C().hy_head_delta_scan(qkv, beta, dt, dt_bias, A_log, state, meta.cu_seqlens, meta.context_lens, _slots(meta), int(heads), int(kv_heads),
+                                          int(dim), int(vdim), float(q_scale), float(unit_eps), int(meta.max_q_len))
+        dt, dt_bias = dt[:, :heads].float().repeat_interleave(dim, 1), dt_bias.repeat_interleave(dim)
+    dt = dt.float()
     return C().hy_delta_scan(qkv, beta, dt, dt_bias, A_log, state, meta.cu_seqlens, meta.context_lens, _slots(meta), int(heads), int(kv_heads), int(dim),
                              int(vdim), float(q_scale), float(unit_eps), int(meta.max_q_len))
 
 
 def qk_norm_rope_append(rows, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w, kn_w, eps: float, inv_freq, kpool, vpool, meta: BatchMeta,
-                        half: bool = False, norm_after: bool = False, rot_mult: float = 1.0, v_first=None, v_lambda: float = 0.0):
+                        half: bool = False, norm_after: bool = False, rot_mult: float = 1.0, v_first=None, v_lambda: float = 0.0, whole: bool = False):
     return C().hy_qk_norm_rope_append(rows, int(q_col0), int(k_col0), int(v_col0), int(heads), int(dim), qn_w, kn_w, float(eps), inv_freq, kpool, vpool,
-                                      meta.slot_mapping, meta.positions, bool(half), bool(norm_after), float(rot_mult), v_first, float(v_lambda))
+                                      meta.slot_mapping, meta.positions, bool(half), bool(norm_after), float(rot_mult), v_first, float(v_lambda), bool(whole))
 
 
 SINK_FLASH_MIN_ROWS = 16         # portions of at least so many tokens take the tensor-core kernel (64 query rows per CTA)
 
 
-def _sink_flash_ok(kpool, vpool, meta: BatchMeta, out, out_col0: int) -> bool:
+def _sink_flash_ok(kpool, vpool, meta: BatchMeta, out, out_col0: int, slopes=None, dist_bias=None) -> bool:
+    if dist_bias is not None and (slopes is not None or dist_bias.shape[1] > C().hy_sink_flash_bias_max()):
+        return False
     return (kpool.dtype == torch.bfloat16 and meta.max_q_len >= SINK_FLASH_MIN_ROWS and C().hy_sink_flash_supported(kpool.shape[3], vpool.shape[3])
             and (out is None or (out.stride(0) % 2 == 0 and out_col0 % 2 == 0)))
 
 
 def sink_attention(q, kpool, vpool, sink, meta: BatchMeta, scale: float, block: int = 0, window: int = 0, out_mult: float = 1.0, out_dtype=None,
-                   out=None, out_col0: int = 0, keep_first: int = 0, gate=None):
+                   out=None, out_col0: int = 0, keep_first: int = 0, gate=None, slopes=None, dist_bias=None):
     """bf16 steps with long portions: the tensor-core kernel on the whole ragged batch (``attention_prefill.cu``); decode steps, short
     portions, exact mode and odd head sizes: ``sinkattn.cu``."""
-    if _sink_flash_ok(kpool, vpool, meta, out, out_col0):
+    if _sink_flash_ok(kpool, vpool, meta, out, out_col0, slopes, dist_bias):
         return C().hy_sink_flash(q, kpool, vpool, sink, meta.block_tables, meta.context_lens, meta.cu_seqlens, float(scale), int(block), int(window),
-                                 float(out_mult), out, int(out_col0), int(keep_first), gate)
+                                 float(out_mult), out, int(out_col0), int(keep_first), gate, slopes, dist_bias)
     return C().hy_sink_attention(q, kpool, vpool, sink, meta.block_tables, meta.positions, meta.cu_seqlens, float(scale), int(block), int(window),
-                                 float(out_mult), int(meta.max_ctx_len), out, int(out_col0), int(keep_first), gate)
+                                 float(out_mult), int(meta.max_ctx_len), out, int(out_col0), int(keep_first), gate, slopes, dist_bias)
 
 
 SINK_PREFILL_MIN_BLOCK = 256     # blocks of fewer positions: the products are too small to pay for their launches; the ragged kernel runs

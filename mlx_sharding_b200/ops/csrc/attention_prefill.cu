@@ -13,8 +13,8 @@
 // kernel is the planned replacement; the GEMMs that dominate prefill FLOPs already run on tcgen05.
 //
 // SINK form (attention of sinkattn.cu for long portions): keys visible inside blocks of positions or a sliding window beside kept first
-// tokens (only tiles with visible keys are walked), a sink that joins the softmax denominator, a gate per head, and run-time head sizes up to
-// DK / DV (multiples of 8; the missing key columns are zeros).  The queries are fp32: each enters the product as the sum of two bf16 numbers,
+// tokens (only tiles with visible keys are walked), a bias by distance on the scores (DIST 1: slope per head, 2: table per head, in shared
+// memory), a sink that joins the softmax denominator, a gate per head or element, and run-time head sizes up to DK / DV (multiples of 8; the missing key columns are zeros).  The queries are fp32: each enters the product as the sum of two bf16 numbers,
 // so that the scores are those of the fp32 queries, as in the other forms.
 #include "kernels.h"
 #include "launch.h"
@@ -48,7 +48,8 @@ __device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const void* 
 
 struct SinkForm {                            // what the SINK form adds (unused otherwise)
   const float* q32;                          // [T, heads, d]
-  const float* sink; const __nv_bfloat16* gate; long long ld_gate;
+  const float* sink; const __nv_bfloat16* gate; long long ld_gate; bool gate_elem;
+  const float* slopes; const float* bias; int bias_len, bias_n;      // bias_n: entries of a head's row that visible keys can reach
   int d, v, block, window, keep;
   float scale, out_mult;                     // scale multiplies the queries (scale_log2 is log2(e) alone)
 };
@@ -57,7 +58,7 @@ __device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], const void* smem) 
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(smem)));
 }
 
-template <int DK, int DV, bool SINK>
+template <int DK, int DV, bool SINK, int DIST = 0>
 __global__ void __launch_bounds__(kThreads)
 flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long long q_ld_h,
                      const __nv_bfloat16* __restrict__ kpool, const __nv_bfloat16* __restrict__ vpool,
@@ -69,6 +70,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* sK = reinterpret_cast<__nv_bfloat16*>(smem_raw);      // [2][kBN][KS]
   __nv_bfloat16* sV = sK + 2 * kBN * KS;                               // [2][kBN][VS]
+  float* sB = reinterpret_cast<float*>(sV + 2 * kBN * VS);             // [bias_n] (DIST 2)
 
   // ---- which (sequence, q tile) is this CTA?
   int tile = blockIdx.x, seq = 0, q0 = 0, qlen = 0;
@@ -172,6 +174,10 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   load_tile(row_of(tile_at(0)), 0);
   size_t next_row = ntiles > 1 ? row_of(tile_at(1)) : 0;
   const int last_lo = SINK ? first_key(pos0 + rows - 1) : 0;
+  if constexpr (DIST == 2) {                 // (the first tile's barrier comes before any use)
+    for (int i = threadIdx.x; i < x.bias_n; i += kThreads) sB[i] = x.bias[(size_t)hq * x.bias_len + i];
+  }
+  const float slope = DIST == 1 ? x.slopes[hq] : 0.f;
   for (int j = 0; j < ntiles; ++j) {
     const int buf = j & 1;
     if (j + 1 < ntiles) {
@@ -208,6 +214,22 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
     }
     // ---- mask (tiles that every row of the CTA sees as a whole need none), online softmax (base 2) on the raw scores
     const int kbase = tile_at(j) * kBN;
+    if constexpr (DIST == 1) {
+      const float na = (float)(kbase + c2 - qpos_a), nb = na - 8.f;          // minus the distance of the thread's first key
+#pragma unroll
+      for (int nt = 0; nt < kBN / 8; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) { s[nt][e] = fmaf(slope, na + (float)(nt * 8 + e), s[nt][e]); s[nt][2 + e] = fmaf(slope, nb + (float)(nt * 8 + e), s[nt][2 + e]); }
+    } else if constexpr (DIST == 2) {
+      const int na = qpos_a - kbase - c2, last = x.bias_n - 1;               // keys that are not visible: any entry, masked below
+#pragma unroll
+      for (int nt = 0; nt < kBN / 8; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          s[nt][e] += sB[min(max(na - nt * 8 - e, 0), last)];
+          s[nt][2 + e] += sB[min(max(na + 8 - nt * 8 - e, 0), last)];
+        }
+    }
     float mx_a = m_a, mx_b = m_b;
     if (kbase + kBN - 1 > pos0 || (SINK && kbase < last_lo && kbase + kBN > x.keep)) {
 #pragma unroll
@@ -266,7 +288,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
   if constexpr (SINK) {
     if (x.sink != nullptr) { const float sk = x.sink[hq] * 1.4426950408889634f; l_a += exp2f(fmaf(-m_a, scale_log2, sk)); l_b += exp2f(fmaf(-m_b, scale_log2, sk)); }
     fa = fb = x.out_mult;
-    if (x.gate != nullptr) {
+    if (x.gate != nullptr && !x.gate_elem) {
       auto sig = [&](int r) { return 1.f / (1.f + expf(-__bfloat162float(x.gate[(size_t)(tok0 + r) * x.ld_gate + hq]))); };
       if (ra < rows) fa *= sig(ra);
       if (rb < rows) fb *= sig(rb);
@@ -276,6 +298,14 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, long long q_ld_t, long
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) {
     if (SINK && i * 8 >= V) break;
+    if constexpr (SINK) {
+      if (x.gate != nullptr && x.gate_elem) {
+        const __nv_bfloat16* gp = x.gate + (size_t)(tok0 + ra) * x.ld_gate + (size_t)hq * V + i * 8 + c2;
+        auto sig = [&](const __nv_bfloat16* p) { return 1.f / (1.f + expf(-__bfloat162float(*p))); };
+        if (ra < rows) { o[i][0] *= sig(gp); o[i][1] *= sig(gp + 1); }
+        if (rb < rows) { o[i][2] *= sig(gp + 8 * x.ld_gate); o[i][3] *= sig(gp + 8 * x.ld_gate + 1); }
+      }
+    }
     if (ra < rows)
       *reinterpret_cast<uint32_t*>(out + (size_t)(tok0 + ra) * o_ld_t + (size_t)hq * V + i * 8 + c2) = pack_bf16(o[i][0] * ia, o[i][1] * ia);
     if (rb < rows)
@@ -301,21 +331,35 @@ cudaError_t launch_prefill(const FlashPrefillArgs& a, cudaStream_t s) {
   return cudaGetLastError();
 }
 
-template <int DK, int DV>
+constexpr int kBiasMax = 8192;               // entries of a distance table that shared memory takes
+
+template <int DK, int DV, int DIST>
 cudaError_t launch_sink(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s) {
-  constexpr int smem = 2 * kBN * ((DK + 8) + (DV + 8)) * 2;
-  auto kern = flash_prefill_kernel<DK, DV, true>;
+  constexpr int tiles = 2 * kBN * ((DK + 8) + (DV + 8)) * 2;
+  auto kern = flash_prefill_kernel<DK, DV, true, DIST>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, tiles + (DIST == 2 ? kBiasMax * 4 : 0));
     if (e != cudaSuccess) return e;
     configured = true;
   }
-  const SinkForm x{a.q, a.sink, static_cast<const __nv_bfloat16*>(a.gate), a.ld_gate, a.D, a.V, a.block, a.window, a.keep, a.scale, a.out_mult};
-  kern<<<dim3(max_tiles, a.H), kThreads, smem, s>>>(nullptr, 0, 0, static_cast<const __nv_bfloat16*>(a.kpool), static_cast<const __nv_bfloat16*>(a.vpool),
-                                                    a.block_tables, a.max_blocks, a.cu, context_lens, a.B, a.H, a.G, a.page, 1.4426950408889634f,
-                                                    static_cast<__nv_bfloat16*>(a.out), a.ld_out, x);
+  int reach = a.bias_len;                    // distances of visible keys: below the window / block unless first tokens are kept
+  if (a.keep == 0 && a.window > 0 && a.window < reach) reach = a.window;
+  if (a.keep == 0 && a.block > 0 && a.block < reach) reach = a.block;
+  if (DIST == 2 && reach > kBiasMax) return cudaErrorInvalidValue;
+  const SinkForm x{a.q, a.sink, static_cast<const __nv_bfloat16*>(a.gate), a.ld_gate, a.gate_elem, a.slopes, a.bias, a.bias_len, reach,
+                   a.D, a.V, a.block, a.window, a.keep, a.scale, a.out_mult};
+  kern<<<dim3(max_tiles, a.H), kThreads, tiles + (DIST == 2 ? (reach + 3) / 4 * 16 : 0), s>>>(
+      nullptr, 0, 0, static_cast<const __nv_bfloat16*>(a.kpool), static_cast<const __nv_bfloat16*>(a.vpool), a.block_tables, a.max_blocks, a.cu, context_lens, a.B, a.H,
+      a.G, a.page, 1.4426950408889634f, static_cast<__nv_bfloat16*>(a.out), a.ld_out, x);
   return cudaGetLastError();
+}
+
+template <int DIST>
+cudaError_t launch_sink_sizes(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s) {
+  if (a.D <= 64 && a.V <= 64) return launch_sink<64, 64, DIST>(a, context_lens, max_tiles, s);
+  if (a.D <= 128) return launch_sink<128, 128, DIST>(a, context_lens, max_tiles, s);
+  return launch_sink<192, 128, DIST>(a, context_lens, max_tiles, s);
 }
 
 }  // namespace
@@ -334,13 +378,15 @@ cudaError_t flash_prefill_launch(const FlashPrefillArgs& a, cudaStream_t s) {
 }
 
 bool sink_flash_supported(int D, int V) { return D % 8 == 0 && V % 8 == 0 && D >= 8 && V >= 8 && D <= 192 && V <= 128; }
+int sink_flash_bias_max() { return kBiasMax; }
 
 cudaError_t sink_flash_launch(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s) {
   if (!sink_flash_supported(a.D, a.V) || a.ld_out % 2 != 0 || a.keep < 0) return cudaErrorInvalidValue;
   if (a.B == 0 || max_tiles == 0) return cudaSuccess;
-  if (a.D <= 64 && a.V <= 64) return launch_sink<64, 64>(a, context_lens, max_tiles, s);
-  if (a.D <= 128) return launch_sink<128, 128>(a, context_lens, max_tiles, s);
-  return launch_sink<192, 128>(a, context_lens, max_tiles, s);
+  if (a.slopes != nullptr && a.bias != nullptr) return cudaErrorInvalidValue;
+  if (a.slopes != nullptr) return launch_sink_sizes<1>(a, context_lens, max_tiles, s);
+  if (a.bias != nullptr) return launch_sink_sizes<2>(a, context_lens, max_tiles, s);
+  return launch_sink_sizes<0>(a, context_lens, max_tiles, s);
 }
 
 }  // namespace b200

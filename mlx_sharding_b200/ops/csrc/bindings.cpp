@@ -10,6 +10,7 @@
 
 #include "gemm_tcgen05.h"
 #include "kernels.h"
+#include "headdelta.h"
 #include "hybrid.h"
 #include "diffattn.h"
 #include "selscan.h"
@@ -864,30 +865,60 @@ Tensor hy_rmsnorm_cast(const Tensor& x, const Tensor& w, double eps, bool out_f3
   return out;
 }
 
-Tensor hy_gated_rmsnorm(const Tensor& y, const Tensor& g, const Tensor& w, double eps, int64_t groups, int64_t mode, bool out_f32) {
+// out (optional): activation type [T, >= col0 + C], the result goes to its columns col0 .. col0 + C
+Tensor hy_gated_rmsnorm(const Tensor& y, const Tensor& g, const Tensor& w, double eps, int64_t groups, int64_t mode, bool out_f32,
+                        const c10::optional<Tensor>& out_, int64_t col0) {
   check_f32c(y, "y"); check_f32c(w, "w"); check_act(g, "gate"); check_rows(g, "gate");
   TORCH_CHECK(is_f32(g) == out_f32 && g.size(0) == y.size(0) && g.size(1) == y.size(1) && w.numel() == y.size(1) && groups >= 1 && y.size(1) % groups == 0);
   const c10::cuda::CUDAGuard guard(y.device());
-  Tensor out = torch::empty({y.size(0), y.size(1)}, y.options().dtype(act_type(out_f32)));
-  LAUNCH_OK(b200::gated_rmsnorm_launch(y.data_ptr<float>(), g.data_ptr(), g.stride(0), w.data_ptr<float>(), out.data_ptr(), out_f32, (int)y.size(1),
-                                       (int)groups, (int)mode, (float)eps, (int)y.size(0), cur_stream()));
+  Tensor out = out_.has_value() ? *out_ : torch::empty({y.size(0), y.size(1)}, y.options().dtype(act_type(out_f32)));
+  check_rows(out, "out");
+  TORCH_CHECK(out.scalar_type() == g.scalar_type() && out.size(0) == y.size(0) && col0 >= 0 && col0 + y.size(1) <= out.size(1));
+  if (y.size(0) == 0) return out;
+  LAUNCH_OK(b200::gated_rmsnorm_launch(y.data_ptr<float>(), g.data_ptr(), g.stride(0), w.data_ptr<float>(),
+                                       static_cast<char*>(out.data_ptr()) + col0 * out.element_size(), out_f32, (int)y.size(1), (int)groups, (int)mode, (float)eps,
+                                       (int)y.size(0), out.stride(0), cur_stream()));
   return out;
 }
 
-Tensor hy_causal_conv_silu(const Tensor& u, const Tensor& w, const Tensor& bias, Tensor cstate, const Tensor& cu, const Tensor& ctx,
-                           const Tensor& slots, int64_t max_q) {
-  check_act(u, "u"); check_rows(u, "u"); check_f32c(w, "w"); check_f32c(bias, "bias"); check_i32(cu, "cu_seqlens"); check_i32(ctx, "context_lens");
-  check_i32(slots, "state_slots");
-  const int64_t T = u.size(0), C = u.size(1), K = w.size(1), B = slots.numel();
-  TORCH_CHECK(w.size(0) == C && bias.numel() == C && cstate.is_contiguous() && cstate.scalar_type() == u.scalar_type() && cu.numel() == B + 1);
+static void check_conv(const Tensor& u, const Tensor& w, const Tensor& cstate, const Tensor& cu, const Tensor& ctx, const Tensor& slots) {
+  check_act(u, "u"); check_rows(u, "u"); check_f32c(w, "w"); check_i32(cu, "cu_seqlens"); check_i32(ctx, "context_lens"); check_i32(slots, "state_slots");
+  const int64_t C = u.size(1), K = w.size(1), B = slots.numel();
+  TORCH_CHECK(w.size(0) == C && cstate.is_contiguous() && cstate.scalar_type() == u.scalar_type() && cu.numel() == B + 1);
   TORCH_CHECK(K == 1 || (cstate.dim() == 3 && cstate.size(1) == K - 1 && cstate.size(2) == C), "conv state must be [slots, taps - 1, channels]");
   TORCH_CHECK(K >= 1 && K <= 17, "short convolution: at most 17 taps");
+}
+
+Tensor hy_causal_conv_silu(const Tensor& u, const Tensor& w, const c10::optional<Tensor>& bias, Tensor cstate, const Tensor& cu, const Tensor& ctx,
+                           const Tensor& slots, int64_t max_q) {
+  check_conv(u, w, cstate, cu, ctx, slots);
+  const int64_t T = u.size(0), C = u.size(1), K = w.size(1), B = slots.numel();
+  if (bias.has_value()) { check_f32c(*bias, "bias"); TORCH_CHECK(bias->numel() == C); }
   const c10::cuda::CUDAGuard guard(u.device());
   Tensor out = torch::empty({T, C}, u.options());
   if (T == 0) return out;
-  LAUNCH_OK(b200::causal_conv_silu_launch(u.data_ptr(), u.stride(0), w.data_ptr<float>(), bias.data_ptr<float>(), cstate.data_ptr(), cu.data_ptr<int>(),
+  LAUNCH_OK(b200::causal_conv_silu_launch(u.data_ptr(), u.stride(0), w.data_ptr<float>(), bias.has_value() ? bias->data_ptr<float>() : nullptr, cstate.data_ptr(), cu.data_ptr<int>(),
                                           ctx.data_ptr<int>(), slots.data_ptr<int>(), (int)B, (int)C, (int)K, out.data_ptr(), is_f32(u), (int)max_q, (int)T, cur_stream()));
   return out;
+}
+
+// queries (first H * D columns of u) -> fp32 [T, H, D]; keys and values behind them (if any) -> the pools
+Tensor hy_conv_qkv_append(const Tensor& u, const Tensor& w, Tensor cstate, int64_t H, int64_t D, Tensor kpool, Tensor vpool, const Tensor& slot_map, const Tensor& cu,
+                          const Tensor& ctx, const Tensor& slots, int64_t max_q) {
+  check_conv(u, w, cstate, cu, ctx, slots); check_i32(slot_map, "slot_mapping");
+  TORCH_CHECK(kpool.dim() == 4 && vpool.dim() == 4 && kpool.is_contiguous() && vpool.is_contiguous() && kpool.scalar_type() == u.scalar_type() &&
+              vpool.scalar_type() == u.scalar_type() && kpool.size(0) == vpool.size(0) && kpool.size(1) == vpool.size(1) && kpool.size(2) == vpool.size(2) &&
+              kpool.size(3) == D, "pools [pages, kv_heads, page, d] in the activation type");
+  const int64_t T = u.size(0), C = u.size(1), K = w.size(1), B = slots.numel(), G = kpool.size(1), V = vpool.size(3);
+  TORCH_CHECK((C == H * D || C == H * D + G * (D + V)) && slot_map.numel() >= T, "columns [q | k | v] or queries alone");
+  const c10::cuda::CUDAGuard guard(u.device());
+  Tensor q = torch::empty({T, H, D}, u.options().dtype(torch::kFloat32));
+  if (T == 0) return q;
+  LAUNCH_OK(b200::conv_qkv_append_launch(u.data_ptr(), u.stride(0), w.data_ptr<float>(), cstate.data_ptr(), cu.data_ptr<int>(), ctx.data_ptr<int>(), slots.data_ptr<int>(),
+                                         (int)B, (int)C, (int)K, q.data_ptr<float>(), (int)(H * D), kpool.data_ptr(), vpool.data_ptr(), slot_map.data_ptr<int>(), (int)G,
+                                         (int)D, (int)V, (int)kpool.size(2), is_f32(u), (int)max_q, (int)T, cur_stream()));
+  if (max_q > 1 && K > 1) ++g_launches;       // state update
+  return q;
 }
 
 Tensor hy_ssm_scan(const Tensor& xbc, const Tensor& dt, const Tensor& dt_bias, const Tensor& A_log, const Tensor& D, Tensor state, const Tensor& cu,
@@ -995,7 +1026,7 @@ Tensor hy_sink_softmax(const Tensor& s, const c10::optional<Tensor>& sink, int64
   return out;
 }
 
-// x += (y + extra * sigmoid(gate)) * ls on the fp32 residual stream (in place); returns rms(x) * w in the activation type
+// x += (y + extra * sigmoid(gate)) * ls (gate optional: factor 1) on the fp32 residual stream (in place); returns rms(x) * w in the activation type
 Tensor hy_scaled_add_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor>& ls, const Tensor& w, double eps, bool act_f32,
                            const c10::optional<Tensor>& extra, const c10::optional<Tensor>& gate, double mult) {
   check_f32c(x, "x"); check_f32c(w, "w"); check_rows(y, "y");
@@ -1003,10 +1034,14 @@ Tensor hy_scaled_add_norm_(Tensor x, const Tensor& y, const c10::optional<Tensor
   const float* lsp = nullptr; const float* ep = nullptr; const float* gp = nullptr; long long lde = 0, ldg = 0;
   if (ls.has_value()) { check_f32c(*ls, "ls"); TORCH_CHECK(ls->numel() == x.size(1)); lsp = ls->data_ptr<float>(); }
   if (extra.has_value()) {
-    TORCH_CHECK(gate.has_value() && extra->is_cuda() && extra->scalar_type() == torch::kFloat32 && gate->scalar_type() == torch::kFloat32 && gate->is_cuda());
+    TORCH_CHECK(extra->is_cuda() && extra->scalar_type() == torch::kFloat32);
     check_rows(*extra, "extra");
-    TORCH_CHECK(extra->size(0) == x.size(0) && extra->size(1) == x.size(1) && gate->dim() == 1 && gate->size(0) == x.size(0));
-    ep = extra->data_ptr<float>(); lde = extra->stride(0); gp = gate->data_ptr<float>(); ldg = gate->stride(0);
+    TORCH_CHECK(extra->size(0) == x.size(0) && extra->size(1) == x.size(1));
+    ep = extra->data_ptr<float>(); lde = extra->stride(0);
+    if (gate.has_value()) {
+      TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == torch::kFloat32 && gate->dim() == 1 && gate->size(0) == x.size(0));
+      gp = gate->data_ptr<float>(); ldg = gate->stride(0);
+    }
   }
   const c10::cuda::CUDAGuard guard(x.device());
   Tensor xa = torch::empty({x.size(0), x.size(1)}, x.options().dtype(act_type(act_f32)));
@@ -1036,15 +1071,15 @@ Tensor hy_mlstm_scan(const Tensor& qkv, const Tensor& gates, const Tensor& gate_
   return out;
 }
 
-std::vector<Tensor> hy_sigmoid_topk(const Tensor& z, int64_t E, int64_t top, int64_t mode, const c10::optional<Tensor>& bias) {
+std::vector<Tensor> hy_sigmoid_topk(const Tensor& z, int64_t E, int64_t top, int64_t mode, const c10::optional<Tensor>& bias, bool normalise, double scale) {
   check_rows(z, "z");
   TORCH_CHECK(z.is_cuda() && z.scalar_type() == torch::kFloat32 && z.dim() == 2 && z.size(1) >= E && top >= 1 && top <= E && (mode == 0 || mode == 1));
-  if (bias.has_value()) { check_f32c(*bias, "bias"); TORCH_CHECK(bias->numel() >= E && mode == 1); }
+  if (bias.has_value()) { check_f32c(*bias, "bias"); TORCH_CHECK(bias->numel() >= E); }
   const c10::cuda::CUDAGuard guard(z.device());
   Tensor idx = torch::empty({z.size(0), top}, z.options().dtype(torch::kInt32)), w = torch::empty({z.size(0), top}, z.options());
   if (z.size(0) == 0) return {idx, w};
   LAUNCH_OK(b200::router_topk_launch(z.data_ptr<float>(), z.stride(0), bias.has_value() ? bias->data_ptr<float>() : nullptr, (int)mode, (int)E, (int)top,
-                                     idx.data_ptr<int>(), w.data_ptr<float>(), (int)z.size(0), cur_stream()));
+                                     idx.data_ptr<int>(), w.data_ptr<float>(), normalise, (float)scale, (int)z.size(0), cur_stream()));
   return {idx, w};
 }
 
@@ -1183,14 +1218,21 @@ Tensor hy_diff_head_norm(const Tensor& a, int64_t T, int64_t H, double lam, doub
 }
 
 // ---- several residual streams, gated delta rule, attention with a sink, minGRU, group-limited router (streams.cu) ----------------------
-Tensor hy_stream_embed(const Tensor& table, const Tensor& ids, double scale, int64_t S) {
+// pos [positions, width] in the table's type, added at positions[t] (optional)
+Tensor hy_stream_embed(const Tensor& table, const Tensor& ids, double scale, int64_t S, const c10::optional<Tensor>& pos, const c10::optional<Tensor>& positions) {
   check_act(table, "table"); check_rows(table, "table");
   TORCH_CHECK(ids.is_cuda() && ids.scalar_type() == torch::kInt64 && ids.is_contiguous() && S >= 1 && S <= 8, "streams: 1 .. 8");
   const c10::cuda::CUDAGuard guard(table.device());
   Tensor xs = torch::empty({ids.numel(), S, table.size(1)}, table.options().dtype(torch::kFloat32));
   if (ids.numel() == 0) return xs;
+  if (pos.has_value()) {
+    TORCH_CHECK(positions.has_value() && pos->is_cuda() && pos->is_contiguous() && pos->dim() == 2 && pos->size(0) >= 1 && pos->size(1) == table.size(1) &&
+                pos->scalar_type() == table.scalar_type() && positions->numel() >= ids.numel(), "position table [positions, width] in the embedding's type");
+    check_i32(*positions, "positions");
+  }
   LAUNCH_OK(b200::stream_embed_launch(table.data_ptr(), is_f32(table), table.stride(0), reinterpret_cast<const long long*>(ids.data_ptr<int64_t>()), (float)scale,
-                                      (int)S, (int)table.size(1), xs.data_ptr<float>(), (int)ids.numel(), cur_stream()));
+                                      (int)S, (int)table.size(1), xs.data_ptr<float>(), pos.has_value() ? pos->data_ptr() : nullptr,
+                                      pos.has_value() ? positions->data_ptr<int>() : nullptr, pos.has_value() ? (int)pos->size(0) : 0, (int)ids.numel(), cur_stream()));
   return xs;
 }
 
@@ -1256,6 +1298,29 @@ Tensor hy_delta_scan(const Tensor& qkv, const Tensor& beta, const Tensor& dt, co
   return out;
 }
 
+// one decay per head: beta, dt raw in the activation type [T, >= H], dt_bias [H]
+Tensor hy_head_delta_scan(const Tensor& qkv, const Tensor& beta, const Tensor& dt, const Tensor& dt_bias, const Tensor& A_log, Tensor state, const Tensor& cu,
+                          const Tensor& ctx, const Tensor& slots, int64_t H, int64_t G, int64_t Dk, int64_t V, double q_scale, double unit_eps, int64_t max_q) {
+  check_act(qkv, "qkv"); check_rows(qkv, "qkv"); check_rows(beta, "beta"); check_rows(dt, "dt"); check_f32c(dt_bias, "dt_bias");
+  check_f32c(A_log, "A_log"); check_f32c(state, "state"); check_i32(cu, "cu_seqlens"); check_i32(ctx, "context_lens"); check_i32(slots, "state_slots");
+  const int64_t T = qkv.size(0), B = slots.numel();
+  TORCH_CHECK(G >= 1 && H % G == 0 && qkv.size(1) >= 2 * G * Dk + H * V && beta.is_cuda() && beta.scalar_type() == qkv.scalar_type() && beta.size(0) == T &&
+              beta.size(1) >= H && dt.is_cuda() && dt.scalar_type() == qkv.scalar_type() && dt.size(0) == T && dt.size(1) >= H && dt_bias.numel() == H &&
+              A_log.numel() == H && cu.numel() == B + 1 && ctx.numel() >= B);
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == H && state.size(2) == Dk && state.size(3) == V, "delta-rule state [slots, heads, dim, vdim]");
+  const c10::cuda::CUDAGuard guard(qkv.device());
+  Tensor out = torch::empty({T, H * V}, qkv.options().dtype(torch::kFloat32));
+  if (T == 0) return out;
+  b200::HeadDeltaArgs a{qkv.data_ptr(), qkv.stride(0), beta.data_ptr(), beta.stride(0), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr<float>(), A_log.data_ptr<float>(),
+                        state.data_ptr<float>(), cu.data_ptr<int>(), ctx.data_ptr<int>(), slots.data_ptr<int>(), out.data_ptr<float>(), (int)B, (int)T, (int)H, (int)G,
+                        (int)Dk, (int)V, (float)q_scale, (float)unit_eps, nullptr};
+  const long long ws = b200::head_delta_workspace(a, (int)max_q);
+  Tensor pre;
+  if (ws > 0) { pre = torch::empty({(int64_t)ws}, out.options()); a.pre = pre.data_ptr<float>(); ++g_launches; }
+  LAUNCH_OK(b200::head_delta_launch(a, is_f32(qkv), (int)max_q, cur_stream()));
+  return out;
+}
+
 // out (optional): AT [T, >= col0 + width], the result goes to its columns col0 .. col0 + width
 Tensor hy_mingru_scan(const Tensor& rows, int64_t z0, int64_t x0, int64_t g0, int64_t R, Tensor state, const Tensor& cu, const Tensor& ctx, const Tensor& slots,
                       double out_mult, int64_t max_q, const c10::optional<Tensor>& out_, int64_t col0) {
@@ -1276,10 +1341,10 @@ Tensor hy_mingru_scan(const Tensor& rows, int64_t z0, int64_t x0, int64_t g0, in
 // qn, kn, v_first optional
 Tensor hy_qk_norm_rope_append(const Tensor& rows, int64_t q0, int64_t k0, int64_t v0, int64_t H, int64_t D, const c10::optional<Tensor>& qn,
                               const c10::optional<Tensor>& kn, double eps, const Tensor& inv_freq, Tensor kpool, Tensor vpool, const Tensor& slot_map,
-                              const Tensor& positions, bool half, bool norm_after, double rot_mult, const c10::optional<Tensor>& v_first, double lam) {
+                              const Tensor& positions, bool half, bool norm_after, double rot_mult, const c10::optional<Tensor>& v_first, double lam, bool whole) {
   check_act(rows, "rows"); check_rows(rows, "rows"); check_f32c(inv_freq, "inv_freq"); check_i32(slot_map, "slot_mapping"); check_i32(positions, "positions");
-  if (qn.has_value()) { check_f32c(*qn, "q norm"); TORCH_CHECK(qn->numel() == D); }
-  if (kn.has_value()) { check_f32c(*kn, "k norm"); TORCH_CHECK(kn->numel() == D); }
+  if (qn.has_value()) { check_f32c(*qn, "q norm"); TORCH_CHECK(qn->numel() == (whole ? H * D : D)); }
+  if (kn.has_value()) { check_f32c(*kn, "k norm"); TORCH_CHECK(kn->numel() == (whole ? kpool.size(1) * D : D)); }
   TORCH_CHECK(kpool.dim() == 4 && vpool.dim() == 4 && kpool.is_contiguous() && vpool.is_contiguous() && kpool.scalar_type() == rows.scalar_type() &&
               vpool.scalar_type() == rows.scalar_type() && kpool.size(0) == vpool.size(0) && kpool.size(1) == vpool.size(1) && kpool.size(2) == vpool.size(2) &&
               kpool.size(3) == D, "pools [pages, kv_heads, page, d] in the activation type");
@@ -1297,7 +1362,7 @@ Tensor hy_qk_norm_rope_append(const Tensor& rows, int64_t q0, int64_t k0, int64_
                                              qn.has_value() ? qn->data_ptr<float>() : nullptr, kn.has_value() ? kn->data_ptr<float>() : nullptr, (float)eps,
                                              inv_freq.data_ptr<float>(), (int)rot, positions.data_ptr<int>(), slot_map.data_ptr<int>(), (int)kpool.size(2),
                                              q.data_ptr<float>(), kpool.data_ptr(), vpool.data_ptr(), is_f32(rows), half, norm_after, (float)rot_mult,
-                                             v_first.has_value() ? v_first->data_ptr() : nullptr, v_first.has_value() ? v_first->stride(0) : 0, (float)lam, (int)T,
+                                             v_first.has_value() ? v_first->data_ptr() : nullptr, v_first.has_value() ? v_first->stride(0) : 0, (float)lam, whole, (int)T,
                                              cur_stream()));
   return q;
 }
@@ -1306,7 +1371,7 @@ namespace {
 // the arguments both forms of the attention with a sink share; `out` is allocated when it is not given
 b200::SinkAttnArgs sink_args(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
                              const Tensor& cu, double scale, int64_t block, int64_t window, int64_t keep, double out_mult, const c10::optional<Tensor>& gate,
-                             Tensor& out, const c10::optional<Tensor>& out_, int64_t col0) {
+                             Tensor& out, const c10::optional<Tensor>& out_, int64_t col0, const c10::optional<Tensor>& slopes, const c10::optional<Tensor>& bias) {
   check_f32c(q, "q"); check_i32(block_tables, "block_tables"); check_i32(cu, "cu_seqlens");
   TORCH_CHECK(q.dim() == 3 && kpool.dim() == 4 && vpool.dim() == 4 && kpool.is_contiguous() && vpool.is_contiguous() && kpool.scalar_type() == vpool.scalar_type() &&
               kpool.size(1) == vpool.size(1) && kpool.size(2) == vpool.size(2) && kpool.size(3) == q.size(2),
@@ -1318,8 +1383,15 @@ b200::SinkAttnArgs sink_args(const Tensor& q, const Tensor& kpool, const Tensor&
   if (sink.has_value()) { check_f32c(*sink, "sink"); TORCH_CHECK(sink->numel() == H); a.sink = sink->data_ptr<float>(); }
   if (gate.has_value()) {
     check_rows(*gate, "gate");
-    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == kpool.scalar_type() && gate->size(0) == T && gate->size(1) == H, "gate must be [T, heads] in the activation type");
-    a.gate = gate->data_ptr(); a.ld_gate = gate->stride(0);
+    TORCH_CHECK(gate->is_cuda() && gate->scalar_type() == kpool.scalar_type() && gate->size(0) == T && (gate->size(1) == H || gate->size(1) == H * V),
+                "gate must be [T, heads] or [T, heads * vdim] in the activation type");
+    a.gate = gate->data_ptr(); a.ld_gate = gate->stride(0); a.gate_elem = gate->size(1) != H;
+  }
+  if (slopes.has_value()) { check_f32c(*slopes, "slopes"); TORCH_CHECK(slopes->numel() == H); a.slopes = slopes->data_ptr<float>(); }
+  if (bias.has_value()) {
+    check_f32c(*bias, "distance bias");
+    TORCH_CHECK(bias->dim() == 2 && bias->size(0) == H && bias->size(1) >= 1, "distance bias must be [heads, distances]");
+    a.bias = bias->data_ptr<float>(); a.bias_len = (int)bias->size(1);
   }
   out = out_.has_value() ? *out_ : torch::empty({T, H * V}, kpool.options());
   check_rows(out, "out");
@@ -1338,11 +1410,12 @@ b200::SinkAttnArgs sink_args(const Tensor& q, const Tensor& kpool, const Tensor&
 
 Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
                          const Tensor& positions, const Tensor& cu, double scale, int64_t block, int64_t window, double out_mult, int64_t max_ctx,
-                         const c10::optional<Tensor>& out_, int64_t col0, int64_t keep, const c10::optional<Tensor>& gate) {
+                         const c10::optional<Tensor>& out_, int64_t col0, int64_t keep, const c10::optional<Tensor>& gate, const c10::optional<Tensor>& slopes,
+                         const c10::optional<Tensor>& bias) {
   check_i32(positions, "positions");
   const c10::cuda::CUDAGuard guard(q.device());
   Tensor out;
-  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0);
+  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0, slopes, bias);
   const int64_t T = q.size(0), H = a.H, G = a.G, V = a.V;
   TORCH_CHECK(V <= 512 && positions.numel() >= T, "attention with a sink: vdim <= 512");
   if (T == 0) return out;
@@ -1372,11 +1445,11 @@ Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpo
 // bf16, any number of sequences and query rows, tensor cores
 Tensor hy_sink_flash(const Tensor& q, const Tensor& kpool, const Tensor& vpool, const c10::optional<Tensor>& sink, const Tensor& block_tables,
                      const Tensor& ctx, const Tensor& cu, double scale, int64_t block, int64_t window, double out_mult, const c10::optional<Tensor>& out_,
-                     int64_t col0, int64_t keep, const c10::optional<Tensor>& gate) {
+                     int64_t col0, int64_t keep, const c10::optional<Tensor>& gate, const c10::optional<Tensor>& slopes, const c10::optional<Tensor>& bias) {
   check_i32(ctx, "context_lens"); check_bf16(kpool, "kpool");
   const c10::cuda::CUDAGuard guard(q.device());
   Tensor out;
-  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0);
+  b200::SinkAttnArgs a = sink_args(q, kpool, vpool, sink, block_tables, cu, scale, block, window, keep, out_mult, gate, out, out_, col0, slopes, bias);
   TORCH_CHECK(ctx.numel() >= a.B && out.stride(0) % 2 == 0 && col0 % 2 == 0, "tensor-core attention: even output columns and rows");
   if (q.size(0) == 0) return out;
   LAUNCH_OK(b200::sink_flash_launch(a, ctx.data_ptr<int>(), (int)((q.size(0) + 63) / 64 + a.B), cur_stream()));
@@ -1502,8 +1575,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("hy_gelu_erf_", &hy_gelu_erf_);
   m.def("hy_post_norm_add_", &hy_post_norm_add_);
   m.def("hy_rmsnorm_cast", &hy_rmsnorm_cast);
-  m.def("hy_gated_rmsnorm", &hy_gated_rmsnorm);
+  m.def("hy_gated_rmsnorm", &hy_gated_rmsnorm, py::arg("y"), py::arg("gate"), py::arg("w"), py::arg("eps"), py::arg("groups"), py::arg("mode"), py::arg("out_f32"),
+        py::arg("out") = py::none(), py::arg("col0") = 0);
   m.def("hy_causal_conv_silu", &hy_causal_conv_silu);
+  m.def("hy_conv_qkv_append", &hy_conv_qkv_append);
   m.def("hy_ssm_scan", &hy_ssm_scan);
   m.def("hy_decay_scan", &hy_decay_scan);
   m.def("hy_latent_prologue", &hy_latent_prologue, py::arg("x"), py::arg("q_rank"), py::arg("kv_rank"), py::arg("qn_w"), py::arg("kvn_w"), py::arg("eps"),
@@ -1516,7 +1591,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("hy_scaled_add_norm_", &hy_scaled_add_norm_, py::arg("x"), py::arg("y"), py::arg("ls"), py::arg("w"), py::arg("eps"), py::arg("act_f32"),
         py::arg("extra") = py::none(), py::arg("gate") = py::none(), py::arg("mult") = 1.0);
   m.def("hy_mlstm_scan", &hy_mlstm_scan);
-  m.def("hy_sigmoid_topk", &hy_sigmoid_topk, py::arg("z"), py::arg("E"), py::arg("top"), py::arg("mode") = 0, py::arg("bias") = py::none());
+  m.def("hy_sigmoid_topk", &hy_sigmoid_topk, py::arg("z"), py::arg("E"), py::arg("top"), py::arg("mode") = 0, py::arg("bias") = py::none(),
+        py::arg("normalise") = false, py::arg("scale") = 1.0);
   m.def("hy_clamped_glu", &hy_clamped_glu, py::arg("gate"), py::arg("up"), py::arg("limit"), py::arg("row_of") = py::none(), py::arg("scale") = py::none(),
         py::arg("kind") = 0);
   m.def("hy_gather_sum", &hy_gather_sum, py::arg("y"), py::arg("row_of"), py::arg("k"), py::arg("wts") = py::none());
@@ -1526,21 +1602,24 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("hy_paged_kv_append", &hy_paged_kv_append);
   m.def("hy_diff_attention", &hy_diff_attention);
   m.def("hy_diff_head_norm", &hy_diff_head_norm);
-  m.def("hy_stream_embed", &hy_stream_embed);
+  m.def("hy_stream_embed", &hy_stream_embed, py::arg("table"), py::arg("ids"), py::arg("scale"), py::arg("streams"), py::arg("pos") = py::none(),
+        py::arg("positions") = py::none());
   m.def("hy_hyper_step_", &hy_hyper_step_);
   m.def("hy_relu2_", &hy_relu2_);
   m.def("hy_delta_scan", &hy_delta_scan);
+  m.def("hy_head_delta_scan", &hy_head_delta_scan);
   m.def("hy_mingru_scan", &hy_mingru_scan, py::arg("rows"), py::arg("z0"), py::arg("x0"), py::arg("g0"), py::arg("width"), py::arg("state"), py::arg("cu"),
         py::arg("ctx"), py::arg("slots"), py::arg("out_mult"), py::arg("max_q"), py::arg("out") = py::none(), py::arg("col0") = 0);
   m.def("hy_qk_norm_rope_append", &hy_qk_norm_rope_append, py::arg("rows"), py::arg("q0"), py::arg("k0"), py::arg("v0"), py::arg("heads"), py::arg("dim"),
         py::arg("qn"), py::arg("kn"), py::arg("eps"), py::arg("inv_freq"), py::arg("kpool"), py::arg("vpool"), py::arg("slot_map"), py::arg("positions"),
-        py::arg("half") = false, py::arg("norm_after") = false, py::arg("rot_mult") = 1.0, py::arg("v_first") = py::none(), py::arg("lam") = 0.0);
+        py::arg("half") = false, py::arg("norm_after") = false, py::arg("rot_mult") = 1.0, py::arg("v_first") = py::none(), py::arg("lam") = 0.0, py::arg("whole") = false);
   m.def("hy_sink_attention", &hy_sink_attention, py::arg("q"), py::arg("kpool"), py::arg("vpool"), py::arg("sink"), py::arg("block_tables"), py::arg("positions"),
         py::arg("cu"), py::arg("scale"), py::arg("block"), py::arg("window"), py::arg("out_mult"), py::arg("max_ctx"), py::arg("out") = py::none(),
-        py::arg("col0") = 0, py::arg("keep") = 0, py::arg("gate") = py::none());
+        py::arg("col0") = 0, py::arg("keep") = 0, py::arg("gate") = py::none(), py::arg("slopes") = py::none(), py::arg("bias") = py::none());
   m.def("hy_sink_flash", &hy_sink_flash, py::arg("q"), py::arg("kpool"), py::arg("vpool"), py::arg("sink"), py::arg("block_tables"), py::arg("context_lens"),
         py::arg("cu"), py::arg("scale"), py::arg("block"), py::arg("window"), py::arg("out_mult"), py::arg("out") = py::none(), py::arg("col0") = 0,
-        py::arg("keep") = 0, py::arg("gate") = py::none());
+        py::arg("keep") = 0, py::arg("gate") = py::none(), py::arg("slopes") = py::none(), py::arg("bias") = py::none());
+  m.def("hy_sink_flash_bias_max", []() { return b200::sink_flash_bias_max(); });
   m.def("hy_sink_flash_supported", [](int64_t d, int64_t v) { return b200::sink_flash_supported((int)d, (int)v); });
   m.def("hy_selective_scan", &hy_selective_scan);
   m.def("hy_group_softmax_topk", &hy_group_softmax_topk);

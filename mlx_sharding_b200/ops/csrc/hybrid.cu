@@ -67,10 +67,48 @@ __global__ void rmsnorm_cast_kernel(const float* __restrict__ x, long long ld_x,
   for (int c = threadIdx.x; c < n; c += blockDim.x) stf<AT>(out + t * n + c, xr[c] * r * w[c]);
 }
 
-// mode 0: norm_groups(y * silu(g)) * w      mode 1: norm(y) * w * sigmoid(g)        grid (T, groups)
+// mode 0: norm_groups(y * silu(g)) * w      mode 1: norm(y) * w * sigmoid(g)      mode 2: norm(y) * w * silu(g)
+__device__ __forceinline__ float post_gate(int mode, float v, float g) { return mode == 1 ? v * sigmoid_f(g) : mode == 2 ? v * silu_f(g) : v; }
+
+// One warp per (row, group), four adjacent entries per lane at a time (group size a multiple of 4, at most 128 NV; 16-byte aligned fp32 rows,
+// gate and output rows aligned to four entries).                                        grid ceil(T * groups / 8), block 256
+template <typename AT, int NV>
+__global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ y, const AT* __restrict__ g, long long ld_g, const float* __restrict__ w,
+                                         AT* __restrict__ out, long long ld_o, int C, int groups, int mode, float eps, long long n) {
+  const long long i = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (i >= n) return;
+  const long long t = i / groups;
+  const int gs = C / groups, c0 = (int)(i % groups) * gs, lane = threadIdx.x & 31;
+  float v[NV][4], gv[NV][4], ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = 4 * (lane + 32 * k);
+    if (c < gs) {
+      const float4 a = *reinterpret_cast<const float4*>(y + t * C + c0 + c);
+      v[k][0] = a.x; v[k][1] = a.y; v[k][2] = a.z; v[k][3] = a.w;
+      load4<AT>(g + t * ld_g + c0 + c, gv[k]);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) { if (mode == 0) v[k][e] *= silu_f(gv[k][e]); ss += v[k][e] * v[k][e]; }
+    }
+  }
+  const float r = rsqrtf(warp_sum(ss) / (float)gs + eps);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int c = 4 * (lane + 32 * k);
+    if (c < gs) {
+      const float4 wv = *reinterpret_cast<const float4*>(w + c0 + c);
+      const float f[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[k][e] = post_gate(mode, v[k][e] * r * f[e], gv[k][e]);
+      store4<AT>(out + t * ld_o + c0 + c, v[k]);
+    }
+  }
+}
+
+// any size                                                                              grid (T, groups)
 template <typename AT>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ y, const AT* __restrict__ g, long long ld_g, const float* __restrict__ w,
-                                     AT* __restrict__ out, int C, int groups, int mode, float eps) {
+                                     AT* __restrict__ out, long long ld_o, int C, int groups, int mode, float eps) {
   __shared__ float red[32];
   const long long t = blockIdx.x;
   const int gs = C / groups, c0 = blockIdx.y * gs;
@@ -87,22 +125,40 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ y, const AT* __re
     float v = yr[c];
     const float gv = ldf<AT>(gr + c);
     if (mode == 0) v *= silu_f(gv);
-    v = v * r * w[c0 + c];
-    if (mode == 1) v *= sigmoid_f(gv);
-    stf<AT>(out + t * C + c0 + c, v);
+    stf<AT>(out + t * ld_o + c0 + c, post_gate(mode, v * r * w[c0 + c], gv));
   }
 }
 
 // ---------------------------------------------------------------------------------------------------------- short convolution
-// out[t, c] = silu(b[c] + sum_k w[c, k] * in(t - (K-1) + k, c)); inputs before this step come from the sequence's conv state
+// out[t, c] = f(b[c] + sum_k w[c, k] * in(t - (K-1) + k, c)), f and the place of the result as ConvOut says (b nullable); inputs before this step come from the sequence's conv state
 // ([slots, K-1, C], the last K-1 inputs), inputs before position 0 are zero.  A thread walks kConvRows rows of one channel with the last
 // K-1 inputs in registers (KT = K - 1 as a constant; the rows' loads are issued together).     grid (ceil(C / blockDim), ceil(T / kConvRows))
 constexpr int kConvRows = 8;
 
-template <typename AT, int KT>
-__global__ void causal_conv_silu_kernel(const AT* __restrict__ u, long long ld_u, const float* __restrict__ w, const float* __restrict__ bias,
-                                        const AT* __restrict__ cstate, const int* __restrict__ cu, const int* __restrict__ ctx,
-                                        const int* __restrict__ slots, int B, int C, int T, AT* __restrict__ out) {
+// QKV = false: silu(.) -> out [T, C].  QKV = true: no activation; the channels are [q: qc | k: G D | v: G V]: queries -> fp32 q [T, qc], keys and
+// values -> the paged pools at slot_map[t] (C == qc: queries alone).
+template <typename AT, bool QKV> struct ConvOut {
+  AT* out; float* q; AT* kpool; AT* vpool; const int* slot_map;
+  int C, qc, G, D, V, page;
+  struct Column { long long base; int stride, kind; };           // of one channel: kind 0 queries, 1 keys, 2 values
+  __device__ __forceinline__ Column column(int c) const {
+    if (!QKV || c < qc) return {c, 0, 0};
+    const bool key = c - qc < G * D;
+    const int i = key ? c - qc : c - qc - G * D, d = key ? D : V;
+    return {(long long)(i / d) * page * d + i % d, d, key ? 1 : 2};
+  }
+  __device__ __forceinline__ void put(const Column& k, long long t, float v) const {
+    if (!QKV) { stf<AT>(out + t * C + k.base, silu_f(v)); return; }
+    if (k.kind == 0) { q[t * qc + k.base] = v; return; }
+    const int slot = slot_map[t], pg = slot / page, off = slot - pg * page;
+    stf<AT>((k.kind == 1 ? kpool : vpool) + (long long)pg * G * page * k.stride + (long long)off * k.stride + k.base, v);
+  }
+};
+
+template <typename AT, int KT, bool QKV>
+__global__ void causal_conv_kernel(const AT* __restrict__ u, long long ld_u, const float* __restrict__ w, const float* __restrict__ bias,
+                                   const AT* __restrict__ cstate, const int* __restrict__ cu, const int* __restrict__ ctx,
+                                   const int* __restrict__ slots, int B, int C, int T, ConvOut<AT, QKV> dst) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x, t0 = blockIdx.y * kConvRows, t1 = min(T, t0 + kConvRows);
   if (c >= C) return;
   AT raw[kConvRows];
@@ -111,7 +167,8 @@ __global__ void causal_conv_silu_kernel(const AT* __restrict__ u, long long ld_u
   float wr[KT + 1], win[KT + 1];
 #pragma unroll
   for (int k = 0; k <= KT; ++k) wr[k] = w[(long long)c * (KT + 1) + k];
-  const float b0 = bias[c];
+  const float b0 = bias != nullptr ? bias[c] : 0.f;
+  const auto col = dst.column(c);
   int b = seq_of(cu, B, t0);
   auto enter = [&](int t) {                  // the KT inputs in front of row t of sequence b
     const int j = t - cu[b], c0 = ctx[b] - (cu[b + 1] - cu[b]);
@@ -136,7 +193,7 @@ __global__ void causal_conv_silu_kernel(const AT* __restrict__ u, long long ld_u
     float acc = b0;
 #pragma unroll
     for (int k = 0; k <= KT; ++k) acc = fmaf(wr[k], win[k], acc);
-    stf<AT>(out + (long long)t * C + c, silu_f(acc));
+    dst.put(col, t, acc);
 #pragma unroll
     for (int k = 0; k < KT; ++k) win[k] = win[k + 1];
   }
@@ -144,9 +201,9 @@ __global__ void causal_conv_silu_kernel(const AT* __restrict__ u, long long ld_u
 
 // One token per sequence: convolution and state shift in one pass.  A thread owns one (sequence, channel) column.
 //                                                                                       grid (ceil(C / blockDim), B)
-template <typename AT, int KT>
+template <typename AT, int KT, bool QKV>
 __global__ void conv_step_kernel(const AT* __restrict__ u, long long ld_u, const float* __restrict__ w, const float* __restrict__ bias, AT* __restrict__ cstate,
-                                 const int* __restrict__ cu, const int* __restrict__ ctx, const int* __restrict__ slots, int C, AT* __restrict__ out) {
+                                 const int* __restrict__ cu, const int* __restrict__ ctx, const int* __restrict__ slots, int C, ConvOut<AT, QKV> dst) {
   const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y, t = cu[b];
   if (c >= C || cu[b + 1] == t) return;
   const bool fresh = ctx[b] == 1;
@@ -155,13 +212,13 @@ __global__ void conv_step_kernel(const AT* __restrict__ u, long long ld_u, const
 #pragma unroll
   for (int k = 0; k < KT; ++k) h[k] = st[(long long)k * C];
   h[KT] = u[t * ld_u + c];
-  float acc = bias[c];
+  float acc = bias != nullptr ? bias[c] : 0.f;
 #pragma unroll
   for (int k = 0; k <= KT; ++k) {
     if (fresh && k < KT) stf<AT>(&h[k], 0.f);
     acc = fmaf(w[(long long)c * (KT + 1) + k], ldf<AT>(&h[k]), acc);
   }
-  stf<AT>(out + (long long)t * C + c, silu_f(acc));
+  dst.put(dst.column(c), t, acc);
 #pragma unroll
   for (int k = 0; k < KT; ++k) st[(long long)k * C] = h[k + 1];
 }
@@ -518,7 +575,7 @@ __global__ void sink_softmax_kernel(const float* __restrict__ s, const float* __
 }
 
 // ---------------------------------------------------------------------------------------------------------- pre-norm residual step
-// x += (y + extra * sigmoid(gate[t])) * ls * mult   (x, y, extra fp32; ls, extra nullable);   xa = (AT)(x * rsqrt(mean(x^2) + eps) * w)
+// x += (y + extra * sigmoid(gate[t])) * ls * mult   (x, y, extra fp32; ls, extra, gate nullable: without a gate the factor of extra is 1);   xa = (AT)(x * rsqrt(mean(x^2) + eps) * w)
 template <typename AT>
 __global__ void scaled_add_norm_kernel(float* __restrict__ x, const float* __restrict__ y, long long ld_y, const float* __restrict__ ls,
                                        const float* __restrict__ extra, long long ld_e, const float* __restrict__ gate, long long ld_gate,
@@ -527,7 +584,7 @@ __global__ void scaled_add_norm_kernel(float* __restrict__ x, const float* __res
   const long long t = blockIdx.x;
   const float* yr = y + t * ld_y;
   const float* er = extra != nullptr ? extra + t * ld_e : nullptr;
-  const float sg = extra != nullptr ? sigmoid_f(gate[t * ld_gate]) : 0.f;
+  const float sg = gate != nullptr ? sigmoid_f(gate[t * ld_gate]) : 1.f;
   float ss = 0.f;
   for (int c = threadIdx.x; c < n; c += blockDim.x) {
     float v = yr[c];
@@ -561,7 +618,7 @@ __global__ void scaled_add_norm_vec_kernel(float* __restrict__ x, const float* _
     const int c = min(threadIdx.x + i * blockDim.x, n4 - 1);
     xv[i] = xr[c]; yv[i] = yr[c]; wv[i] = wr[c];
   }
-  const float sg = extra != nullptr ? sigmoid_f(gate[t * ld_gate]) : 0.f;
+  const float sg = gate != nullptr ? sigmoid_f(gate[t * ld_gate]) : 1.f;
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -709,15 +766,17 @@ __global__ void mlstm_scan_kernel(MlstmArgs a, int PB, int R, int kTok) {
 }
 
 // ---------------------------------------------------------------------------------------------------------- mixture of experts
-// Router on fp32 logits, the `top` largest scores (ties: lowest id).  One warp per token.  mode 0: scores sigmoid(z), weights = the chosen
-// scores; mode 1: scores z + bias (bias nullable), weights = softmax over the chosen scores alone.
+// Router on fp32 logits, the `top` largest scores (ties: lowest id).  One warp per token.  mode 0: choice by sigmoid(z) + bias, weights = the
+// chosen experts' sigmoid(z), divided by their sum + 1e-20 (normalise), times `scale`; mode 1: choice by z + bias, weights = softmax over the
+// chosen ones alone.  bias nullable.
 __global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z, const float* __restrict__ bias, int mode, int E, int top,
-                                    int* __restrict__ idx, float* __restrict__ w) {
+                                    int* __restrict__ idx, float* __restrict__ w, bool normalise, float scale) {
   extern __shared__ float sc[];             // [E]
   const long long t = blockIdx.x;
   const int lane = threadIdx.x;
-  for (int e = lane; e < E; e += 32) sc[e] = mode == 0 ? sigmoid_f(z[t * ld_z + e]) : z[t * ld_z + e] + (bias != nullptr ? bias[e] : 0.f);
+  for (int e = lane; e < E; e += 32) sc[e] = (mode == 0 ? sigmoid_f(z[t * ld_z + e]) : z[t * ld_z + e]) + (bias != nullptr ? bias[e] : 0.f);
   __syncwarp();
+  float sum = 0.f;
   for (int j = 0; j < top; ++j) {
     float best = -INFINITY; int bi = 0x7fffffff;
     for (int e = lane; e < E; e += 32) { const float v = sc[e]; if (v > best) { best = v; bi = e; } }   // ascending e: first maximum wins
@@ -727,12 +786,18 @@ __global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z,
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
     }
-    if (lane == 0) { idx[t * top + j] = bi; w[t * top + j] = best; sc[bi] = -INFINITY; }
+    if (lane == 0) {
+      const float v = mode == 0 && bias != nullptr ? sigmoid_f(z[t * ld_z + bi]) : best;
+      idx[t * top + j] = bi; w[t * top + j] = v * scale; sc[bi] = -INFINITY;
+      sum += v;
+    }
     __syncwarp();
   }
+  if (mode == 0 && normalise && lane == 0)
+    for (int j = 0; j < top; ++j) w[t * top + j] /= sum + 1e-20f;
   if (mode == 1 && lane == 0) {             // the first chosen score is the largest
     const float m = w[t * top];
-    float sum = 0.f;
+    sum = 0.f;
     for (int j = 0; j < top; ++j) sum += expf(w[t * top + j] - m);
     for (int j = 0; j < top; ++j) w[t * top + j] = expf(w[t * top + j] - m) / sum;
   }
@@ -826,33 +891,59 @@ cudaError_t rmsnorm_cast_launch(const float* x, long long ld_x, const float* w, 
 }
 
 cudaError_t gated_rmsnorm_launch(const float* y, const void* g, long long ld_g, const float* w, void* out, bool f32, int C, int groups,
-                                 int mode, float eps, int T, cudaStream_t s) {
+                                 int mode, float eps, int T, long long ld_o, cudaStream_t s) {
+  const int gs = C / groups, es = f32 ? 4 : 2;
+  auto ok = [&](const void* p, long long ld) { return (reinterpret_cast<uintptr_t>(p) % (4 * es)) == 0 && ld % 4 == 0; };
+  if (gs % 4 == 0 && gs <= 512 && C % 4 == 0 && ok(g, ld_g) && ok(out, ld_o) && ((reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w)) & 15) == 0) {
+    const long long n = (long long)T * groups;
+    const unsigned grid = (unsigned)((n + 7) / 8);
+    if (gs <= 128) AT_DISPATCH(f32, (gated_rmsnorm_vec_kernel<AT, 1><<<grid, 256, 0, s>>>(y, (const AT*)g, ld_g, w, (AT*)out, ld_o, C, groups, mode, eps, n)));
+    else AT_DISPATCH(f32, (gated_rmsnorm_vec_kernel<AT, 4><<<grid, 256, 0, s>>>(y, (const AT*)g, ld_g, w, (AT*)out, ld_o, C, groups, mode, eps, n)));
+    return last();
+  }
   dim3 grid(T, groups);
-  AT_DISPATCH(f32, (gated_rmsnorm_kernel<AT><<<grid, 256, 0, s>>>(y, (const AT*)g, ld_g, w, (AT*)out, C, groups, mode, eps)));
+  AT_DISPATCH(f32, (gated_rmsnorm_kernel<AT><<<grid, 256, 0, s>>>(y, (const AT*)g, ld_g, w, (AT*)out, ld_o, C, groups, mode, eps)));
   return last();
 }
 
-template <typename AT, int KT>
+template <typename AT, int KT, bool QKV>
 static cudaError_t conv_t(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu, const int* ctx, const int* slots, int B, int C,
-                          void* out, int max_q, int T, cudaStream_t s) {
+                          const ConvOut<AT, QKV>& dst, int max_q, int T, cudaStream_t s) {
   const int nc = (C + 127) / 128;
   if (max_q <= 1) {
-    conv_step_kernel<AT, KT><<<dim3(nc, B), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (AT*)cstate, cu, ctx, slots, C, (AT*)out);
+    conv_step_kernel<AT, KT, QKV><<<dim3(nc, B), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (AT*)cstate, cu, ctx, slots, C, dst);
     return last();
   }
-  causal_conv_silu_kernel<AT, KT><<<dim3(nc, (T + kConvRows - 1) / kConvRows), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (const AT*)cstate, cu, ctx, slots, B, C, T, (AT*)out);
+  causal_conv_kernel<AT, KT, QKV><<<dim3(nc, (T + kConvRows - 1) / kConvRows), 128, 0, s>>>((const AT*)u, ld_u, w, bias, (const AT*)cstate, cu, ctx, slots, B, C, T, dst);
   if (KT > 0) conv_state_update_kernel<AT><<<dim3(B, (C + 255) / 256), 256, 0, s>>>((const AT*)u, ld_u, (AT*)cstate, cu, ctx, slots, C, KT + 1);
   return last();
 }
 
-cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
-                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int max_q, int T, cudaStream_t s) {
-#define CONV_CASE(KK) case KK: AT_DISPATCH(f32, return (conv_t<AT, KK - 1>(u, ld_u, w, bias, cstate, cu, ctx, slots, B, C, out, max_q, T, s))); break;
+template <typename AT, bool QKV>
+static cudaError_t conv_taps(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu, const int* ctx, const int* slots, int B,
+                             int C, int K, const ConvOut<AT, QKV>& dst, int max_q, int T, cudaStream_t s) {
+#define CONV_CASE(KK) case KK: return conv_t<AT, KK - 1, QKV>(u, ld_u, w, bias, cstate, cu, ctx, slots, B, C, dst, max_q, T, s);
   switch (K) {
     CONV_CASE(1) CONV_CASE(2) CONV_CASE(3) CONV_CASE(4) CONV_CASE(5) CONV_CASE(6) CONV_CASE(7) CONV_CASE(8) CONV_CASE(9) CONV_CASE(10) CONV_CASE(11) CONV_CASE(12)
     CONV_CASE(13) CONV_CASE(14) CONV_CASE(15) CONV_CASE(16) CONV_CASE(17)
   }
 #undef CONV_CASE
+  return cudaErrorInvalidValue;
+}
+
+cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
+                                    const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int max_q, int T, cudaStream_t s) {
+  AT_DISPATCH(f32, const ConvOut<AT, false> dst{(AT*)out, nullptr, nullptr, nullptr, nullptr, C, 0, 1, 1, 1, 1};
+              return conv_taps(u, ld_u, w, bias, cstate, cu, ctx, slots, B, C, K, dst, max_q, T, s));
+  return cudaErrorInvalidValue;
+}
+
+cudaError_t conv_qkv_append_launch(const void* u, long long ld_u, const float* w, void* cstate, const int* cu, const int* ctx, const int* slots, int B, int C, int K,
+                                   float* q, int qc, void* kpool, void* vpool, const int* slot_map, int G, int D, int V, int page, bool f32, int max_q, int T,
+                                   cudaStream_t s) {
+  if (C != qc && C != qc + G * (D + V)) return cudaErrorInvalidValue;
+  AT_DISPATCH(f32, const ConvOut<AT, true> dst{nullptr, q, (AT*)kpool, (AT*)vpool, slot_map, C, qc, G, D, V, page};
+              return conv_taps(u, ld_u, w, nullptr, cstate, cu, ctx, slots, B, C, K, dst, max_q, T, s));
   return cudaErrorInvalidValue;
 }
 
@@ -979,10 +1070,10 @@ cudaError_t mlstm_scan_launch(const void* in, long long ld_in, const float* gate
   return last();
 }
 
-cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias, int mode, int E, int top, int* idx, float* w, int T,
+cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias, int mode, int E, int top, int* idx, float* w, bool normalise, float scale, int T,
                                cudaStream_t s) {
   if (top > E || (size_t)E * sizeof(float) > 48 * 1024) return cudaErrorInvalidValue;
-  sigmoid_topk_kernel<<<T, 32, E * sizeof(float), s>>>(z, ld_z, bias, mode, E, top, idx, w);
+  sigmoid_topk_kernel<<<T, 32, E * sizeof(float), s>>>(z, ld_z, bias, mode, E, top, idx, w, normalise, scale);
   return last();
 }
 

@@ -13,9 +13,13 @@ cudaError_t post_norm_add_launch(float* x, const float* y, long long ld_y, const
                                  cudaStream_t s);
 cudaError_t rmsnorm_cast_launch(const float* x, long long ld_x, const float* w, void* out, bool f32, int n, float eps, int T, cudaStream_t s);
 cudaError_t gated_rmsnorm_launch(const float* y, const void* g, long long ld_g, const float* w, void* out, bool f32, int C, int groups,
-                                 int mode, float eps, int T, cudaStream_t s);
+                                 int mode, float eps, int T, long long ld_o, cudaStream_t s);
 cudaError_t causal_conv_silu_launch(const void* u, long long ld_u, const float* w, const float* bias, void* cstate, const int* cu,
                                     const int* ctx, const int* slots, int B, int C, int K, void* out, bool f32, int max_q, int T, cudaStream_t s);
+// no activation, no bias; channels [q: qc | k: G D | v: G V] (or q alone) -> q fp32 [T, qc] and the paged pools
+cudaError_t conv_qkv_append_launch(const void* u, long long ld_u, const float* w, void* cstate, const int* cu, const int* ctx, const int* slots, int B, int C, int K,
+                                   float* q, int qc, void* kpool, void* vpool, const int* slot_map, int G, int D, int V, int page, bool f32, int max_q, int T,
+                                   cudaStream_t s);
 cudaError_t ssm_scan_launch(const void* xbc, long long ld_x, const void* dt, long long ld_dt, const float* dt_bias, const float* A_log,
                             const float* D, float* state, const int* cu, const int* ctx, const int* slots, float* out, int B, int H, int N,
                             int P, int G, bool f32, int max_q, cudaStream_t s);
@@ -39,8 +43,9 @@ cudaError_t scaled_add_norm_launch(float* x, const float* y, long long ld_y, con
 cudaError_t mlstm_scan_launch(const void* in, long long ld_in, const float* gates, long long ld_g, const float* gate_bias, float* S, float* n,
                               float* m, const int* cu, const int* ctx, const int* slots, float* out, int B, int H, int N, int P, int PB,
                               float cap, float q_scale, bool f32, int max_q, cudaStream_t s);
-// mode 0: sigmoid scores, weights = chosen scores; mode 1: logits + bias, weights = softmax over the chosen logits
-cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias, int mode, int E, int top, int* idx, float* w, int T,
+// mode 0: sigmoid scores + bias, weights = chosen scores without it (normalise: over their sum) * scale; mode 1: logits + bias, weights = softmax
+// over the chosen logits
+cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias, int mode, int E, int top, int* idx, float* w, bool normalise, float scale, int T,
                                cudaStream_t s);
 // kind 0: clamped GLU (limit); kind 1: silu(g) * u * scale; kind 2: gelu_tanh(g) * u * scale
 cudaError_t clamped_glu_launch(const void* g, long long ld_g, const void* u, long long ld_u, int F, float limit, const int* row_of,

@@ -31,6 +31,23 @@ template <> __device__ __forceinline__ void unpack16<__nv_bfloat16>(const uint4&
   for (int i = 0; i < 4; ++i) { dst[2 * i] = __uint_as_float(w[i] << 16); dst[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
 }
 
+// four adjacent activations <-> floats (pointers aligned to four entries)
+template <typename T> __device__ __forceinline__ void load4(const T* p, float* f);
+template <> __device__ __forceinline__ void load4<float>(const float* p, float* f) {
+  const float4 a = *reinterpret_cast<const float4*>(p);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+}
+template <> __device__ __forceinline__ void load4<__nv_bfloat16>(const __nv_bfloat16* p, float* f) {
+  const uint2 a = *reinterpret_cast<const uint2*>(p);
+  f[0] = __uint_as_float(a.x << 16); f[1] = __uint_as_float(a.x & 0xffff0000u); f[2] = __uint_as_float(a.y << 16); f[3] = __uint_as_float(a.y & 0xffff0000u);
+}
+template <typename T> __device__ __forceinline__ void store4(T* p, const float* f);
+template <> __device__ __forceinline__ void store4<float>(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+template <> __device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, const float* f) {
+  __nv_bfloat162 lo = __floats2bfloat162_rn(f[0], f[1]), hi = __floats2bfloat162_rn(f[2], f[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(reinterpret_cast<unsigned&>(lo), reinterpret_cast<unsigned&>(hi));
+}
+
 // two floats in one 64-bit register: packed multiply and multiply-add
 __device__ __forceinline__ float2 mul2(float2 a, float2 b) {
   float2 r;
@@ -59,6 +76,37 @@ __device__ __forceinline__ float warp_max(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
   return v;
+}
+// Sums of NV values over LK lanes, every lane gets all of them: each level sends half of the values that are left one way and keeps the other
+// half (NV - 1 shuffles in all instead of NV log2 LK), then the totals are handed round.
+template <int NV, int LK> __device__ __forceinline__ void sum_over_lanes(float (&v)[NV], int lane) {
+  int left = NV;
+#pragma unroll
+  for (int w = 1; w < LK; w <<= 1) {
+    if (left > 1) {
+      left >>= 1;
+      const bool up = lane & w;
+#pragma unroll
+      for (int i = 0; i < NV / 2; ++i)
+        if (i < left) {
+          const float send = up ? v[i] : v[i + left], keep = up ? v[i + left] : v[i];
+          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+        }
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], w);
+    }
+  }
+  float r[NV];
+#pragma unroll
+  for (int x = 0; x < NV; ++x) {
+    int src = 0, n = NV;
+#pragma unroll
+    for (int w = 1; w < LK; w <<= 1)
+      if (n > 1) { n >>= 1; if (x & n) src |= w; }
+    r[x] = __shfl_sync(0xffffffffu, v[x % left], src, LK);
+  }
+#pragma unroll
+  for (int x = 0; x < NV; ++x) v[x] = r[x];
 }
 // sum over the block (blockDim.x <= 1024, multiple of 32); every thread gets the result
 __device__ __forceinline__ float block_sum(float v, float* red) {

@@ -1,5 +1,5 @@
 // Grouped-query attention over paged keys / values with a sink in the softmax: keys visible inside fixed blocks of positions or a sliding
-// window, beside kept first tokens; the result of a head times a gate.  For steps of few query rows (decode, short portions), for exact
+// window, beside kept first tokens; a bias by distance (slope per head, table per head) on the scores; the result times a gate.  For steps of few query rows (decode, short portions), for exact
 // mode and for any size; long bf16 portions run on the tensor cores (attention_prefill.cu).
 //
 // Conventions as in hybrid.cu; scores, softmax and accumulators are fp32.  The visible keys of a query at position p are numbered
@@ -24,8 +24,16 @@ struct Visible {
   __device__ __forceinline__ int key_at(int i) const { return i < kept ? i : lo + i - kept; }
 };
 
-template <typename AT> __device__ __forceinline__ float head_factor(const SinkAttnArgs& a, long long t, int h) {
-  return a.gate != nullptr ? a.out_mult * sigmoid_f(ldf<AT>((const AT*)a.gate + t * a.ld_gate + h)) : a.out_mult;
+// factor of element d of head h
+template <typename AT> __device__ __forceinline__ float out_factor(const SinkAttnArgs& a, long long t, int h, int d) {
+  return a.gate != nullptr ? a.out_mult * sigmoid_f(ldf<AT>((const AT*)a.gate + t * a.ld_gate + (a.gate_elem ? h * a.V + d : h))) : a.out_mult;
+}
+// added to the score of head h and a key n tokens back
+__device__ __forceinline__ float distance_bias(const SinkAttnArgs& a, int h, int n) {
+  float b = 0.f;
+  if (a.slopes != nullptr) b -= a.slopes[h] * (float)n;
+  if (a.bias != nullptr) b += a.bias[h * a.bias_len + min(n, a.bias_len - 1)];
+  return b;
 }
 
 // ---------------------------------------------------------------------------------------------------------- vector form
@@ -58,44 +66,13 @@ __device__ __forceinline__ void chunk_get(const float* p, float2* f) {
 
 constexpr int kRowWarps = 4;
 
-// Sums of NV values over LK lanes, every lane gets all of them: each level sends half of the values that are left one way and keeps the other
-// half (NV - 1 shuffles in all instead of NV log2 LK), then the totals are handed round.
-template <int NV, int LK> __device__ __forceinline__ void sum_over_lanes(float (&v)[NV], int lane) {
-  int left = NV;
-#pragma unroll
-  for (int w = 1; w < LK; w <<= 1) {
-    if (left > 1) {
-      left >>= 1;
-      const bool up = lane & w;
-#pragma unroll
-      for (int i = 0; i < NV / 2; ++i)
-        if (i < left) {
-          const float send = up ? v[i] : v[i + left], keep = up ? v[i + left] : v[i];
-          v[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
-        }
-    } else {
-      v[0] += __shfl_xor_sync(0xffffffffu, v[0], w);
-    }
-  }
-  float r[NV];
-#pragma unroll
-  for (int x = 0; x < NV; ++x) {
-    int src = 0, n = NV;
-#pragma unroll
-    for (int w = 1; w < LK; w <<= 1)
-      if (n > 1) { n >>= 1; if (x & n) src |= w; }
-    r[x] = __shfl_sync(0xffffffffu, v[x % left], src, LK);
-  }
-#pragma unroll
-  for (int x = 0; x < NV; ++x) v[x] = r[x];
-}
-
 // grid (tokens, G * ceil((H/G) / RG), key splits), 4 warps.  LK lanes share a key: each holds 8 adjacent entries of the key and of the value
 // (dim and vdim multiples of 8, at most 8 LK), so a warp takes 32 / LK keys at a time, U of them per lane group and step, straight from the
 // pages by asynchronous copies of S - 1 steps ahead — every thread reads back only what it copied itself, so no barrier is involved — and
 // uses them for RG query heads.  Every lane group runs an online softmax (base 2) of its own over its keys;
-// the groups are merged at the end, over the lanes of a warp by shuffles and over the warps in shared memory.
-template <typename AT, int LK, int RG, int U, int S>
+// the groups are merged at the end, over the lanes of a warp by shuffles and over the warps in shared memory.  BIAS: distance_bias on the scores,
+// fetched before the wait for the keys.
+template <typename AT, int LK, int RG, int U, int S, bool BIAS>
 __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_kernel(SinkAttnArgs a) {
   extern __shared__ __align__(16) unsigned char ring[];      // [S][U][key, value][thread] chunks
   constexpr int KPW = 32 / LK, STEP = kRowWarps * KPW;
@@ -163,10 +140,19 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
   }
   int stage = 0;
   for (int k = 0; k < steps; ++k) {
+    const int i0 = first + k * U * STEP;
+    float db[BIAS ? U * RG : 1];
+    if constexpr (BIAS) {
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int n = pos - vis.key_at(min(i0 + u * STEP, iend - 1));
+#pragma unroll
+        for (int r = 0; r < RG; ++r) db[u * RG + r] = r0 + r < Rg ? distance_bias(a, g * Rg + r0 + r, n) : 0.f;
+      }
+    }
     asm volatile("cp.async.wait_group %0;" ::"n"(S - 2) : "memory");
     const AT* cur = slot + stage * U * 2 * kSlots;
     stage = stage + 1 == S ? 0 : stage + 1;
-    const int i0 = first + k * U * STEP;
     float s[U * RG];
 #pragma unroll
     for (int u = 0; u < U; ++u) {
@@ -181,6 +167,10 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
       }
     }
     sum_over_lanes<U * RG, LK>(s, lane);
+    if constexpr (BIAS) {
+#pragma unroll
+      for (int e = 0; e < U * RG; ++e) s[e] = fmaf(db[e], kLog2e, s[e]);
+    }
 #pragma unroll
     for (int u = 0; u < U; ++u)
       if (i0 + u * STEP >= iend) {
@@ -249,7 +239,7 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
     }
     if (a.nsplit == 1) {
       if (a.sink != nullptr) den += exp2f(a.sink[h] * kLog2e - base);       // joins the denominator only: no value
-      stf<AT>((AT*)a.out + (long long)t * a.ld_out + (long long)h * V + d, acc * head_factor<AT>(a, t, h) / den);
+      stf<AT>((AT*)a.out + (long long)t * a.ld_out + (long long)h * V + d, acc * out_factor<AT>(a, t, h, d) / den);
     } else {
       float* pp = a.part + (((long long)t * a.H + h) * a.nsplit + blockIdx.z) * (V + 2);
       pp[2 + d] = acc;
@@ -306,7 +296,7 @@ __global__ void sink_attention_kernel(SinkAttnArgs a) {
       const float* kr = ks + lane * ldk;
       float d = 0.f;
       for (int i = 0; i < D; ++i) d += qh[i] * kr[i];
-      sc = d;
+      sc = d + distance_bias(a, h, pos - vis.key_at(i0 + lane));
     }
     const float nm = fmaxf(m, warp_max(sc));
     const float cf = m == -INFINITY ? 0.f : expf(m - nm);
@@ -329,10 +319,9 @@ __global__ void sink_attention_kernel(SinkAttnArgs a) {
   if (a.nsplit == 1) {
     // the query's own position is always visible: l > 0.  The sink joins the denominator only: exp(sink - m), no value.
     if (a.sink != nullptr) l += expf(a.sink[h] - m);
-    const float f = head_factor<AT>(a, t, h) / l;
     AT* orow = (AT*)a.out + (long long)t * a.ld_out + (long long)h * V;
 #pragma unroll
-    for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) stf<AT>(orow + d, o[i] * f); }
+    for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) stf<AT>(orow + d, o[i] * out_factor<AT>(a, t, h, d) / l); }
   } else {
     float* pp = a.part + (((long long)t * a.H + h) * a.nsplit + blockIdx.z) * (V + 2);
     if (lane == 0) { pp[0] = m; pp[1] = l; }
@@ -361,10 +350,9 @@ __global__ void sink_combine_kernel(SinkAttnArgs a) {
     for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) acc[i] += pz[2 + d] * e; }
   }
   if (a.sink != nullptr) den += expf(a.sink[h] - M);
-  const float f = head_factor<AT>(a, t, h) / den;
   AT* orow = (AT*)a.out + t * a.ld_out + (long long)h * V;
 #pragma unroll
-  for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) stf<AT>(orow + d, acc[i] * f); }
+  for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; if (d < V) stf<AT>(orow + d, acc[i] * out_factor<AT>(a, t, h, d) / den); }
 }
 
 bool vector_form(int D, int V) { return D % 8 == 0 && V % 8 == 0 && D <= 256 && V <= 256; }
@@ -380,7 +368,7 @@ cudaError_t combine(const SinkAttnArgs& a, int T, cudaStream_t s) {
   return last();
 }
 
-template <typename AT, int LK>
+template <typename AT, int LK, bool BIAS>
 cudaError_t rows_form(const SinkAttnArgs& a, int T, cudaStream_t s) {
   const int Rg = a.H / a.G, hp = heads_of(Rg);
   const dim3 grid(T, a.G * ((Rg + hp - 1) / hp), a.nsplit);
@@ -391,9 +379,9 @@ cudaError_t rows_form(const SinkAttnArgs& a, int T, cudaStream_t s) {
     k<<<grid, 32 * kRowWarps, smem, s>>>(a);
     return last();
   };
-  if (hp == 1) return go(sink_rows_kernel<AT, LK, 1, U, S>);
-  if (hp == 2) return go(sink_rows_kernel<AT, LK, 2, U, S>);
-  return go(sink_rows_kernel<AT, LK, 4, U, S>);
+  if (hp == 1) return go(sink_rows_kernel<AT, LK, 1, U, S, BIAS>);
+  if (hp == 2) return go(sink_rows_kernel<AT, LK, 2, U, S, BIAS>);
+  return go(sink_rows_kernel<AT, LK, 4, U, S, BIAS>);
 }
 
 template <typename AT, int NPL>
@@ -406,11 +394,17 @@ cudaError_t general_form(const SinkAttnArgs& a, int T, cudaStream_t s) {
   return last();
 }
 
+template <typename AT, bool BIAS>
+cudaError_t vector_rows(const SinkAttnArgs& a, int T, cudaStream_t s) {
+  const int mx = a.D > a.V ? a.D : a.V;
+  return mx <= 64 ? rows_form<AT, 8, BIAS>(a, T, s) : mx <= 128 ? rows_form<AT, 16, BIAS>(a, T, s) : rows_form<AT, 32, BIAS>(a, T, s);
+}
+
 template <typename AT>
 cudaError_t attention(const SinkAttnArgs& a, int T, cudaStream_t s) {
   cudaError_t e;
-  const int mx = a.D > a.V ? a.D : a.V, npl = (a.V + 31) / 32;
-  if (vector_form(a.D, a.V)) e = mx <= 64 ? rows_form<AT, 8>(a, T, s) : mx <= 128 ? rows_form<AT, 16>(a, T, s) : rows_form<AT, 32>(a, T, s);
+  const int npl = (a.V + 31) / 32;
+  if (vector_form(a.D, a.V)) e = a.slopes != nullptr || a.bias != nullptr ? vector_rows<AT, true>(a, T, s) : vector_rows<AT, false>(a, T, s);
   else e = npl <= 2 ? general_form<AT, 2>(a, T, s) : npl <= 4 ? general_form<AT, 4>(a, T, s) : general_form<AT, 16>(a, T, s);
   if (e == cudaSuccess && a.nsplit > 1) e = combine<AT>(a, T, s);
   return e;

@@ -15,7 +15,10 @@ struct SinkAttnArgs {
   // visible keys j <= p: same block of `block` positions (0: all) and p - j < window (0: all), or j < keep
   int block, window, keep;
   float scale, out_mult;
-  const void* gate; long long ld_gate;      // activation type [T, H]: the head's result times sigmoid(gate) (nullable)
+  // what is added to the score of a key n = p - j tokens back: -slopes[h] n and bias[h * bias_len + min(n, bias_len - 1)] (both nullable)
+  const float* slopes; const float* bias; int bias_len;
+  const void* gate; long long ld_gate;      // activation type: the result times sigmoid(gate) (nullable); one logit per head [T, H] or,
+  bool gate_elem;                           // with gate_elem, per element [T, H V]
   void* out; long long ld_out;              // activation type, row t at out + t * ld_out, head h at column h * V
   int nsplit, chunk;                        // keys split into nsplit parts of `chunk` visible keys
   float* part;                              // [T, H, nsplit, V + 2] = (m, l, o[V]) when nsplit > 1
@@ -27,5 +30,6 @@ int sink_attention_chunk_unit();
 cudaError_t sink_attention_launch(const SinkAttnArgs& a, bool f32, int T, cudaStream_t s);
 // bf16 on the tensor cores, 64 query rows per CTA (context_lens instead of positions; nsplit, chunk, part unused)
 bool sink_flash_supported(int D, int V);
+int sink_flash_bias_max();                  // longest distance table (slopes and a table together: the vector form alone)
 cudaError_t sink_flash_launch(const SinkAttnArgs& a, const int* context_lens, int max_tiles, cudaStream_t s);
 }  // namespace b200

@@ -15,14 +15,16 @@ namespace {
 constexpr int kMaxStreams = 8;
 
 // ---------------------------------------------------------------------------------------------------------- streams
-// xs[t, s, :] = table[ids[t], :] * scale for every stream s
+// xs[t, s, :] = table[ids[t], :] * scale (+ pos[positions[t], :], pos nullable) for every stream s
 template <typename TT>
 __global__ void stream_embed_kernel(const TT* __restrict__ table, long long ld, const long long* __restrict__ ids, float scale, int S, int n,
-                                    float* __restrict__ xs) {
+                                    float* __restrict__ xs, const TT* __restrict__ pos, const int* __restrict__ positions, int n_pos) {
   const long long t = blockIdx.x;
   const TT* row = table + ids[t] * ld;
+  const TT* prow = pos != nullptr ? pos + (long long)min(max(positions[t], 0), n_pos - 1) * n : nullptr;      // (the host admits no position behind the table)
   for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < n; c += gridDim.y * blockDim.x) {
-    const float v = ldf<TT>(row + c) * scale;
+    float v = ldf<TT>(row + c) * scale;
+    if (prow != nullptr) v += ldf<TT>(prow + c);
     for (int s = 0; s < S; ++s) xs[(t * S + s) * n + c] = v;
   }
 }
@@ -408,7 +410,8 @@ __global__ void mingru_scan_kernel(const AT* __restrict__ rows, long long ld, in
 struct PrologueArgs {
   const void* rows; long long ld;           // AT, query heads from column q0 on, keys k0, values v0
   int q0, k0, v0, H, G, D, V;
-  const float* qn; const float* kn;         // [D] norm weights (nullable)
+  const float* qn; const float* kn;         // [D] norm weights, [H D] / [G D] with `whole` (nullable)
+  bool whole;                               // ONE norm over all query (key) heads' entries instead of one per head (before the rotation only)
   float eps;
   const float* inv_freq; int rot;           // angles per position of the rot / 2 pairs
   float rot_mult;                           // factor on cos and sin
@@ -437,18 +440,32 @@ __global__ void qk_norm_rope_append_kernel(PrologueArgs a) {
   __syncthreads();
   const int slot = a.slot_map[t], pg = slot / a.page, off = slot % a.page;
   const AT* r = (const AT*)a.rows + t * a.ld;
+  float inv_q = 1.f, inv_k = 1.f;
+  if (a.whole) {
+    __shared__ float red[32];
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x; i < H * D; i += blockDim.x) { const float v = ldf<AT>(r + a.q0 + i); sq += v * v; }
+    for (int i = threadIdx.x; i < G * D; i += blockDim.x) { const float v = ldf<AT>(r + a.k0 + i); sk += v * v; }
+    inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)(H * D) + a.eps);
+    inv_k = 1.f / sqrtf(block_sum(sk, red) / (float)(G * D) + a.eps);
+  }
   for (int hh = warp; hh < H + G; hh += nw) {
     const bool isq = hh < H;
     const AT* src = isq ? r + a.q0 + hh * D : r + a.k0 + (hh - H) * D;
     const float* w = isq ? a.qn : a.kn;
+    if (a.whole && w != nullptr) w += (isq ? hh : hh - H) * D;
     float v[NPL], inv = 1.f;
 #pragma unroll
     for (int i = 0; i < NPL; ++i) v[i] = lane + 32 * i < D ? ldf<AT>(src + lane + 32 * i) : 0.f;
     auto scale = [&]() {
-      float ss = 0.f;
+      if (a.whole) {
+        inv = isq ? inv_q : inv_k;
+      } else {
+        float ss = 0.f;
 #pragma unroll
-      for (int i = 0; i < NPL; ++i) ss += v[i] * v[i];
-      inv = 1.f / sqrtf(warp_sum(ss) / (float)D + a.eps);
+        for (int i = 0; i < NPL; ++i) ss += v[i] * v[i];
+        inv = 1.f / sqrtf(warp_sum(ss) / (float)D + a.eps);
+      }
 #pragma unroll
       for (int i = 0; i < NPL; ++i) { const int d = lane + 32 * i; v[i] *= w != nullptr && d < D ? inv * w[d] : inv; }
     };
@@ -548,12 +565,11 @@ __global__ void group_softmax_topk_kernel(const float* __restrict__ z, long long
 }  // namespace
 
 // =========================================================================================================== launchers
-cudaError_t stream_embed_launch(const void* table, bool table_f32, long long ld, const long long* ids, float scale, int S, int n, float* xs, int T,
-                                cudaStream_t s) {
+cudaError_t stream_embed_launch(const void* table, bool table_f32, long long ld, const long long* ids, float scale, int S, int n, float* xs, const void* pos,
+                                const int* positions, int n_pos, int T, cudaStream_t s) {
   if (S < 1 || S > kMaxStreams) return cudaErrorInvalidValue;
   dim3 grid(T, (n + 1023) / 1024);
-  if (table_f32) stream_embed_kernel<float><<<grid, 256, 0, s>>>((const float*)table, ld, ids, scale, S, n, xs);
-  else stream_embed_kernel<__nv_bfloat16><<<grid, 256, 0, s>>>((const __nv_bfloat16*)table, ld, ids, scale, S, n, xs);
+  AT_DISPATCH(table_f32, (stream_embed_kernel<AT><<<grid, 256, 0, s>>>((const AT*)table, ld, ids, scale, S, n, xs, (const AT*)pos, positions, n_pos)));
   return last();
 }
 
@@ -657,9 +673,9 @@ static void prologue_t(const PrologueArgs& a, bool half, bool after, int T, cuda
 cudaError_t qk_norm_rope_append_launch(const void* rows, long long ld, int q0, int k0, int v0, int H, int G, int D, int V, const float* qn,
                                        const float* kn, float eps, const float* inv_freq, int rot, const int* positions, const int* slot_map,
                                        int page, float* qout, void* kpool, void* vpool, bool f32, bool half, bool norm_after, float rot_mult,
-                                       const void* v_first, long long ld_vf, float lam, int T, cudaStream_t s) {
-  if (rot % 2 != 0 || rot > D || D > 1024) return cudaErrorInvalidValue;
-  const PrologueArgs a{rows, ld, q0, k0, v0, H, G, D, V, qn, kn, eps, inv_freq, rot, rot_mult, positions, slot_map, page, v_first, ld_vf, lam, qout, kpool, vpool};
+                                       const void* v_first, long long ld_vf, float lam, bool whole, int T, cudaStream_t s) {
+  if (rot % 2 != 0 || rot > D || D > 1024 || (whole && norm_after)) return cudaErrorInvalidValue;
+  const PrologueArgs a{rows, ld, q0, k0, v0, H, G, D, V, qn, kn, whole, eps, inv_freq, rot, rot_mult, positions, slot_map, page, v_first, ld_vf, lam, qout, kpool, vpool};
   if (D <= 64) AT_DISPATCH(f32, (prologue_t<AT, 2>(a, half, norm_after, T, s)));
   else if (D <= 128) AT_DISPATCH(f32, (prologue_t<AT, 4>(a, half, norm_after, T, s)));
   else if (D <= 256) AT_DISPATCH(f32, (prologue_t<AT, 8>(a, half, norm_after, T, s)));

@@ -5,8 +5,9 @@
 #include <cuda_runtime.h>
 
 namespace b200 {
-cudaError_t stream_embed_launch(const void* table, bool table_f32, long long ld, const long long* ids, float scale, int S, int n, float* xs, int T,
-                                cudaStream_t s);
+// pos [n_pos, n] in the table's type, added at positions[t] (nullable)
+cudaError_t stream_embed_launch(const void* table, bool table_f32, long long ld, const long long* ids, float scale, int S, int n, float* xs, const void* pos,
+                                const int* positions, int n_pos, int T, cudaStream_t s);
 // y == nullptr: only the read.  y2, gate, ls nullable.
 cudaError_t hyper_step_launch(float* xs, const float* y, long long ld_y, const float* y2, long long ld_y2, const void* gate, long long ld_g,
                               const float* ls, const float* mix, const float* out_w, float mult, const float* in_w, float alpha, const float* w,
@@ -21,11 +22,11 @@ bool delta_scan_wants_prepare(int N, int max_q);
 long long delta_scan_prepare_width(int G, int H, int N, int P);
 cudaError_t mingru_scan_launch(const void* rows, long long ld, int z0, int x0, int g0, int R, float* state, const int* cu, const int* ctx,
                                const int* slots, float out_mult, void* out, long long ld_out, int B, bool f32, int max_q, cudaStream_t s);
-// qn, kn, v_first nullable
+// qn, kn, v_first nullable; whole: one norm over all query (key) heads' entries, weights [H D] / [G D]
 cudaError_t qk_norm_rope_append_launch(const void* rows, long long ld, int q0, int k0, int v0, int H, int G, int D, int V, const float* qn,
                                        const float* kn, float eps, const float* inv_freq, int rot, const int* positions, const int* slot_map,
                                        int page, float* qout, void* kpool, void* vpool, bool f32, bool half, bool norm_after, float rot_mult,
-                                       const void* v_first, long long ld_vf, float lam, int T, cudaStream_t s);
+                                       const void* v_first, long long ld_vf, float lam, bool whole, int T, cudaStream_t s);
 cudaError_t group_softmax_topk_launch(const float* z, long long ld_z, const float* corr, int E, int top, int ng, int keep, int* idx, float* w, int T,
                                       cudaStream_t s);
 }  // namespace b200

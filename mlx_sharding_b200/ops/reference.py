@@ -359,21 +359,38 @@ def side_gate(gx: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, col0: in
     return (F.gelu(gx.float(), approximate="tanh") * e).to(gx.dtype)
 
 
-def causal_conv_silu(u: torch.Tensor, w: torch.Tensor, b: torch.Tensor, conv_state: torch.Tensor, meta: BatchMeta) -> torch.Tensor:
-    """Per-channel causal convolution + SiLU over a ragged batch.  ``u`` ``[T, C]`` (may be a column view), ``w`` ``[C, K]`` (last
-    column = current token), ``conv_state`` ``[slots, K-1, C]`` = the last ``K-1`` inputs of each sequence (updated here)."""
+def _causal_conv(u: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], conv_state: torch.Tensor, meta: BatchMeta) -> torch.Tensor:
+    """Per-channel causal convolution over a ragged batch, fp32 result (see :func:`causal_conv_silu`)."""
     K = w.shape[1]
-    out = torch.empty(u.shape, dtype=u.dtype, device=u.device)
+    out = torch.empty(u.shape, dtype=torch.float32, device=u.device)
     for s, e, c0, slot in _seq_ranges(meta):
         hist = conv_state[slot].to(u.dtype) if c0 > 0 else torch.zeros(K - 1, u.shape[1], dtype=u.dtype, device=u.device)
         full = torch.cat([hist, u[s:e]])
-        acc = b.float().expand(e - s, -1).clone()
+        acc = torch.zeros(e - s, u.shape[1], device=u.device) if b is None else b.float().expand(e - s, -1).clone()
         for k in range(K):
             acc += full[k:k + e - s].float() * w[:, k].float()
-        out[s:e] = F.silu(acc).to(u.dtype)
-        if K > 1:
+        out[s:e] = acc
+        if K > 1 and e > s:
             conv_state[slot] = full[-(K - 1):].to(conv_state.dtype)
     return out
+
+
+def causal_conv_silu(u: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], conv_state: torch.Tensor, meta: BatchMeta) -> torch.Tensor:
+    """Per-channel causal convolution + SiLU over a ragged batch.  ``u`` ``[T, C]`` (may be a column view), ``w`` ``[C, K]`` (last
+    column = current token), ``b`` ``[C]`` or ``None``, ``conv_state`` ``[slots, K-1, C]`` = the last ``K-1`` inputs of each sequence (updated here)."""
+    return F.silu(_causal_conv(u, w, b, conv_state, meta)).to(u.dtype)
+
+
+def conv_qkv_append(u: torch.Tensor, w: torch.Tensor, conv_state: torch.Tensor, heads: int, dim: int, kpool: torch.Tensor, vpool: torch.Tensor,
+                    meta: BatchMeta) -> torch.Tensor:
+    """Attention prologue of layers whose queries, keys and values pass a short causal convolution (no bias, no activation; arguments as in
+    :func:`causal_conv_silu`).  Columns of ``u``: ``[q: heads*dim | k: G*dim | v: G*dv]``; the convolved keys and values go to the pools
+    ``[pages, G, page, d]`` at ``meta.slot_mapping``.  ``u`` with query columns alone: nothing is appended (the layer reads another layer's
+    pools).  Returns the convolved queries fp32 ``[T, heads, dim]``."""
+    y = _causal_conv(u, w, None, conv_state, meta)
+    if u.shape[1] > heads * dim:
+        paged_kv_append(y, heads * dim, heads * dim + kpool.shape[1] * dim, kpool, vpool, meta)
+    return y[:, :heads * dim].reshape(-1, heads, dim).contiguous()
 
 
 def ssm_scan(xbc: torch.Tensor, dt_raw: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
@@ -417,9 +434,10 @@ def decay_scan(qkv: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, meta
 
 
 def gated_rmsnorm(y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: float, groups: int, mode: str,
-                  out_dtype: torch.dtype) -> torch.Tensor:
-    """``mode='silu_pre'``: RMS norm in ``groups`` equal parts of ``y * silu(gate)``; ``mode='sigmoid_post'``: ``norm(y) * sigmoid(gate)``.
-    Both times ``w``; fp32 arithmetic."""
+                  out_dtype: torch.dtype, out: Optional[torch.Tensor] = None, out_col0: int = 0) -> torch.Tensor:
+    """``mode='silu_pre'``: RMS norm in ``groups`` equal parts of ``y * silu(gate)``; ``mode='sigmoid_post'``: ``norm(y) * sigmoid(gate)``;
+    ``mode='silu_post'``: ``norm(y) * silu(gate)``.  All times ``w``; fp32 arithmetic.  The result goes to ``out[:, out_col0 : out_col0 + C]`` (a
+    fresh tensor by default)."""
     yf, g = y.float(), gate.float()
     if mode == "silu_pre":
         yf = yf * F.silu(g)
@@ -428,7 +446,12 @@ def gated_rmsnorm(y: torch.Tensor, gate: torch.Tensor, w: torch.Tensor, eps: flo
     v = (v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps)).view(T, C) * w.float()
     if mode == "sigmoid_post":
         v = v * torch.sigmoid(g)
-    return v.to(out_dtype)
+    elif mode == "silu_post":
+        v = v * F.silu(g)
+    if out is None:
+        return v.to(out_dtype)
+    out[:, out_col0:out_col0 + C] = v.to(out.dtype)
+    return out
 
 
 def _rot_half(v: torch.Tensor, pos: torch.Tensor, inv_freq: torch.Tensor, mult: float = 1.0) -> torch.Tensor:
@@ -518,11 +541,11 @@ def latent_attention_prefill(q, pool, sink, meta: BatchMeta, scale: float, kv_ra
 def scaled_add_norm_(x: torch.Tensor, y: torch.Tensor, ls: Optional[torch.Tensor], w: torch.Tensor, eps: float, act_dtype: torch.dtype,
                      extra: Optional[torch.Tensor] = None, extra_gate: Optional[torch.Tensor] = None, mult: float = 1.0) -> torch.Tensor:
     """Pre-norm residual step on the fp32 stream ``x`` (in place): ``x += (y + extra * sigmoid(extra_gate)) * ls * mult`` (``ls``: per-channel
-    layer scale or ``None``; ``extra`` / ``extra_gate``: an always-on branch with one gate logit per row; ``mult``: one factor for all
-    channels), then returns ``x / sqrt(mean(x^2) + eps) * w`` in the activation dtype: the input of the sublayer that follows."""
+    layer scale or ``None``; ``extra``: a second branch, with one gate logit per row in ``extra_gate`` or as it is (``None``); ``mult``: one
+    factor for all channels), then returns ``x / sqrt(mean(x^2) + eps) * w`` in the activation dtype: the input of the sublayer that follows."""
     yf = y.float()
     if extra is not None:
-        yf = yf + extra.float() * torch.sigmoid(extra_gate.float()).reshape(-1, 1)
+        yf = yf + (extra.float() if extra_gate is None else extra.float() * torch.sigmoid(extra_gate.float()).reshape(-1, 1))
     if ls is not None:
         yf = yf * ls.float()
     x += yf * mult if mult != 1.0 else yf
@@ -576,12 +599,17 @@ def mlstm_scan(qkv: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, 
     return o.view(T, H * vdim)
 
 
-def sigmoid_topk(z: torch.Tensor, num_experts: int, top: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """Router on fp32 logits ``z[:, :num_experts]``: scores ``sigmoid(z)``, the ``top`` largest (ties: lowest id), weights = the chosen
-    scores as they are.  Returns ``(idx int32 [T, top], w fp32 [T, top])``."""
+def sigmoid_topk(z: torch.Tensor, num_experts: int, top: int, correction: Optional[torch.Tensor] = None, normalise: bool = False,
+                 scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Router on fp32 logits ``z[:, :num_experts]``: scores ``s = sigmoid(z)``; the ``top`` largest ``s + correction`` are chosen (ties: lowest
+    id); weights = the chosen experts' ``s``, divided by their sum ``+ 1e-20`` (``normalise``), times ``scale``.  Returns ``(idx int32 [T, top],
+    w fp32 [T, top])``."""
     sc = torch.sigmoid(z[:, :num_experts].float())
-    order = torch.sort(sc, dim=-1, descending=True, stable=True).indices[:, :top]
-    return order.to(torch.int32), torch.gather(sc, 1, order)
+    order = torch.sort(sc if correction is None else sc + correction.float(), dim=-1, descending=True, stable=True).indices[:, :top]
+    w = torch.gather(sc, 1, order)
+    if normalise:
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return order.to(torch.int32), w * scale if scale != 1.0 else w
 
 
 def clamped_glu(g: torch.Tensor, u: torch.Tensor, limit: float, out_dtype: torch.dtype, row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -600,9 +628,9 @@ def clamped_gated_up(x: torch.Tensor, Wg: LinearWeight, Wu: LinearWeight, limit:
 
 
 def moe_clamped_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight,
-                        limit: float) -> torch.Tensor:
+                        limit: float, on_input: bool = True) -> torch.Tensor:
     """``y[t] = sum_j expert_{idx[t,j]}(w[t,j] x[t])`` with clamped-GLU experts (:func:`clamped_glu`): the router weight scales the
-    expert's INPUT.  Banks ``Wg``, ``Wu`` ``[E, F, K]``, ``Wd`` ``[E, K, F]``.  Returns fp32 ``[T, K]``."""
+    expert's INPUT; ``on_input=False``: its OUTPUT, ``y[t] = sum_j w[t,j] expert_{idx[t,j]}(x[t])``.  Banks ``Wg``, ``Wu`` ``[E, F, K]``, ``Wd`` ``[E, K, F]``.  Returns fp32 ``[T, K]``."""
     T, k = idx.shape
     y = torch.zeros(T, Wd.weight.shape[1], dtype=torch.float32, device=x.device)
     il = idx.long()
@@ -610,9 +638,11 @@ def moe_clamped_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, Wg:
         tok, slot = torch.where(il == e)
         if tok.numel() == 0:
             continue
-        xe = (x[tok].float() * w[tok, slot].float()[:, None]).to(x.dtype)
+        we = w[tok, slot].float()[:, None]
+        xe = (x[tok].float() * we).to(x.dtype) if on_input else x[tok]
         h = clamped_glu(xe.float() @ Wg.weight[e].float().t(), xe.float() @ Wu.weight[e].float().t(), limit, x.dtype)
-        y.index_add_(0, tok, h.float() @ Wd.weight[e].float().t())
+        ye = h.float() @ Wd.weight[e].float().t()
+        y.index_add_(0, tok, ye if on_input else ye * we)
     return y
 
 
@@ -733,9 +763,13 @@ def relu2_(x: torch.Tensor) -> torch.Tensor:
     return x.copy_((torch.relu(x.float()) ** 2).to(x.dtype))
 
 
-def stream_embed(table: torch.Tensor, ids: torch.Tensor, scale: float, streams: int) -> torch.Tensor:
-    """``streams`` equal copies of ``table[ids] * scale``: the fp32 residual streams ``[T, streams, width]`` at the start of a stack."""
+def stream_embed(table: torch.Tensor, ids: torch.Tensor, scale: float, streams: int, pos_table: Optional[torch.Tensor] = None,
+                 positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``streams`` equal copies of ``table[ids] * scale`` (``+ pos_table[positions]``: learned positions): the fp32 residual streams ``[T,
+    streams, width]`` at the start of a stack."""
     x = table[ids.long()].float() * float(scale)
+    if pos_table is not None:
+        x = x + pos_table[positions.long()].float()
     return x[:, None, :].repeat(1, int(streams), 1).contiguous()
 
 
@@ -766,11 +800,11 @@ def hyper_step_(xs: torch.Tensor, y: Optional[torch.Tensor], y2: Optional[torch.
 
 def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, state: torch.Tensor,
                meta: BatchMeta, heads: int, kv_heads: int, dim: int, vdim: int, q_scale: float, unit_eps: float = 1e-6) -> torch.Tensor:
-    """Gated delta rule with one decay per head and key channel (fp32), per head ``h`` with query / key head ``h // (heads / kv_heads)``:
+    """Gated delta rule with one decay per head and key channel, or one per head (fp32), per head ``h`` with query / key head ``h // (heads / kv_heads)``:
     ``q, k`` made unit vectors (``x / sqrt(sum x^2 + unit_eps)``; ``q`` times ``q_scale``), ``b = sigmoid(beta_h)``,
-    ``g = exp(-exp(A_log_h) softplus(dt + dt_bias))`` (``[dim]``), then ``S <- g[:, None] S``, ``u = b (v - S^T k)``, ``S <- S + k u^T``,
+    ``g = exp(-exp(A_log_h) softplus(dt + dt_bias))`` (``[dim]``, or one number where ``dt_bias`` has ``heads`` entries), then ``S <- g[:, None] S``, ``u = b (v - S^T k)``, ``S <- S + k u^T``,
     ``o = S^T q``.  ``qkv`` columns ``[q: kv_heads*dim | k: kv_heads*dim | v: heads*vdim]`` (after the short convolution), ``beta``
-    ``[T, heads]`` raw, ``dt`` ``[T, heads*dim]`` raw; ``state`` ``[slots, heads, dim, vdim]`` fp32.  Returns fp32 ``[T, heads*vdim]``."""
+    ``[T, heads]`` raw, ``dt`` ``[T, heads*dim]`` (``[T, heads]``) raw; ``state`` ``[slots, heads, dim, vdim]`` fp32.  Returns fp32 ``[T, heads*vdim]``."""
     T, H, G, D, V = qkv.shape[0], heads, kv_heads, dim, vdim
     q = qkv[:, :G * D].float().view(T, G, D)
     k = qkv[:, G * D:2 * G * D].float().view(T, G, D)
@@ -778,7 +812,8 @@ def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, dt: torch.Tensor, dt_bias:
     q = (q * torch.rsqrt(q.pow(2).sum(-1, keepdim=True) + unit_eps) * q_scale).repeat_interleave(H // G, 1)
     k = (k * torch.rsqrt(k.pow(2).sum(-1, keepdim=True) + unit_eps)).repeat_interleave(H // G, 1)
     bt = torch.sigmoid(beta[:, :H].float())
-    g = torch.exp(-torch.exp(A_log.float()).view(1, H, 1) * F.softplus(dt[:, :H * D].float() + dt_bias.float(), threshold=30.0).view(T, H, D))
+    n = dt_bias.numel()
+    g = torch.exp(-torch.exp(A_log.float()).view(1, H, 1) * F.softplus(dt[:, :n].float() + dt_bias.float(), threshold=30.0).view(T, H, n // H))
     o = torch.empty(T, H, V, dtype=torch.float32, device=qkv.device)
     for s, e, c0, slot in _seq_ranges(meta):
         if e == s:
@@ -796,11 +831,12 @@ def delta_scan(qkv: torch.Tensor, beta: torch.Tensor, dt: torch.Tensor, dt_bias:
 def qk_norm_rope_append(rows: torch.Tensor, q_col0: int, k_col0: int, v_col0: int, heads: int, dim: int, qn_w: Optional[torch.Tensor],
                         kn_w: Optional[torch.Tensor], eps: float, inv_freq: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, meta: BatchMeta,
                         half: bool = False, norm_after: bool = False, rot_mult: float = 1.0, v_first: Optional[torch.Tensor] = None,
-                        v_lambda: float = 0.0) -> torch.Tensor:
+                        v_lambda: float = 0.0, whole: bool = False) -> torch.Tensor:
     """Attention prologue on a fused projection's rows ``[.. q: heads*dim .. k: G*dim .. v: G*dv ..]``: per head ``x / sqrt(mean(x^2) + eps)
     * w`` on queries and keys (weights ``[dim]`` shared by the heads, or ``None``), and rotation of the first ``2 len(inv_freq)`` entries by
     ``position * inv_freq[i]`` in adjacent pairs ``(2i, 2i+1)`` or (``half``) pairs ``(i, i + len(inv_freq))``, cos and sin times
-    ``rot_mult``; the norm comes before the rotation or (``norm_after``) behind it.  Values: as they are, or ``(1 - v_lambda) v + v_lambda
+    ``rot_mult``; the norm comes before the rotation or (``norm_after``) behind it.  ``whole``: ONE norm over all heads' entries of the
+    query (key) row instead of one per head, weights ``[heads * dim]`` / ``[G * dim]`` (before the rotation).  Values: as they are, or ``(1 - v_lambda) v + v_lambda
     v_first`` with ``v_first`` ``[T, G*dv]``.  Keys and values go to the pools ``[pages, G, page, d]`` at ``meta.slot_mapping``.  Returns
     the queries fp32 ``[T, heads, dim]``."""
     P, G, page, dk = kpool.shape
@@ -818,7 +854,10 @@ def qk_norm_rope_append(rows: torch.Tensor, q_col0: int, k_col0: int, v_col0: in
 
     q = rows[:, q_col0:q_col0 + heads * dim].float().view(T, heads, dim)
     k = rows[:, k_col0:k_col0 + G * dk].float().view(T, G, dk)
-    q, k = (norm(rotate(q), qn_w), norm(rotate(k), kn_w)) if norm_after else (rotate(norm(q, qn_w)), rotate(norm(k, kn_w)))
+    if whole:
+        q, k = (rotate(norm(x.reshape(T, -1), w).view(x.shape)) for x, w in ((q, qn_w), (k, kn_w)))
+    else:
+        q, k = (norm(rotate(q), qn_w), norm(rotate(k), kn_w)) if norm_after else (rotate(norm(q, qn_w)), rotate(norm(k, kn_w)))
     v = rows[:, v_col0:v_col0 + G * dv]
     if v_first is not None:
         v = (1.0 - v_lambda) * v.float() + v_lambda * v_first.float()
@@ -831,13 +870,15 @@ def qk_norm_rope_append(rows: torch.Tensor, q_col0: int, k_col0: int, v_col0: in
 
 def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, sink: Optional[torch.Tensor], meta: BatchMeta, scale: float,
                    block: int = 0, window: int = 0, out_mult: float = 1.0, out_dtype: torch.dtype = torch.float32,
-                   out: Optional[torch.Tensor] = None, out_col0: int = 0, keep_first: int = 0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   out: Optional[torch.Tensor] = None, out_col0: int = 0, keep_first: int = 0, gate: Optional[torch.Tensor] = None,
+                   slopes: Optional[torch.Tensor] = None, dist_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal grouped-query attention over paged keys / values.  ``q`` ``[T, H, d]`` (normed and rotated), pools ``[pages, G, page, d]`` /
     ``[pages, G, page, dv]``; head ``h`` reads key / value head ``h // (H / G)``.  The query at position ``i`` sees keys ``j <= i`` with
     ``floor(j / block) == floor(i / block)`` (``block > 0``: blocks counted from position 0 of the sequence) and ``i - j < window``
     (``window > 0``); the first ``keep_first`` positions of the sequence are visible beside them.  ``p_j = exp(s_j) / (exp(sink_h) + sum
-    exp(s))`` (``sink=None``: the ordinary softmax).  The result times ``out_mult`` and (``gate`` ``[T, H]``: one logit per head) times
-    ``sigmoid(gate)`` goes to ``out[:, out_col0 : out_col0 + H * dv]`` (a fresh ``[T, H * dv]`` tensor by default), which is returned."""
+    exp(s))`` (``sink=None``: the ordinary softmax), scores ``s = q . k * scale - slopes[h] (i - j) + dist_bias[h, min(i - j, L - 1)]`` (``slopes``
+    ``[H]``, ``dist_bias`` ``[H, L]``, both fp32 and optional).  The result times ``out_mult`` and (``gate`` ``[T, H]``: one logit per head, or ``[T, H *
+    dv]``: one per element) times ``sigmoid(gate)`` goes to ``out[:, out_col0 : out_col0 + H * dv]`` (a fresh ``[T, H * dv]`` tensor by default), which is returned."""
     T, H, D = q.shape
     P, G, page, _ = kpool.shape
     dv, rep = vpool.shape[3], H // G
@@ -852,6 +893,11 @@ def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, si
         V = vpool[pg, :, off].float().repeat_interleave(rep, 1)                           # [n, H, dv]
         sc = torch.einsum("thd,nhd->thn", qf[s:e], K) * scale
         qpos = (c0 + torch.arange(e - s, device=q.device))[:, None]
+        back = (qpos - idx[None, :]).clamp(min=0)                                         # [t, n] tokens back
+        if slopes is not None:
+            sc = sc - slopes.float()[None, :, None] * back[:, None, :].float()
+        if dist_bias is not None:
+            sc = sc + dist_bias.float()[:, back.clamp(max=dist_bias.shape[1] - 1)].transpose(0, 1)
         hidden = torch.zeros(e - s, n, dtype=torch.bool, device=q.device)
         if block > 0:
             hidden = hidden | ((idx[None, :] // block) != (qpos // block))
@@ -866,7 +912,7 @@ def sink_attention(q: torch.Tensor, kpool: torch.Tensor, vpool: torch.Tensor, si
             p = torch.softmax(torch.cat([sc, sk], -1), -1)[..., :n]
         res[s:e] = torch.einsum("thn,nhv->thv", p, V)
     if gate is not None:
-        res = res * torch.sigmoid(gate.float())[:, :, None]
+        res = res * torch.sigmoid(gate.float()).view(T, H, -1)
     res = res.view(T, H * dv) * out_mult
     if out is None:
         return res.to(out_dtype)

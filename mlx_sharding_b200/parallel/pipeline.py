@@ -211,6 +211,11 @@ class LocalPipeline:
         return getattr(self.stages[0].kv, "num_slots", 0)
 
     @property
+    def max_positions(self) -> int:
+        """Positions the model has (learned position table); 0: no limit of its own."""
+        return getattr(self.stages[0].model, "max_positions", 0)
+
+    @property
     def h2d_bytes(self) -> int:
         return sum(r.h2d_bytes for r in self.runners)
 

@@ -39,7 +39,7 @@ def synthetic_model_dir(name: str) -> str:
     mlx-community checkpoint), so ``mlx-sharding-api --model synthetic:llama3-8b`` serves a full-size model without a download."""
     import tempfile
 
-    from ..config import deepseek_v2_lite_config, gemma2_9b_config, gifetar_config, gokapel_config, llama3_8b_config, podurax_config
+    from ..config import deepseek_v2_lite_config, gemma2_9b_config, gifetar_config, gokapel_config, llama3_8b_config, lomusun_config, podurax_config
 
     tiny = lambda: dict(model_type="llama", vocab_size=320, hidden_size=64, intermediate_size=128, num_hidden_layers=4,
                         num_attention_heads=4, num_key_value_heads=2, rms_norm_eps=1e-5, rope_theta=10000.0,
@@ -49,9 +49,11 @@ def synthetic_model_dir(name: str) -> str:
                                           block_size=24, gru_width=40)
     tiny_podurax = lambda: podurax_config(width=64, vocab=320, blocks=1, heads=4, kv_heads=2, dim=16, vdim=24, ff=96, window=24, keep_first=3, inner=80,
                                           state=8, dt_rank=5)
+    tiny_lomusun = lambda: lomusun_config(width=64, vocab=320, blocks=1, heads=4, kv_heads=2, dim=16, vdim=24, experts=4, top=2, expert_ff=32, window=24,
+                                          max_positions=2048)
     canned = {"deepseek-v2-lite": deepseek_v2_lite_config, "llama3-8b": llama3_8b_config, "gemma2-9b": gemma2_9b_config,
               "tiny-llama": tiny, "gifetar": gifetar_config, "tiny-gifetar": tiny_gifetar, "gokapel": gokapel_config, "tiny-gokapel": tiny_gokapel,
-              "podurax": podurax_config, "tiny-podurax": tiny_podurax}
+              "podurax": podurax_config, "tiny-podurax": tiny_podurax, "lomusun": lomusun_config, "tiny-lomusun": tiny_lomusun}
     if name not in canned:
         raise FileNotFoundError(f"unknown synthetic model '{name}' (known: {sorted(canned)})")
     d = _SYNTH_DIRS.get(name)
@@ -101,7 +103,7 @@ def key_in_shard(key: str, spec: ShardSpec, tied_embeddings: bool = False, model
     """True if checkpoint tensor ``key`` belongs to stage ``spec`` (half-layer boundaries included)."""
     if "rotary_emb.inv_freq" in key:
         return False
-    if model_type in ("perelorn", "gusolorn", "gifetar", "gokapel", "podurax"):       # keys: embed, side.embed, l<i>.*, final.norm, head (single-stage model: everything or a layer range)
+    if model_type in ("perelorn", "gusolorn", "gifetar", "gokapel", "podurax", "lomusun"):       # keys: embed, pos, side.embed, l<i>.*, final.norm, head (single-stage model: everything or a layer range)
         m = re.match(r"l(\d+)\.", key)
         if m:
             return spec.owns_layer(int(m.group(1)))
@@ -269,6 +271,9 @@ def random_state_dict(cfg: ModelConfig, spec: Optional[ShardSpec] = None, dtype=
         return
     if cfg.model_type == "podurax":
         yield from _podurax_random(cfg, gen, dtype, device, seed)
+        return
+    if cfg.model_type == "lomusun":
+        yield from _lomusun_random(cfg, gen, dtype, device, seed)
         return
     H = cfg.hidden_size
     q = quantization
@@ -652,3 +657,57 @@ def _podurax_random(cfg: ModelConfig, gen, dtype, device, seed: int):
             yield p + "mlp.down", lin(W, F)
     yield "final.norm", vec(W)
     yield "head", lin(cfg.vocab_size, W)
+
+
+def _lomusun_random(cfg: ModelConfig, gen, dtype, device, seed: int, bias_rows: int = 32):
+    """Random-init Lomusun tensors (checkpoint names and shapes of that design: learned positions, RMS norms, attention with whole-row query /
+    key norms, a sink and a gate per element beside a gated delta rule with short convolutions, attention with convolved queries, keys and
+    values, a distance-bias table and a gate per head, per-expert matrices, router with correction; the LM head is the embedding table).
+    ``bias_rows``: rows of the distance tables (a tensor shape, not configuration)."""
+    gen.manual_seed(seed * 1000003 + 59)
+    W = cfg.hidden_size
+    rn = lambda *shape, std=1.0: torch.randn(*shape, generator=gen, device=device, dtype=torch.float32) * std
+    lin = lambda o, i, gain=1.0: (rn(o, i) * gain / (i ** 0.5)).to(dtype)
+    vec = lambda n: (1.0 + 0.1 * rn(n)).to(dtype)
+    small = lambda n, std=0.2: (std * rn(n)).to(dtype)
+    conv = lambda c, k: (0.5 * rn(c, k)).to(dtype)
+    yield "embed", rn(cfg.vocab_size, W, std=0.5).to(dtype)
+    yield "pos", rn(cfg.max_position_embeddings, W, std=0.3).to(dtype)
+    for i, L in enumerate(cfg.layer_specs):
+        p, m, mlp = f"l{i}.", L["mixer"], L["mlp"]
+        yield p + "norm1", vec(W)
+        if L["type"] == "parallel":
+            H, G, D, V = (int(m["left"][k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * V), ("g", H * V)):
+                yield p + "mix.left." + n, lin(rows, W)
+            yield p + "mix.left.q.norm", vec(H * D)
+            yield p + "mix.left.k.norm", vec(G * D)
+            yield p + "mix.left.sink", small(H, 1.0)
+            yield p + "mix.left.o", lin(W, H * V)
+            H, G, D, V, K = (int(m["right"][k]) for k in ("heads", "kv_heads", "dim", "vdim", "conv"))
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * V)):
+                yield p + "mix.right." + n, lin(rows, W)
+                yield p + "mix.right." + n + ".conv", conv(rows, K)
+            for n, rows in (("a", H), ("b", H), ("g", H * V)):
+                yield p + "mix.right." + n, lin(rows, W)
+            yield p + "mix.right.A_log", torch.log(torch.rand(H, generator=gen, device=device) * 1.5 + 0.05).to(dtype)
+            yield p + "mix.right.dt_bias", (rn(H) - 1.0).to(dtype)
+            yield p + "mix.right.norm", vec(V)
+            yield p + "mix.right.o", lin(W, H * V)
+        else:
+            H, G, D, V, K = (int(m[k]) for k in ("heads", "kv_heads", "dim", "vdim", "conv"))
+            for n, rows in (("q", H * D), ("k", G * D), ("v", G * V))[:3 if m.get("kv_from") is None else 1]:
+                yield p + "mix." + n, lin(rows, W)
+                yield p + "mix." + n + ".conv", conv(rows, K)
+            yield p + "mix.rel", rn(bias_rows, H).to(dtype)
+            yield p + "mix.g", lin(H, W)
+            yield p + "mix.o", lin(W, H * V)
+        if mlp:
+            F, E = int(mlp["expert"]["ff"]), int(mlp["router"]["experts"])
+            for e in range(E):
+                yield p + f"mlp.e{e}.gate", lin(F, W)
+                yield p + f"mlp.e{e}.up", lin(F, W)
+                yield p + f"mlp.e{e}.down", lin(W, F)
+            yield p + "mlp.router", lin(E, W, 3.0)
+            yield p + "mlp.correction", small(E, 0.1)
+    yield "final.norm", vec(W)
