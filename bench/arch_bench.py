@@ -1,4 +1,8 @@
-"""Hybrid designs beside the framework's closest existing model.  ``--arch podurax``: Podurax beside Gokapel (the other stack of recurrent
+"""Hybrid designs beside the framework's closest existing model.  ``--arch lomusun``: Lomusun beside Gokapel (the other stack with a gated delta
+rule, attention with a sink beside a recurrence, and routed experts) at equal width, depth, heads and experts, and each of its kernels beside
+the like kernel (delta rule with one decay per head / one per key channel, windowed attention with slopes or a bias table / Podurax's windowed
+attention, convolution into the pools / convolution + SiLU and the prologue, whole-row norms / norms per head, two-branch residual step /
+Podurax's, corrected sigmoid / group-limited softmax router, output-weighted / input-weighted clamped-GLU experts).  ``--arch podurax``: Podurax beside Gokapel (the other stack of recurrent
 layers and attention with a sink over its own key / value pools on an fp32 residual) at equal width, depth, heads and feed-forward, and each
 of its kernels beside the like kernel (selective scan with a step size per channel / Perelorn's selective scan with one per head, attention
 in a window beside kept first tokens with a gate / Gokapel's inside blocks and Llama's paged and flash attention, prologue with value mixing /
@@ -17,7 +21,7 @@ add, clamped-GLU experts / the SwiGLU expert path).  ``--arch perelorn``: Perelo
 about the same weight bytes), random weights, bf16, one GPU: prefill and decode throughput of the whole stack, and the time of each
 new kernel against the HBM roofline (``MEASURED_PEAKS.json``), with the like kernel of the closest model where there is one.
 
-    python bench.py --arch perelorn|gusolorn|gifetar|gokapel [--arch-sizes 1024,2048]        (prints one JSON line per measurement)
+    python bench.py --arch perelorn|gusolorn|gifetar|gokapel|podurax|lomusun [--arch-sizes 1024,2048]        (prints one JSON line per measurement)
 
 Timing: CUDA events on the launching stream, 3 warm-up runs, an L2 flush (256 MiB write) before every timed run, median of 7.
 """
@@ -32,7 +36,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 
-from mlx_sharding_b200.config import deepseek_v2_lite_config, gifetar_config, gokapel_config, gusolorn_config, perelorn_config, podurax_config  # noqa: E402
+from mlx_sharding_b200.config import deepseek_v2_lite_config, gifetar_config, gokapel_config, gusolorn_config, lomusun_config, perelorn_config, podurax_config  # noqa: E402
 from mlx_sharding_b200.ops.meta import BatchMeta  # noqa: E402
 from mlx_sharding_b200.parallel.pipeline import StageExecutor  # noqa: E402
 from mlx_sharding_b200.utils.loader import random_model  # noqa: E402
@@ -571,7 +575,118 @@ def podurax_main(sizes=(1024, 2048)):
         print(json.dumps(dict(bench="arch-kernel", roofline=f"{hbm} GB/s {tag}", **row)), flush=True)
 
 
+def lomusun_kernel_table(width, dev, hbm):
+    """Lomusun's kernels alone at one layer's shapes beside the like kernels; bytes = what the kernel must move.  Decode = 64 sequences at
+    context 2048, prefill = one 2048-token prompt; windows of 1024 positions, distance tables of 32 rows up to 512 tokens back."""
+    from mlx_sharding_b200.models.lomusun import distance_bias
+    from mlx_sharding_b200.ops import b200 as O
+    from mlx_sharding_b200.ops.weights import LinearWeight
+
+    rows = []
+    H, G, D, V, W, WIN = 16, 4, 128, 128, width, 1024
+    bf = torch.bfloat16
+
+    def add(name, ms, nbytes, like=None, flops=None):
+        r = dict(kernel=name, ms=round(ms, 4), gbs=round(nbytes / ms / 1e6, 1), frac_hbm=round(nbytes / ms / 1e6 / hbm, 3))
+        if flops:
+            r["tflops"] = round(flops / ms / 1e9, 1)
+        if like:
+            r["like_kernel"] = like
+        rows.append(r)
+
+    for phase, B, q, ctx0 in (("decode", 64, 1, 2047), ("prefill", 1, 2048, 0)):
+        meta, _ = step_meta(B, q, ctx0, dev, True)
+        T, npg = B * q, 1 + B * ((ctx0 + q + PS - 1) // PS)
+        rn = lambda *s: torch.randn(*s, device=dev)
+        # ---- gated delta rule: state [slots, H, D, V] fp32 read and written once per step
+        st, C = torch.zeros(B + 1, H, D, V, device=dev), 2 * H * D + H * V
+        qkv, beta = rn(T, C).to(bf), rn(T, H).to(bf)
+        dt1, db1, alog = rn(T, H).to(bf), rn(H) - 1.0, torch.log(torch.rand(H, device=dev) + 0.1)
+        dtn, dbn = rn(T, H * D), rn(H * D) - 1.0
+        sbytes = (2 * B * H * D * V * 4 if q == 1 else 0) + T * C * 2 + T * H * V * 4
+        name = f"delta_scan(one decay per head) {phase}"
+        add(name, timed(lambda: O.delta_scan(qkv, beta, dt1, db1, alog, st, meta, H, H, D, V, D ** -0.5)), sbytes)
+        add(f"delta_scan(decay per key channel) (Gokapel) {phase}", timed(lambda: O.delta_scan(qkv, beta, dtn, dbn, alog, st, meta, H, H, D, V, D ** -0.5)),
+            sbytes + T * H * D * 4, like=name)
+        y, gate, gw = rn(T, H * V), rn(T, H * V).to(bf), torch.ones(H * V, device=dev)
+        name = f"gated_rmsnorm(silu behind the norm) {phase}"
+        add(name, timed(lambda: O.gated_rmsnorm(y, gate, gw, 1e-6, H, "silu_post", bf)), T * H * V * (4 + 2 + 2))
+        add(f"gated_rmsnorm(sigmoid) (Gokapel) {phase}", timed(lambda: O.gated_rmsnorm(y, gate, gw, 1e-6, H, "sigmoid_post", bf)), T * H * V * (4 + 2 + 2), like=name)
+        cw, cst = rn(C, 4), torch.zeros(B + 1, 3, C, device=dev).to(bf)
+        add(f"causal_conv_silu (shared) {phase}", timed(lambda: O.causal_conv_silu(qkv, cw, None, cst, meta)), T * C * 4 + (2 * B * 3 * C * 2 if q == 1 else 0))
+        # ---- attention
+        kp, vp = rn(npg, G, PS, D).to(bf), rn(npg, G, PS, V).to(bf)
+        C2 = (H + G) * D + G * V
+        rows_, cw2, cst2 = rn(T, C2 + H * V).to(bf), rn(C2, 3), torch.zeros(B + 1, 2, C2, device=dev).to(bf)
+        pbytes = T * C2 * 2 + T * H * D * 4 + T * G * (D + V) * 2
+        name = f"conv_qkv_append {phase}"
+        add(name, timed(lambda: O.conv_qkv_append(rows_[:, :C2], cw2, cst2, H, D, kp, vp, meta)), pbytes + (2 * B * 2 * C2 * 2 if q == 1 else 0))
+        qn, kn, qn1, none = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev), torch.ones(D, device=dev), torch.zeros(0, device=dev)
+        inv = (10000.0 ** (-2.0 * torch.arange(D // 4, dtype=torch.float64) / (D // 2))).float().to(dev)
+        whole = lambda: O.qk_norm_rope_append(rows_, 0, H * D, (H + G) * D, H, D, qn, kn, 1e-6, none, kp, vp, meta, whole=True)
+        qf = whole()
+        add(f"qk_norm_rope_append(whole rows) {phase}", timed(whole), pbytes)
+        ms = timed(lambda: O.qk_norm_rope_append(rows_, 0, H * D, (H + G) * D, H, D, qn1, qn1, 1e-6, inv, kp, vp, meta))
+        add(f"qk_norm_rope_append(per head, rotation) (Gokapel) {phase}", ms, pbytes, like=f"qk_norm_rope_append(whole rows) {phase}")
+        n_of = lambda p: min(p + 1, WIN)
+        flops = 2 * H * (D + V) * (B * n_of(ctx0) if q == 1 else sum(n_of(p) for p in range(q)))
+        abytes = (B * n_of(ctx0) * G * (D + V) * 2 if q == 1 else q * G * (D + V) * 2) + T * H * (D * 4 + V * 2)
+        sink, slopes = rn(H), torch.tensor([2.0 ** (-8.0 * (h + 1) / H) for h in range(H)], device=dev)
+        table, eg, hg = distance_bias(rn(32, H).cpu(), 512).to(dev), rows_[:, C2:], rows_[:, C2:C2 + H]
+        first = f"sink_attention(window {WIN}, slopes, sink, gate per element) {phase}"
+        add(first, timed(lambda: O.sink_attention(qf, kp, vp, sink, meta, D ** -0.5, 0, WIN, 0.7, bf, gate=eg, slopes=slopes)), abytes + T * H * V * 2, flops=flops)
+        second = f"sink_attention(window {WIN}, distance table, gate per head) {phase}"
+        add(second, timed(lambda: O.sink_attention(qf, kp, vp, None, meta, D ** -0.5, 0, WIN, 1.0, bf, gate=hg, dist_bias=table)), abytes, flops=flops)
+        ms = timed(lambda: O.sink_attention(qf, kp, vp, sink, meta, D ** -0.5, 0, WIN, 1.0, bf, gate=hg))
+        add(f"sink_attention(window {WIN}, gate per head) (Podurax) {phase}", ms, abytes, like=f"{first} and {second}", flops=flops)
+        # ---- residual step, embedding, router, experts
+        x, y1, y2, nw = rn(T, W), rn(T, W), rn(T, W), torch.ones(W, device=dev)
+        name = f"scaled_add_norm_(two branches) {phase}"
+        add(name, timed(lambda: O.scaled_add_norm_(x, y1, None, nw, 1e-6, bf, extra=y2)), T * W * (4 * 4 + 2))
+        add(f"scaled_add_norm_(one branch) (Podurax) {phase}", timed(lambda: O.scaled_add_norm_(x, y1, None, nw, 1e-6, bf, mult=0.5)), T * W * (4 * 3 + 2), like=name)
+        emb, pos, ids = rn(32000, W).to(bf), rn(4096, W).to(bf), torch.randint(0, 32000, (T,), device=dev)
+        name = f"stream_embed(+ positions) {phase}"
+        add(name, timed(lambda: O.stream_embed(emb, ids, 1.0, 1, pos, meta.positions)), T * W * (2 + 2 + 4))
+        add(f"stream_embed (Podurax) {phase}", timed(lambda: O.stream_embed(emb, ids, 1.0, 1)), T * W * (2 + 4), like=name)
+        E, F, k = 16, W // 2, 2
+        xa, rw, corr = rn(T, W).to(bf), rn(E, W), 0.1 * rn(E)
+        add(f"router_logits (shared) {phase}", timed(lambda: O.router_logits(xa, rw)), T * W * 2 + E * W * 4 + T * E * 4)
+        z = O.router_logits(xa, rw)
+        name = f"sigmoid_topk(correction, normalised) {phase}"
+        add(name, timed(lambda: O.sigmoid_topk(z, E, k, corr, True, 1.5)), T * E * 4 + T * k * 8)
+        add(f"group_softmax_topk (Gokapel) {phase}", timed(lambda: O.group_softmax_topk(z, corr, E, k, 4, 2)), T * E * 4 + T * k * 8, like=name)
+        idx, wts = O.sigmoid_topk(z, E, k, corr, True, 1.5)
+        wg, wu = (LinearWeight(weight=(rn(E, F, W) * W ** -0.5).to(bf)) for _ in range(2))
+        wd = LinearWeight(weight=(rn(E, W, F) * F ** -0.5).to(bf))
+        ebytes = min(E, T * k) * 3 * F * W * 2 + T * W * (2 + 4) + T * k * (2 * W * 2 + 2 * F * 2 + 2 * W * 4)
+        name = f"moe_clamped_experts(weight on the output) {phase}"
+        add(name, timed(lambda: O.moe_clamped_experts(xa, idx, wts, wg, wu, wd, 7.0, on_input=False)), ebytes, flops=6 * T * k * F * W)
+        add(f"moe_clamped_experts(weight on the input) (Gusolorn) {phase}", timed(lambda: O.moe_clamped_experts(xa, idx, wts, wg, wu, wd, 7.0)), ebytes, like=name, flops=6 * T * k * F * W)
+        for nm, n_, k_ in (("mixer in projection", H * D + G * (D + V) + H * V + C + H * V + 2 * H, W), ("mixer out projection", W, 2 * H * V), ("LM head", 32000, W)):
+            w_, x_ = LinearWeight(weight=(rn(n_, k_) * k_ ** -0.5).to(bf)), rn(T, k_).to(bf)
+            add(f"linear_any {nm} {n_}x{k_} {phase}", timed(lambda: O.linear_any(x_, w_, bf)), n_ * k_ * 2 + T * (n_ + k_) * 2, flops=2 * T * n_ * k_)
+    return rows
+
+
+def lomusun_main(sizes=(1024, 2048)):
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    hbm, tag = peaks()
+    for width in sizes:
+        for name, cfg in (("lomusun", lomusun_config(width=width, vocab=32000, blocks=2, heads=16, kv_heads=4, experts=16, top=2, expert_ff=width // 2)),
+                          ("gokapel", gokapel_config(width=width, vocab=32000, blocks=2, heads=16, kv_heads=4, ff=4 * width, experts=16, top=2, expert_ff=width // 2))):
+            m = random_model(cfg, dtype=torch.bfloat16, device=dev, seed=1)
+            r = model_runs(name, m, 32, 1024, 2048, dev, True)
+            print(json.dumps(dict(bench="arch", model=name, width=width, layers=len(cfg["layers"]), **{k: (round(v, 3) if isinstance(v, float) else v) for k, v in r.items()})), flush=True)
+            del m
+            torch.cuda.empty_cache()
+    for row in lomusun_kernel_table(sizes[-1], dev, hbm):
+        print(json.dumps(dict(bench="arch-kernel", roofline=f"{hbm} GB/s {tag}", **row)), flush=True)
+
+
 def main(sizes=(1024, 2048), arch="perelorn"):
+    if arch == "lomusun":
+        return lomusun_main(sizes)
     if arch == "podurax":
         return podurax_main(sizes)
     if arch == "gokapel":

@@ -663,7 +663,7 @@ def _lomusun_random(cfg: ModelConfig, gen, dtype, device, seed: int, bias_rows: 
     """Random-init Lomusun tensors (checkpoint names and shapes of that design: learned positions, RMS norms, attention with whole-row query /
     key norms, a sink and a gate per element beside a gated delta rule with short convolutions, attention with convolved queries, keys and
     values, a distance-bias table and a gate per head, per-expert matrices, router with correction; the LM head is the embedding table).
-    ``bias_rows``: rows of the distance tables (a tensor shape, not configuration)."""
+    ``bias_rows``: most rows of a distance table (a tensor shape, not configuration)."""
     gen.manual_seed(seed * 1000003 + 59)
     W = cfg.hidden_size
     rn = lambda *shape, std=1.0: torch.randn(*shape, generator=gen, device=device, dtype=torch.float32) * std
@@ -699,7 +699,7 @@ def _lomusun_random(cfg: ModelConfig, gen, dtype, device, seed: int, bias_rows: 
             for n, rows in (("q", H * D), ("k", G * D), ("v", G * V))[:3 if m.get("kv_from") is None else 1]:
                 yield p + "mix." + n, lin(rows, W)
                 yield p + "mix." + n + ".conv", conv(rows, K)
-            yield p + "mix.rel", rn(bias_rows, H).to(dtype)
+            yield p + "mix.rel", rn(max(2, min(bias_rows, int(m["bias_max"]))), H).to(dtype)
             yield p + "mix.g", lin(H, W)
             yield p + "mix.o", lin(W, H * V)
         if mlp:
