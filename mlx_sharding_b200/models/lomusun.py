@@ -180,13 +180,19 @@ class LomusunStage(HybridStage):
         u = O.linear_any(ha, w["proj"], self.dtype)                            # [lq | lk | lv | lg | qkv | a | b | g]
         padded = w["o_split"] != H * V or w["o_cols"] - w["o_split"] != h * v
         both = (torch.zeros if padded else torch.empty)(ha.shape[0], w["o_cols"], dtype=self.dtype, device=u.device)
+
+        def delta():
+            qkv = O.causal_conv_silu(self._cols(u, seg, "qkv"), w["conv"], None, st["conv"], meta)
+            o = O.delta_scan(qkv, self._cols(u, seg, "b"), self._cols(u, seg, "a"), w["dt_bias"], w["A_log"], st["S"], meta, h, g, d, v, float(d) ** -0.5,
+                             self.UNIT_EPS)
+            O.gated_rmsnorm(o, self._cols(u, seg, "g"), w["gnorm"], eps, h, "silu_post", self.dtype, both, w["o_split"])
+
+        join = O.run_aside(delta, 1)                                           # beside the attention: they meet in the output product
         q = O.qk_norm_rope_append(u, seg["lq"][0], seg["lk"][0], seg["lv"][0], H, D, w["qn"], w["kn"], eps, self.rope.inv_freq, kpool, vpool, meta, whole=True)
         O.sink_attention(q, kpool, vpool, w["sink"], meta, float(a["scale"]), 0, int((a.get("mask") or {}).get("size", 0) or 0),
                          float(m.get("left_scale", 1.0)), self.dtype, both, 0, gate=self._cols(u, seg, "lg"), slopes=w["slopes"])
-        qkv = O.causal_conv_silu(self._cols(u, seg, "qkv"), w["conv"], None, st["conv"], meta)
-        o = O.delta_scan(qkv, self._cols(u, seg, "b"), self._cols(u, seg, "a"), w["dt_bias"], w["A_log"], st["S"], meta, h, g, d, v, float(d) ** -0.5,
-                         self.UNIT_EPS)
-        O.gated_rmsnorm(o, self._cols(u, seg, "g"), w["gnorm"], eps, h, "silu_post", self.dtype, both, w["o_split"])
+        if join is not None:
+            join.wait()
         return self._mm(both, w["o"], True)
 
     def _attention(self, w, m, ha, meta, kpool, vpool, st):
@@ -197,10 +203,10 @@ class LomusunStage(HybridStage):
                              gate=self._cols(u, seg, "g"), dist_bias=w["bias"])
         return self._mm(o, w["o"], True)
 
-    def _experts(self, w, mlp, ha):
+    def _experts(self, w, mlp, ha, out):
         O, r = self.ops, mlp["router"]
-        idx, wts = O.sigmoid_topk(O.router_logits(ha, w["router"]), int(r["experts"]), int(r["top"]), w["correction"], True, float(r.get("scale", 1.0)))
-        return O.moe_clamped_experts(ha, idx, wts, w["e_gate"], w["e_up"], w["e_down"], float(mlp["expert"]["limit"]), on_input=False)
+        idx, wts = O.sigmoid_router(ha, w["router"], int(r["experts"]), int(r["top"]), w["correction"], True, float(r.get("scale", 1.0)))
+        O.moe_clamped_experts(ha, idx, wts, w["e_gate"], w["e_up"], w["e_down"], float(mlp["expert"]["limit"]), on_input=False, out=out)
 
     @torch.inference_mode()
     def forward(self, x, meta: BatchMeta, kv, all_logits: bool = False, layer_out=None):
@@ -215,8 +221,13 @@ class LomusunStage(HybridStage):
         for i, L in enumerate(self.specs):
             w = self.layer_weights[i]
             mixer = self._parallel if L["type"] == "parallel" else self._attention
+            ye, join = None, None
+            if L["mlp"]:
+                ye = torch.empty_like(h)
+                join = O.run_aside(lambda: self._experts(w, L["mlp"], ha, ye))  # beside the mixer: they meet in the residual
             y = mixer(w, L["mixer"], ha, meta, kv.k[i], kv.v[i], kv.state[i])
-            ye = self._experts(w, L["mlp"], ha) if L["mlp"] else None
+            if join is not None:
+                join.wait()
             nxt = self.layer_weights[i + 1]["norm1"] if i + 1 < n else self.norm_w
             ha = O.scaled_add_norm_(h, y, None, nxt, c.rms_norm_eps, self.dtype, extra=ye)
             if layer_out is not None:

@@ -211,15 +211,17 @@ class _Join:
 _side_streams = {}
 
 
-def run_aside(fn) -> _Join:
-    """Run ``fn()`` on this device's side stream, forked from the current stream (event record / wait, so it is also legal
+def run_aside(fn, lane: int = 0) -> _Join:
+    """Run ``fn()`` on this device's side stream (``lane``: which of them), forked from the current stream (event record / wait, so it is also legal
     inside CUDA-graph capture and becomes a parallel branch of the graph).  Used to run the shared-expert GEMMs of a
     DeepSeek MoE block concurrently with the router / permutation / expert all-to-all, which do not depend on them.
-    ``fn`` must write its result into a tensor allocated *before* the fork."""
+    ``fn`` must write its result into a tensor allocated *before* the fork.  Split-K products share one workspace: keep them on one
+    stream."""
     cur = torch.cuda.current_stream()
-    side = _side_streams.get(cur.device.index)
+    key = (cur.device.index, lane) if lane else cur.device.index
+    side = _side_streams.get(key)
     if side is None:
-        side = _side_streams[cur.device.index] = torch.cuda.Stream(device=cur.device)
+        side = _side_streams[key] = torch.cuda.Stream(device=cur.device)
     fork = torch.cuda.Event()
     fork.record(cur)
     side.wait_event(fork)
@@ -631,6 +633,17 @@ def sigmoid_topk(z, num_experts: int, top: int, correction=None, normalise: bool
     return idx, w
 
 
+ROUTER_MAX_SMEM = 200 * 1024      # token rows that the fused router stages in shared memory
+
+
+def sigmoid_router(x, w, num_experts: int, top: int, correction=None, normalise: bool = False, scale: float = 1.0):
+    """Router product in fp32 and :func:`sigmoid_topk` in one kernel; rows too wide for its shared memory: the two ops."""
+    if (x.shape[1] + num_experts) * 4 + 64 > ROUTER_MAX_SMEM or x.shape[1] % 4 != 0 or x.stride(0) % 4 != 0:
+        return sigmoid_topk(router_logits(x, w), num_experts, top, correction, normalise, scale)
+    idx, wts = C().hy_sigmoid_router(x, w, correction, int(num_experts), int(top), bool(normalise), float(scale))
+    return idx, wts
+
+
 def softmax_topk(z, bias, num_experts: int, top: int):
     idx, w = C().hy_sigmoid_topk(z, int(num_experts), int(top), 1, bias)
     return idx, w
@@ -658,8 +671,8 @@ def clamped_gated_up(x, Wg: LinearWeight, Wu: LinearWeight, limit: float):
     return C().hy_clamped_glu(lin(x, Wg.weight), lin(x, Wu.weight), float(limit), None, None)
 
 
-def moe_clamped_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, on_input: bool = True):
-    return _moe_experts(x, idx, w, Wg, Wu, Wd, float(limit), 0, on_input)
+def moe_clamped_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, on_input: bool = True, out=None):
+    return _moe_experts(x, idx, w, Wg, Wu, Wd, float(limit), 0, on_input, out)
 
 
 def moe_glu_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight):
@@ -672,7 +685,7 @@ def silu_glu(g, u, out_dtype=None, row_scale=None):
     return C().hy_clamped_glu(g, u, 0.0, None, row_scale, 1)
 
 
-def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, kind: int, on_input: bool = False):
+def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight, limit: float, kind: int, on_input: bool = False, out=None):
     """``kind`` 0: routed clamped-GLU experts, ``kind`` 1: SiLU-GLU experts; the router weight scales the expert's input (``on_input``) or its output.  bf16 banks whose sizes fit the grouped tcgen05 GEMM
     (expert rows multiples of 128, inner sizes multiples of 8): counting-sort permutation that scales each gathered row by its pair's
     weight -> grouped two-weight GEMM with the clamped GLU in its epilogue -> grouped down GEMM (fp32) -> sum per token.  Exact mode
@@ -691,14 +704,14 @@ def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight
         else:
             h = c.grouped_linear(xp, wg, wu, offs, T, ACT_IDS["silu"], False)
         y = c.grouped_linear(h, wd, None, offs, T, 0, True)
-        return c.hy_gather_sum(y, pair_row, int(k), out_wts)
+        return c.hy_gather_sum(y, pair_row, int(k), out_wts, out)
     R = T * k
     if R <= PAIR_KERNEL_MAX_ROWS or torch.cuda.is_current_stream_capturing():
         ids = idx.reshape(-1).contiguous()
         h = c.hy_clamped_glu(c.hy_expert_rows_linear(x, int(k), wg, ids, False), c.hy_expert_rows_linear(x, int(k), wu, ids, False),
                              float(limit), None, in_scale, kind)
         y = c.hy_expert_rows_linear(h, 1, wd, ids, True)
-        return c.hy_gather_sum(y, None, int(k), out_wts)
+        return c.hy_gather_sum(y, None, int(k), out_wts, out)
     flat = idx.reshape(-1).long()
     order = torch.sort(flat, stable=True).indices
     pair_row = torch.empty_like(order, dtype=torch.int32)
@@ -719,7 +732,7 @@ def _moe_experts(x, idx, w, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight
         if n:
             y[r0:r0 + n] = torch.matmul(h[r0:r0 + n], wd[e].t()).float()
         r0 += n
-    return c.hy_gather_sum(y, pair_row, int(k), out_wts)
+    return c.hy_gather_sum(y, pair_row, int(k), out_wts, out)
 
 
 PAIR_KERNEL_MAX_ROWS = 64

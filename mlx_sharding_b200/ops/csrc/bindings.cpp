@@ -1083,6 +1083,21 @@ std::vector<Tensor> hy_sigmoid_topk(const Tensor& z, int64_t E, int64_t top, int
   return {idx, w};
 }
 
+std::vector<Tensor> hy_sigmoid_router(const Tensor& x, const Tensor& w, const c10::optional<Tensor>& bias, int64_t E, int64_t top, bool normalise, double scale) {
+  check_act(x, "x"); check_rows(x, "x"); check_f32c(w, "w");
+  TORCH_CHECK(w.dim() == 2 && w.size(0) >= E && w.size(1) == x.size(1) && top >= 1 && top <= E && x.size(1) % 4 == 0 && x.stride(0) % 4 == 0 &&
+              reinterpret_cast<uintptr_t>(x.data_ptr()) % (4 * x.element_size()) == 0 && reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0,
+              "router: rows of a multiple of 4, aligned to 4 entries");
+  if (bias.has_value()) { check_f32c(*bias, "bias"); TORCH_CHECK(bias->numel() >= E); }
+  const c10::cuda::CUDAGuard guard(x.device());
+  const int64_t T = x.size(0);
+  Tensor idx = torch::empty({T, top}, x.options().dtype(torch::kInt32)), wt = torch::empty({T, top}, x.options().dtype(torch::kFloat32));
+  if (T == 0) return {idx, wt};
+  LAUNCH_OK(b200::sigmoid_router_launch(x.data_ptr(), x.stride(0), w.data_ptr<float>(), bias.has_value() ? bias->data_ptr<float>() : nullptr, (int)x.size(1), (int)E, (int)top,
+                                        normalise, (float)scale, idx.data_ptr<int>(), wt.data_ptr<float>(), is_f32(x), (int)T, cur_stream()));
+  return {idx, wt};
+}
+
 // row_of / scale (both optional, one entry per processed row): block i handles row row_of[i] of g and u with scale[i]
 Tensor hy_clamped_glu(const Tensor& g, const Tensor& u, double limit, const c10::optional<Tensor>& row_of, const c10::optional<Tensor>& scale,
                       int64_t kind) {
@@ -1115,7 +1130,7 @@ Tensor hy_expert_rows_linear(const Tensor& x, int64_t div, const Tensor& W, cons
   return out;
 }
 
-Tensor hy_gather_sum(const Tensor& y, const c10::optional<Tensor>& row_of, int64_t k, const c10::optional<Tensor>& wts) {
+Tensor hy_gather_sum(const Tensor& y, const c10::optional<Tensor>& row_of, int64_t k, const c10::optional<Tensor>& wts, const c10::optional<Tensor>& out_) {
   check_f32c(y, "y");
   if (row_of.has_value()) check_i32(*row_of, "row_of");
   const int64_t pairs = row_of.has_value() ? row_of->numel() : y.size(0);
@@ -1123,7 +1138,9 @@ Tensor hy_gather_sum(const Tensor& y, const c10::optional<Tensor>& row_of, int64
   if (wts.has_value()) { check_f32c(*wts, "wts"); TORCH_CHECK(wts->numel() == pairs); }
   const c10::cuda::CUDAGuard guard(y.device());
   const int64_t T = pairs / k;
-  Tensor out = torch::empty({T, y.size(1)}, y.options());
+  Tensor out = out_.has_value() ? *out_ : torch::empty({T, y.size(1)}, y.options());
+  check_f32c(out, "out");
+  TORCH_CHECK(out.dim() == 2 && out.size(0) == T && out.size(1) == y.size(1));
   if (T == 0) return out;
   LAUNCH_OK(b200::gather_sum_launch(y.data_ptr<float>(), row_of.has_value() ? row_of->data_ptr<int>() : nullptr, wts.has_value() ? wts->data_ptr<float>() : nullptr,
                                     (int)k, (int)y.size(1), out.data_ptr<float>(), (int)T, cur_stream()));
@@ -1435,6 +1452,8 @@ Tensor hy_sink_attention(const Tensor& q, const Tensor& kpool, const Tensor& vpo
     nsplit = (span + chunk - 1) / chunk;
     if (nsplit > 1) { a.nsplit = (int)nsplit; a.chunk = (int)chunk; }
   }
+  a.bias_keys = (int)std::min<int64_t>(span, a.chunk);
+  if (a.bias_keys > b200::sink_attention_bias_keys() || (a.slopes == nullptr && a.bias == nullptr)) a.bias_keys = 0;
   Tensor part;
   if (a.nsplit > 1) { part = torch::empty({T * H * a.nsplit * (V + 2)}, q.options()); a.part = part.data_ptr<float>(); }
   LAUNCH_OK(b200::sink_attention_launch(a, is_f32(kpool), (int)T, cur_stream()));
@@ -1595,7 +1614,8 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("normalise") = false, py::arg("scale") = 1.0);
   m.def("hy_clamped_glu", &hy_clamped_glu, py::arg("gate"), py::arg("up"), py::arg("limit"), py::arg("row_of") = py::none(), py::arg("scale") = py::none(),
         py::arg("kind") = 0);
-  m.def("hy_gather_sum", &hy_gather_sum, py::arg("y"), py::arg("row_of"), py::arg("k"), py::arg("wts") = py::none());
+  m.def("hy_gather_sum", &hy_gather_sum, py::arg("y"), py::arg("row_of"), py::arg("k"), py::arg("wts") = py::none(), py::arg("out") = py::none());
+  m.def("hy_sigmoid_router", &hy_sigmoid_router);
   m.def("hy_expert_rows_linear", &hy_expert_rows_linear);
   m.def("hy_layernorm_cast", &hy_layernorm_cast);
   m.def("hy_post_layernorm_add_norm_", &hy_post_layernorm_add_norm_);

@@ -769,12 +769,10 @@ __global__ void mlstm_scan_kernel(MlstmArgs a, int PB, int R, int kTok) {
 // Router on fp32 logits, the `top` largest scores (ties: lowest id).  One warp per token.  mode 0: choice by sigmoid(z) + bias, weights = the
 // chosen experts' sigmoid(z), divided by their sum + 1e-20 (normalise), times `scale`; mode 1: choice by z + bias, weights = softmax over the
 // chosen ones alone.  bias nullable.
-__global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z, const float* __restrict__ bias, int mode, int E, int top,
-                                    int* __restrict__ idx, float* __restrict__ w, bool normalise, float scale) {
-  extern __shared__ float sc[];             // [E]
-  const long long t = blockIdx.x;
-  const int lane = threadIdx.x;
-  for (int e = lane; e < E; e += 32) sc[e] = (mode == 0 ? sigmoid_f(z[t * ld_z + e]) : z[t * ld_z + e]) + (bias != nullptr ? bias[e] : 0.f);
+// One warp; z: the token's logits, sc: E floats of scratch, idx / w: the token's `top` entries.
+__device__ __forceinline__ void topk_of_row(const float* z, float* sc, const float* bias, int mode, int E, int top, int* idx, float* w, bool normalise, float scale) {
+  const int lane = threadIdx.x & 31;
+  for (int e = lane; e < E; e += 32) sc[e] = (mode == 0 ? sigmoid_f(z[e]) : z[e]) + (bias != nullptr ? bias[e] : 0.f);
   __syncwarp();
   float sum = 0.f;
   for (int j = 0; j < top; ++j) {
@@ -787,20 +785,64 @@ __global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z,
       if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
     }
     if (lane == 0) {
-      const float v = mode == 0 && bias != nullptr ? sigmoid_f(z[t * ld_z + bi]) : best;
-      idx[t * top + j] = bi; w[t * top + j] = v * scale; sc[bi] = -INFINITY;
+      const float v = mode == 0 && bias != nullptr ? sigmoid_f(z[bi]) : best;
+      idx[j] = bi; w[j] = v * scale; sc[bi] = -INFINITY;
       sum += v;
     }
     __syncwarp();
   }
   if (mode == 0 && normalise && lane == 0)
-    for (int j = 0; j < top; ++j) w[t * top + j] /= sum + 1e-20f;
+    for (int j = 0; j < top; ++j) w[j] /= sum + 1e-20f;
   if (mode == 1 && lane == 0) {             // the first chosen score is the largest
-    const float m = w[t * top];
+    const float m = w[0];
     sum = 0.f;
-    for (int j = 0; j < top; ++j) sum += expf(w[t * top + j] - m);
-    for (int j = 0; j < top; ++j) w[t * top + j] = expf(w[t * top + j] - m) / sum;
+    for (int j = 0; j < top; ++j) sum += expf(w[j] - m);
+    for (int j = 0; j < top; ++j) w[j] = expf(w[j] - m) / sum;
   }
+}
+
+__global__ void sigmoid_topk_kernel(const float* __restrict__ z, long long ld_z, const float* __restrict__ bias, int mode, int E, int top,
+                                    int* __restrict__ idx, float* __restrict__ w, bool normalise, float scale) {
+  extern __shared__ float sc[];             // [E]
+  const long long t = blockIdx.x;
+  topk_of_row(z + t * ld_z, sc, bias, mode, E, top, idx + t * top, w + t * top, normalise, scale);
+}
+
+// Router product and choice (mode 0) in one kernel: TB token rows in shared memory as floats, the experts' fp32 weight rows spread over the 8
+// warps, then one warp per token chooses (rows a multiple of 4 wide and aligned to 4 entries).            grid ceil(T / TB), block 256
+template <typename AT, int TB>
+__global__ void __launch_bounds__(256) sigmoid_router_kernel(const AT* __restrict__ x, long long ld_x, const float* __restrict__ w, const float* __restrict__ bias, int K,
+                                                             int E, int top, bool normalise, float scale, int T, int* __restrict__ idx, float* __restrict__ wt) {
+  extern __shared__ __align__(16) float xs[];     // [TB][K] rows | [TB][E] logits | [TB][E] scratch
+  float* z = xs + TB * K;
+  const int t0 = blockIdx.x * TB, nt = min(TB, T - t0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31, k4 = K / 4;
+  for (int e = threadIdx.x; e < TB * k4; e += 256) {
+    const int i = e / k4;
+    float f[4] = {0.f, 0.f, 0.f, 0.f};
+    if (i < nt) load4<AT>(x + (long long)(t0 + i) * ld_x + 4 * (e - i * k4), f);
+    store4<float>(xs + 4 * e, f);
+  }
+  __syncthreads();
+  for (int e = warp; e < E; e += 8) {
+    const float4* wr = reinterpret_cast<const float4*>(w + (long long)e * K);
+    float acc[TB];
+#pragma unroll
+    for (int i = 0; i < TB; ++i) acc[i] = 0.f;
+#pragma unroll 8
+    for (int k = lane; k < k4; k += 32) {
+      const float4 f = wr[k];
+#pragma unroll
+      for (int i = 0; i < TB; ++i) {
+        const float4 v = reinterpret_cast<const float4*>(xs)[i * k4 + k];
+        acc[i] += f.x * v.x + f.y * v.y + f.z * v.z + f.w * v.w;
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TB; ++i) { const float s = warp_sum(acc[i]); if (lane == 0) z[i * E + e] = s; }
+  }
+  __syncthreads();
+  for (int i = warp; i < nt; i += 8)
+    topk_of_row(z + i * E, z + TB * E + i * E, bias, 0, E, top, idx + (long long)(t0 + i) * top, wt + (long long)(t0 + i) * top, normalise, scale);
 }
 
 // gate rows g and up rows u (F wide each, own row strides) -> g' sigmoid(1.702 g') (u' + 1),  g' = min(s g, limit), u' = clamp(s u, +-limit).  Block i handles row
@@ -1074,6 +1116,28 @@ cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias
                                cudaStream_t s) {
   if (top > E || (size_t)E * sizeof(float) > 48 * 1024) return cudaErrorInvalidValue;
   sigmoid_topk_kernel<<<T, 32, E * sizeof(float), s>>>(z, ld_z, bias, mode, E, top, idx, w, normalise, scale);
+  return last();
+}
+
+cudaError_t sigmoid_router_launch(const void* x, long long ld_x, const float* w, const float* bias, int K, int E, int top, bool normalise, float scale, int* idx, float* wt,
+                                  bool f32, int T, cudaStream_t s) {
+  if (top > E || K % 4 != 0) return cudaErrorInvalidValue;
+  const size_t one = ((size_t)K + 2 * E) * sizeof(float);
+  const bool four = T >= 512 && 4 * one <= 200 * 1024;
+  auto go = [&](auto k, int tb) -> cudaError_t {
+    if (tb * one > 48 * 1024) { const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(tb * one)); if (e != cudaSuccess) return e; }
+    return cudaSuccess;
+  };
+  AT_DISPATCH(f32,
+    if (four) {
+      const cudaError_t e = go(sigmoid_router_kernel<AT, 4>, 4);
+      if (e != cudaSuccess) return e;
+      sigmoid_router_kernel<AT, 4><<<(T + 3) / 4, 256, 4 * one, s>>>((const AT*)x, ld_x, w, bias, K, E, top, normalise, scale, T, idx, wt);
+    } else {
+      const cudaError_t e = go(sigmoid_router_kernel<AT, 1>, 1);
+      if (e != cudaSuccess) return e;
+      sigmoid_router_kernel<AT, 1><<<T, 256, one, s>>>((const AT*)x, ld_x, w, bias, K, E, top, normalise, scale, T, idx, wt);
+    });
   return last();
 }
 

@@ -47,6 +47,9 @@ cudaError_t mlstm_scan_launch(const void* in, long long ld_in, const float* gate
 // over the chosen logits
 cudaError_t router_topk_launch(const float* z, long long ld_z, const float* bias, int mode, int E, int top, int* idx, float* w, bool normalise, float scale, int T,
                                cudaStream_t s);
+// router product (w fp32 [E, K]) and choice of mode 0 in one kernel; K and ld_x multiples of 4, x aligned to four entries
+cudaError_t sigmoid_router_launch(const void* x, long long ld_x, const float* w, const float* bias, int K, int E, int top, bool normalise, float scale, int* idx, float* wt,
+                                  bool f32, int T, cudaStream_t s);
 // kind 0: clamped GLU (limit); kind 1: silu(g) * u * scale; kind 2: gelu_tanh(g) * u * scale
 cudaError_t clamped_glu_launch(const void* g, long long ld_g, const void* u, long long ld_u, int F, float limit, const int* row_of,
                                const float* scale, void* out, bool f32, int rows, int kind, cudaStream_t s);

@@ -71,7 +71,7 @@ constexpr int kRowWarps = 4;
 // pages by asynchronous copies of S - 1 steps ahead — every thread reads back only what it copied itself, so no barrier is involved — and
 // uses them for RG query heads.  Every lane group runs an online softmax (base 2) of its own over its keys;
 // the groups are merged at the end, over the lanes of a warp by shuffles and over the warps in shared memory.  BIAS: distance_bias on the scores,
-// fetched before the wait for the keys.
+// evaluated once per key and head for the whole CTA (bias_keys > 0) or where it is used.
 template <typename AT, int LK, int RG, int U, int S, bool BIAS>
 __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_kernel(SinkAttnArgs a) {
   extern __shared__ __align__(16) unsigned char ring[];      // [S][U][key, value][thread] chunks
@@ -83,6 +83,7 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
   const int g = blockIdx.y / nb, r0 = (blockIdx.y % nb) * RG, pos = a.positions[t];
   const int* bt = a.block_tables + (long long)seq_of(a.cu, a.B, t) * a.max_blocks;
   const bool dk = d0 < D, dv = d0 < V;
+  float* bias = reinterpret_cast<float*>(ring + S * U * 2 * 32 * kRowWarps * kChunkBytes<AT>);      // [bias_keys][RG], base 2
   float2 q[RG][4], o[RG][4];
   float m[RG], l[RG];
 #pragma unroll
@@ -132,6 +133,15 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
         if (!dv) stf<AT>(slot + (2 * c + 1) * kSlots + e, 0.f);
       }
   }
+  if constexpr (BIAS) {
+    if (a.bias_keys > 0) {
+      for (int e = threadIdx.x; e < (iend - ibeg) * RG; e += 32 * kRowWarps) {
+        const int i = e / RG, r = e % RG;
+        bias[e] = r0 + r < Rg ? kLog2e * distance_bias(a, g * Rg + r0 + r, pos - vis.key_at(ibeg + i)) : 0.f;
+      }
+      __syncthreads();
+    }
+  }
   if (steps > 0) pages(0);
 #pragma unroll
   for (int k = 0; k < S - 1; ++k) {
@@ -141,15 +151,6 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
   int stage = 0;
   for (int k = 0; k < steps; ++k) {
     const int i0 = first + k * U * STEP;
-    float db[BIAS ? U * RG : 1];
-    if constexpr (BIAS) {
-#pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int n = pos - vis.key_at(min(i0 + u * STEP, iend - 1));
-#pragma unroll
-        for (int r = 0; r < RG; ++r) db[u * RG + r] = r0 + r < Rg ? distance_bias(a, g * Rg + r0 + r, n) : 0.f;
-      }
-    }
     asm volatile("cp.async.wait_group %0;" ::"n"(S - 2) : "memory");
     const AT* cur = slot + stage * U * 2 * kSlots;
     stage = stage + 1 == S ? 0 : stage + 1;
@@ -169,7 +170,20 @@ __global__ void __launch_bounds__(32 * kRowWarps, RG == 4 ? 4 : 5) sink_rows_ker
     sum_over_lanes<U * RG, LK>(s, lane);
     if constexpr (BIAS) {
 #pragma unroll
-      for (int e = 0; e < U * RG; ++e) s[e] = fmaf(db[e], kLog2e, s[e]);
+      for (int u = 0; u < U; ++u) {
+        const int i = min(i0 + u * STEP, iend - 1);
+        if (a.bias_keys > 0) {
+          const float* b = bias + (i - ibeg) * RG;
+          if constexpr (RG == 4) { const float4 f = *reinterpret_cast<const float4*>(b); s[u * RG] += f.x; s[u * RG + 1] += f.y; s[u * RG + 2] += f.z; s[u * RG + 3] += f.w; }
+          else
+#pragma unroll
+            for (int r = 0; r < RG; ++r) s[u * RG + r] += b[r];
+        } else {
+          const int n = pos - vis.key_at(i);
+#pragma unroll
+          for (int r = 0; r < RG; ++r) if (r0 + r < Rg) s[u * RG + r] = fmaf(distance_bias(a, g * Rg + r0 + r, n), kLog2e, s[u * RG + r]);
+        }
+      }
     }
 #pragma unroll
     for (int u = 0; u < U; ++u)
@@ -372,7 +386,8 @@ template <typename AT, int LK, bool BIAS>
 cudaError_t rows_form(const SinkAttnArgs& a, int T, cudaStream_t s) {
   const int Rg = a.H / a.G, hp = heads_of(Rg);
   const dim3 grid(T, a.G * ((Rg + hp - 1) / hp), a.nsplit);
-  constexpr int U = 2, S = sizeof(AT) == 2 ? 4 : 3, smem = S * U * 2 * 32 * kRowWarps * kChunkBytes<AT>;
+  constexpr int U = 2, S = sizeof(AT) == 2 ? 4 : 3;
+  const int smem = S * U * 2 * 32 * kRowWarps * kChunkBytes<AT> + (BIAS ? a.bias_keys * hp * (int)sizeof(float) : 0);
   auto go = [&](auto k) -> cudaError_t {
     const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);      // static and dynamic together may pass 48 KB
     if (e != cudaSuccess) return e;
@@ -414,6 +429,7 @@ cudaError_t attention(const SinkAttnArgs& a, int T, cudaStream_t s) {
 
 int sink_attention_heads_per_cta(int H, int G, int D, int V) { return vector_form(D, V) ? heads_of(H / G) : general_warps(H / G); }
 int sink_attention_chunk_unit() { return 32; }
+int sink_attention_bias_keys() { return 2048; }
 
 cudaError_t sink_attention_launch(const SinkAttnArgs& a, bool f32, int T, cudaStream_t s) {
   if (a.G < 1 || a.H % a.G != 0 || a.V > 512 || (size_t)(8 * a.D + kTile * (a.D + 1) + kTile * a.V) * sizeof(float) > 220 * 1024 || a.keep < 0) return cudaErrorInvalidValue;

@@ -21,12 +21,15 @@ struct SinkAttnArgs {
   bool gate_elem;                           // with gate_elem, per element [T, H V]
   void* out; long long ld_out;              // activation type, row t at out + t * ld_out, head h at column h * V
   int nsplit, chunk;                        // keys split into nsplit parts of `chunk` visible keys
+  int bias_keys;                            // most visible keys of a CTA when their biases are kept in shared memory (0: evaluated key by key)
   float* part;                              // [T, H, nsplit, V + 2] = (m, l, o[V]) when nsplit > 1
 };
 // query heads one CTA serves for these sizes
 int sink_attention_heads_per_cta(int H, int G, int D, int V);
 // granularity of `chunk`
 int sink_attention_chunk_unit();
+// keys of a CTA whose biases shared memory takes
+int sink_attention_bias_keys();
 cudaError_t sink_attention_launch(const SinkAttnArgs& a, bool f32, int T, cudaStream_t s);
 // bf16 on the tensor cores, 64 query rows per CTA (context_lens instead of positions; nsplit, chunk, part unused)
 bool sink_flash_supported(int D, int V);

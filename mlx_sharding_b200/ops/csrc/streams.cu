@@ -505,6 +505,61 @@ __global__ void qk_norm_rope_append_kernel(PrologueArgs a) {
   }
 }
 
+// The form without rotation, value mixing and heads to tell apart: one norm over the query row and one over the key row, four entries per
+// thread and step, the row in registers (NQ steps of 256 threads; sizes multiples of 4, rows and pools aligned to four entries).
+template <typename AT, int NQ>
+__global__ void __launch_bounds__(256) whole_norm_append_kernel(PrologueArgs a) {
+  __shared__ float red[2][8];
+  const long long t = blockIdx.x;
+  const int D = a.D, V = a.V, G = a.G, nq = a.H * D / 4, nk = G * D / 4, nv = G * V / 4;
+  const AT* r = (const AT*)a.rows + t * a.ld;
+  float q[NQ][4], k[NQ][4], sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int c = threadIdx.x + 256 * i;
+    if (c < nq) load4<AT>(r + a.q0 + 4 * c, q[i]);
+    if (c < nk) load4<AT>(r + a.k0 + 4 * c, k[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int c = threadIdx.x + 256 * i;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { if (c < nq) sq += q[i][e] * q[i][e]; if (c < nk) sk += k[i][e] * k[i][e]; }
+  }
+  sq = warp_sum(sq); sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+  const int slot = a.slot_map[t], pg = slot / a.page, off = slot % a.page;
+  for (int c = threadIdx.x; c < nv; c += 256) {
+    const int h = 4 * c / V, d = 4 * c - h * V;
+    float f[4];
+    load4<AT>(r + a.v0 + 4 * c, f);
+    store4<AT>((AT*)a.vpool + (((long long)pg * G + h) * a.page + off) * V + d, f);
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < 8; ++w) { sq += red[0][w]; sk += red[1][w]; }
+  const float iq = 1.f / sqrtf(sq / (float)(4 * nq) + a.eps), ik = 1.f / sqrtf(sk / (float)(4 * nk) + a.eps);
+#pragma unroll
+  for (int i = 0; i < NQ; ++i) {
+    const int c = threadIdx.x + 256 * i;
+    float w[4] = {1.f, 1.f, 1.f, 1.f};
+    if (c < nq) {
+      if (a.qn != nullptr) load4<float>(a.qn + 4 * c, w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) q[i][e] *= iq * w[e];
+      store4<float>(a.qout + 4 * (t * nq + c), q[i]);
+    }
+    if (c < nk) {
+      if (a.kn != nullptr) load4<float>(a.kn + 4 * c, w);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) k[i][e] *= ik * w[e];
+      const int h = 4 * c / D, d = 4 * c - h * D;
+      store4<AT>((AT*)a.kpool + (((long long)pg * G + h) * a.page + off) * D + d, k[i]);
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------- router
 // One warp per token.  s = softmax(z) over all E experts; choice c = s + corr; groups = ng equal runs of neighbours, a group's value is
 // its largest c; experts outside the `keep` best groups count as -inf; the `top` largest c win (ties: lowest id); weights = their s.
@@ -676,6 +731,16 @@ cudaError_t qk_norm_rope_append_launch(const void* rows, long long ld, int q0, i
                                        const void* v_first, long long ld_vf, float lam, bool whole, int T, cudaStream_t s) {
   if (rot % 2 != 0 || rot > D || D > 1024 || (whole && norm_after)) return cudaErrorInvalidValue;
   const PrologueArgs a{rows, ld, q0, k0, v0, H, G, D, V, qn, kn, whole, eps, inv_freq, rot, rot_mult, positions, slot_map, page, v_first, ld_vf, lam, qout, kpool, vpool};
+  const int n4 = H * D / 4, es = f32 ? 4 : 2;
+  auto al = [](const void* p, int b) { return reinterpret_cast<uintptr_t>(p) % b == 0; };
+  if (whole && rot == 0 && v_first == nullptr && G <= H && D % 4 == 0 && V % 4 == 0 && ld % 4 == 0 && q0 % 4 == 0 && k0 % 4 == 0 && v0 % 4 == 0 && n4 <= 8 * 256 &&
+      al(rows, 4 * es) && al(kpool, 4 * es) && al(vpool, 4 * es) && al(qn, 16) && al(kn, 16) && al(qout, 16)) {
+    if (n4 <= 256) AT_DISPATCH(f32, (whole_norm_append_kernel<AT, 1><<<T, 256, 0, s>>>(a)));
+    else if (n4 <= 2 * 256) AT_DISPATCH(f32, (whole_norm_append_kernel<AT, 2><<<T, 256, 0, s>>>(a)));
+    else if (n4 <= 4 * 256) AT_DISPATCH(f32, (whole_norm_append_kernel<AT, 4><<<T, 256, 0, s>>>(a)));
+    else AT_DISPATCH(f32, (whole_norm_append_kernel<AT, 8><<<T, 256, 0, s>>>(a)));
+    return last();
+  }
   if (D <= 64) AT_DISPATCH(f32, (prologue_t<AT, 2>(a, half, norm_after, T, s)));
   else if (D <= 128) AT_DISPATCH(f32, (prologue_t<AT, 4>(a, half, norm_after, T, s)));
   else if (D <= 256) AT_DISPATCH(f32, (prologue_t<AT, 8>(a, half, norm_after, T, s)));

@@ -192,8 +192,8 @@ def moe_route(x: torch.Tensor, gate_w: torch.Tensor, top_k: int, method: str = "
 
 
 # ------------------------------------------------------------------------------------------ K11
-def run_aside(fn):
-    """Backend hook: independent work that the CUDA backend forks onto a side stream runs inline here."""
+def run_aside(fn, lane: int = 0):
+    """Backend hook: independent work that the CUDA backend forks onto a side stream (``lane``: which of them) runs inline here."""
     fn()
     return None
 
@@ -628,11 +628,12 @@ def clamped_gated_up(x: torch.Tensor, Wg: LinearWeight, Wu: LinearWeight, limit:
 
 
 def moe_clamped_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, Wg: LinearWeight, Wu: LinearWeight, Wd: LinearWeight,
-                        limit: float, on_input: bool = True) -> torch.Tensor:
+                        limit: float, on_input: bool = True, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``y[t] = sum_j expert_{idx[t,j]}(w[t,j] x[t])`` with clamped-GLU experts (:func:`clamped_glu`): the router weight scales the
-    expert's INPUT; ``on_input=False``: its OUTPUT, ``y[t] = sum_j w[t,j] expert_{idx[t,j]}(x[t])``.  Banks ``Wg``, ``Wu`` ``[E, F, K]``, ``Wd`` ``[E, K, F]``.  Returns fp32 ``[T, K]``."""
+    expert's INPUT; ``on_input=False``: its OUTPUT, ``y[t] = sum_j w[t,j] expert_{idx[t,j]}(x[t])``.  Banks ``Wg``, ``Wu`` ``[E, F, K]``, ``Wd`` ``[E, K, F]``.  Returns fp32 ``[T, K]``
+    (in ``out`` when given)."""
     T, k = idx.shape
-    y = torch.zeros(T, Wd.weight.shape[1], dtype=torch.float32, device=x.device)
+    y = torch.zeros(T, Wd.weight.shape[1], dtype=torch.float32, device=x.device) if out is None else out.zero_()
     il = idx.long()
     for e in range(Wg.weight.shape[0]):
         tok, slot = torch.where(il == e)
@@ -644,6 +645,12 @@ def moe_clamped_experts(x: torch.Tensor, idx: torch.Tensor, w: torch.Tensor, Wg:
         ye = h.float() @ Wd.weight[e].float().t()
         y.index_add_(0, tok, ye if on_input else ye * we)
     return y
+
+
+def sigmoid_router(x: torch.Tensor, w: torch.Tensor, num_experts: int, top: int, correction: Optional[torch.Tensor] = None, normalise: bool = False,
+                   scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """:func:`sigmoid_topk` of :func:`router_logits` (one kernel on the b200 backend)."""
+    return sigmoid_topk(router_logits(x, w), num_experts, top, correction, normalise, scale)
 
 
 def router_logits(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
