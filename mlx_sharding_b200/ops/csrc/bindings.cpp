@@ -1330,7 +1330,7 @@ Tensor hy_head_delta_scan(const Tensor& qkv, const Tensor& beta, const Tensor& d
   if (T == 0) return out;
   b200::HeadDeltaArgs a{qkv.data_ptr(), qkv.stride(0), beta.data_ptr(), beta.stride(0), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr<float>(), A_log.data_ptr<float>(),
                         state.data_ptr<float>(), cu.data_ptr<int>(), ctx.data_ptr<int>(), slots.data_ptr<int>(), out.data_ptr<float>(), (int)B, (int)T, (int)H, (int)G,
-                        (int)Dk, (int)V, (float)q_scale, (float)unit_eps, nullptr};
+                        (int)Dk, (int)V, (float)q_scale, (float)unit_eps, nullptr, 0};
   const long long ws = b200::head_delta_workspace(a, (int)max_q);
   Tensor pre;
   if (ws > 0) { pre = torch::empty({(int64_t)ws}, out.options()); a.pre = pre.data_ptr<float>(); ++g_launches; }

@@ -16,13 +16,14 @@ namespace b200 {
 namespace {
 
 constexpr int C = 4;                         // tokens of a group
-constexpr int kCoef = 12;                    // numbers per token and head: beta | beta G | G | D_iC | beta D (k . k) lags 1 2 3 | - | D (k . q) lags 0 1 2 3
+constexpr int kCoef = 12;                    // numbers per token i and head: beta, beta G, G, D_iC | beta D_mi (k_m . k_i), m = 0 1 2 | - | D_mi (k_m . q_i), m = 0 .. 3
 constexpr int kGroupsStaged = 4;             // groups per staging buffer of the scan
 
 __device__ __forceinline__ float decay_of(float raw, float bias, float A_log) { return expf(-expf(A_log) * softplus_f(raw + bias)); }
 
-// workspace of one group of C tokens, floats: [k: C][G N] | [q: C][G N] | [v: C][H P] | [coef: H][C][kCoef]
-__host__ __device__ inline long long group_floats(int G, int H, int N, int P) { return (long long)C * (2 * G * N + H * P) + (long long)C * kCoef * H; }
+// workspace of one group of C tokens, floats: [G][k: C, q: C][NP] (rows padded with zeros to NP) | [H][P][v: C] | [H][C][kCoef].  What a CTA of the scan
+// needs of it are three runs of whole 16-byte units, whatever the sizes.
+__host__ __device__ inline long long group_floats(int G, int H, int NP, int P) { return (long long)C * (2 * G * NP + H * P + H * kCoef); }
 // groups of sequence b: numbers cu[b] / C + b, .. (room for the ragged ends of all sequences: T / C + B groups)
 __device__ __forceinline__ int first_group(const int* cu, int b) { return cu[b] / C + b; }
 
@@ -36,11 +37,10 @@ __global__ void head_delta_prepare_kernel(HeadDeltaArgs a) {
   while (lo < hi) { const int mid = (lo + hi + 1) >> 1; if (first_group(a.cu, mid) <= gi) lo = mid; else hi = mid - 1; }
   const int b = lo, s = a.cu[b], q = a.cu[b + 1] - s, j0 = (gi - first_group(a.cu, b)) * C, nt = min(C, q - j0);
   if (nt <= 0) return;
-  const int N = a.N, GN = a.G * N, HP = a.H * a.P;
+  const int N = a.N, NP = a.NP, GN = a.G * N, HP = a.H * a.P;
   const AT* in = reinterpret_cast<const AT*>(a.in) + (long long)(s + j0) * a.ld_in;
-  float* ko = a.pre + (long long)gi * group_floats(a.G, a.H, N, a.P);
-  float* qo = ko + (long long)C * GN;
-  float* vo = qo + (long long)C * GN;
+  float* ko = a.pre + (long long)gi * group_floats(a.G, a.H, NP, a.P);
+  float* vo = ko + (long long)2 * C * a.G * NP;
   float* co = vo + (long long)C * HP;
   auto load = [&](const AT* p, float* f) { if constexpr (VW == 4) load4<AT>(p, f); else f[0] = ldf<AT>(p); };
   auto store = [&](float* p, const float* f) { if constexpr (VW == 4) store4<float>(p, f); else *p = f[0]; };
@@ -85,26 +85,29 @@ __global__ void head_delta_prepare_kernel(HeadDeltaArgs a) {
     for (int i = 0; i < C; ++i)
 #pragma unroll
       for (int m = 0; m <= i; ++m) { const float v = warp_sum(x[z]) * ik[m] * iq[i]; if (lane == 0) dots[g * 16 + z] = v; ++z; }
-    for (int n = VW * lane; n < N; n += 32 * VW) {
+    for (int n = VW * lane; n < NP; n += 32 * VW) {
 #pragma unroll
       for (int i = 0; i < C; ++i) {
         float k[VW], w[VW];
 #pragma unroll
         for (int e = 0; e < VW; ++e) k[e] = w[e] = 0.f;
-        if (i < nt) { load(in + i * a.ld_in + GN + g * N + n, k); load(in + i * a.ld_in + g * N + n, w); }
+        if (i < nt && n < N) { load(in + i * a.ld_in + GN + g * N + n, k); load(in + i * a.ld_in + g * N + n, w); }
 #pragma unroll
         for (int e = 0; e < VW; ++e) { k[e] *= ik[i]; w[e] *= iq[i]; }
-        store(ko + (long long)i * GN + g * N + n, k); store(qo + (long long)i * GN + g * N + n, w);
+        store(ko + (long long)(g * 2 * C + i) * NP + n, k); store(ko + (long long)(g * 2 * C + C + i) * NP + n, w);
       }
     }
   }
-  for (int e = VW * threadIdx.x; e < C * HP; e += VW * blockDim.x) {
-    const int i = e / HP;
-    float v[VW];
+  for (int e = VW * threadIdx.x; e < HP; e += VW * blockDim.x) {
+    float v[C][VW];
 #pragma unroll
-    for (int x = 0; x < VW; ++x) v[x] = 0.f;
-    if (i < nt) load(in + i * a.ld_in + 2 * GN + (e - i * HP), v);
-    store(vo + e, v);
+    for (int i = 0; i < C; ++i) {
+#pragma unroll
+      for (int x = 0; x < VW; ++x) v[i][x] = 0.f;
+      if (i < nt) load(in + i * a.ld_in + 2 * GN + e, v[i]);
+    }
+#pragma unroll
+    for (int x = 0; x < VW; ++x) { const float f[C] = {v[0][x], v[1][x], v[2][x], v[3][x]}; store4<float>(vo + (long long)C * (e + x), f); }
   }
   __syncthreads();
   for (int h = threadIdx.x; h < a.H; h += blockDim.x) {
@@ -130,8 +133,8 @@ __global__ void head_delta_prepare_kernel(HeadDeltaArgs a) {
       float D = 1.f;
 #pragma unroll
       for (int lag = 0; lag <= i; ++lag) {   // D = g_(i-lag+1) .. g_i
-        if (lag > 0) { D *= gd[i - lag + 1]; o[3 + lag] = bt[i] * D * d[zk + i - lag]; }
-        o[8 + lag] = D * d[zq + i - lag];
+        if (lag > 0) { D *= gd[i - lag + 1]; o[4 + i - lag] = bt[i] * D * d[zk + i - lag]; }
+        o[8 + i - lag] = D * d[zq + i - lag];
       }
       zk += i; zq += i + 1;
 #pragma unroll
@@ -144,141 +147,178 @@ __global__ void head_delta_prepare_kernel(HeadDeltaArgs a) {
 __device__ __forceinline__ void copy_async_16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
-__device__ __forceinline__ void copy_async_4(float* dst, const float* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+
+// Sums of NV values over the L lanes of a column group, halving what each lane holds: with M = min(L, NV), value v ends in the lanes l with
+// l % M == v % M as d[v / M].
+template <int L, int NV> __device__ __forceinline__ void fold_lanes(float (&d)[NV], int lane) {
+#pragma unroll
+  for (int w = 1, n = NV / 2; w < L; w <<= 1, n >>= 1) {
+    if (n > 0) {
+#pragma unroll
+      for (int i = 0; i < n; ++i) {
+        const bool odd = lane & w;
+        const float keep = odd ? d[2 * i + 1] : d[2 * i], send = odd ? d[2 * i] : d[2 * i + 1];
+        d[i] = keep + __shfl_xor_sync(0xffffffffu, send, w);
+      }
+    } else {
+      d[0] += __shfl_xor_sync(0xffffffffu, d[0], w);
+    }
+  }
 }
 
-// State in registers: L lanes share a value column, lane l holding the key rows 4 (l + L j) + e (j < NR4, e < 4), so a warp runs 32 / L columns.
-// Groups arrive by asynchronous copies into one of two buffers while the buffer before is computed; rows behind N and columns behind P are
-// zeros, so the loop has no bounds checks.                                    grid (B, H, ceil(P / PB)), PB = warps * 32 / L
-template <int L, int NR4>
-__global__ void __launch_bounds__(128) head_delta_scan_kernel(HeadDeltaArgs a) {
-  constexpr int CPW = 32 / L, NP = 4 * L * NR4;
+// State in registers: L lanes share KC value columns (a key or query fetched from shared memory serves all of them), lane l holding the key rows 4 (l + L j) + e (j < NR4, e < 4), so a warp runs 32 / L *
+// KC columns.  Groups arrive by asynchronous copies into one of two buffers while the buffer before is computed; rows behind N and columns
+// behind P are zeros, so the loop has no bounds checks.                       grid (B, H, ceil(P / PB)), PB = 4 * KC * 32 / L, block 128
+constexpr int kScanThreads = 128;
+
+template <int L, int NR4, int KC>
+__global__ void __launch_bounds__(kScanThreads) head_delta_scan_kernel(HeadDeltaArgs a) {
+  constexpr int CPW = 32 / L, NP = 4 * L * NR4, PB = kScanThreads / 32 * KC * CPW, NV = 2 * C * KC, M = L < NV ? L : NV;
+  static_assert(C == 4 && (KC == 1 || KC == 2), "sums per column group: value v = token | (query << 2) | (column << 3)");
   extern __shared__ __align__(16) float smem[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, PB = nw * CPW;
-  const int l = lane % L, b = blockIdx.x, h = blockIdx.y, N = a.N, P = a.P, H = a.H, p0 = blockIdx.z * PB;
-  const int g = h / (H / a.G), col = warp * CPW + lane / L, pc = p0 + col;
-  const bool colok = pc < P;
-  const int per = 2 * C * NP + C * PB + C * kCoef;         // floats of one group: k | q | v | coef
+  constexpr int per = 2 * C * NP + C * PB + C * kCoef;     // floats of one group: k, q | v | coef
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l = lane % L, b = blockIdx.x, h = blockIdx.y, N = a.N, P = a.P, H = a.H, p0 = blockIdx.z * PB;
+  const int g = h / (H / a.G), col = warp * KC * CPW + lane / L;          // columns col and col + CPW of the CTA's
   const int s = a.cu[b], q = a.cu[b + 1] - s;
   if (q == 0) return;
   const bool fresh = a.ctx[b] - q == 0;
-  float* gS = a.state + ((long long)a.slots[b] * H + h) * N * P + pc;
-  float2 st[2 * NR4];
+  float* gS = a.state + ((long long)a.slots[b] * H + h) * N * P + p0 + col;
+  bool colok[KC];
+  float2 st[KC][2 * NR4];
 #pragma unroll
-  for (int j = 0; j < NR4; ++j)
+  for (int x = 0; x < KC; ++x) {
+    colok[x] = p0 + col + x * CPW < P;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int n = 4 * (l + L * j) + e;
-      const float v = (!fresh && colok && n < N) ? gS[(long long)n * P] : 0.f;
-      if (e & 1) st[2 * j + e / 2].y = v; else st[2 * j + e / 2].x = v;
-    }
-  for (int e = threadIdx.x; e < 2 * kGroupsStaged * per; e += blockDim.x) smem[e] = 0.f;
+    for (int j = 0; j < NR4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = 4 * (l + L * j) + e;
+        const float v = (!fresh && colok[x] && n < N) ? gS[(long long)n * P + x * CPW] : 0.f;
+        if (e & 1) st[x][2 * j + e / 2].y = v; else st[x][2 * j + e / 2].x = v;
+      }
+  }
+  for (int e = threadIdx.x; e < 2 * kGroupsStaged * per; e += kScanThreads) smem[e] = 0.f;
   __syncthreads();
-  const int GN = a.G * N, HP = H * P, vw = min(PB, P - p0), groups = (q + C - 1) / C;
-  const long long gf = group_floats(a.G, H, N, P);
-  const float* pre = a.pre + (long long)first_group(a.cu, b) * gf;
-  const bool vec = N % 4 == 0 && P % 4 == 0 && PB % 4 == 0;          // 16-byte copies: every segment starts and ends on a 16-byte boundary
-  const int n4 = vec ? N / 4 : N, v4 = vec ? vw / 4 : vw, items = C * (2 * n4 + v4) + C * kCoef / 4;
-  auto fetch = [&](int g0, int ng, float* buf) {
-    for (int e = threadIdx.x; e < ng * items; e += blockDim.x) {
-      const int gg = e / items;
-      int c = e - gg * items;
-      const float* src = pre + (g0 + gg) * gf;
+  const int HP = H * P, vw = min(PB, P - p0), groups = (q + C - 1) / C;
+  const long long gf = group_floats(a.G, H, NP, P);
+  // this thread's 16-byte units of a group: keys and queries at 4 threadIdx.x + 512 i; one unit of values or coefficients
+  const float* src = a.pre + (long long)first_group(a.cu, b) * gf + 4 * threadIdx.x;
+  const int extra = (int)threadIdx.x < vw ? 2 * C * a.G * NP + C * (h * P + p0) : 2 * C * a.G * NP + C * HP + h * C * kCoef - 4 * vw;
+  const int xdst = 2 * C * NP + ((int)threadIdx.x < vw ? 0 : C * PB - 4 * vw) + 4 * threadIdx.x;
+  const bool xok = (int)threadIdx.x < vw + C * kCoef / 4;
+  src += g * 2 * C * NP;
+  const float* xsrc = src - g * 2 * C * NP + extra;
+  auto fetch = [&](int ng, float* buf) {     // the next ng groups
+    for (int gg = 0; gg < ng; ++gg) {
       float* dst = buf + gg * per;
-      if (c >= C * (2 * n4 + v4)) {          // coefficients (workspace of a multiple of 4 floats in front of them or 4-byte copies)
-        c -= C * (2 * n4 + v4);
-        src += (long long)C * (2 * GN + HP) + (long long)h * C * kCoef + 4 * c;
-        dst += 2 * C * NP + C * PB + 4 * c;
-        if (vec) copy_async_16(dst, src);
-        else
 #pragma unroll
-          for (int x = 0; x < 4; ++x) copy_async_4(dst + x, src + x);
-        continue;
-      }
-      if (c < 2 * C * n4) {
-        const int row = c / n4, x = c - row * n4;                    // row < C: keys, then queries
-        src += (long long)row * GN + g * N;
-        dst += row * NP;
-        if (vec) copy_async_16(dst + 4 * x, src + 4 * x); else copy_async_4(dst + x, src + x);
-      } else {
-        c -= 2 * C * n4;
-        const int row = c / v4, x = c - row * v4;
-        src += (long long)2 * C * GN + (long long)row * HP + h * P + p0;
-        dst += 2 * C * NP + row * PB;
-        if (vec) copy_async_16(dst + 4 * x, src + 4 * x); else copy_async_4(dst + x, src + x);
-      }
+      for (int i = 0; i < (2 * C * NP / 4 + kScanThreads - 1) / kScanThreads; ++i)
+        if (2 * C * NP / 4 % kScanThreads == 0 || 4 * (int)threadIdx.x + 4 * kScanThreads * i < 2 * C * NP)
+          copy_async_16(dst + 4 * threadIdx.x + 4 * kScanThreads * i, src + 4 * kScanThreads * i);
+      if (xok) copy_async_16(dst + xdst, xsrc);
+      src += gf; xsrc += gf;
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  fetch(0, min(kGroupsStaged, groups), smem);
+  static_assert(PB + C * kCoef / 4 <= kScanThreads, "one unit of values or coefficients per thread");
+  fetch(min(kGroupsStaged, groups), smem);
+  float* out = a.out + (long long)(s + l % C) * HP + h * P + p0 + col;       // token l % C of the group
+  int left = q - l % C;                      // > 0: that token exists
   int blk = 0;
   for (int g0 = 0; g0 < groups; g0 += kGroupsStaged, ++blk) {
     const int ng = min(kGroupsStaged, groups - g0);
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                        // these groups have landed for every thread; the other buffer is no longer read
-    if (g0 + kGroupsStaged < groups) fetch(g0 + kGroupsStaged, min(kGroupsStaged, groups - g0 - kGroupsStaged), smem + ((blk + 1) & 1) * kGroupsStaged * per);
+    if (g0 + kGroupsStaged < groups) fetch(min(kGroupsStaged, groups - g0 - kGroupsStaged), smem + ((blk + 1) & 1) * kGroupsStaged * per);
     const float* cur = smem + (blk & 1) * kGroupsStaged * per;
     for (int gg = 0; gg < ng; ++gg) {
       const float* tk = cur + gg * per;
       const float4* kq4 = reinterpret_cast<const float4*>(tk) + l;
-      float2 acc[2 * C];
+      float2 acc[KC][2 * C];
 #pragma unroll
-      for (int i = 0; i < 2 * C; ++i) acc[i] = make_float2(0.f, 0.f);
+      for (int i = 0; i < 2 * C; ++i)
+#pragma unroll
+        for (int x = 0; x < KC; ++x) acc[x][i] = make_float2(0.f, 0.f);
 #pragma unroll
       for (int j = 0; j < NR4; ++j)
 #pragma unroll
         for (int i = 0; i < 2 * C; ++i) {
           const float4 f = kq4[i * (NP / 4) + j * L];
-          acc[i] = fma2(st[2 * j], make_float2(f.x, f.y), acc[i]);
-          acc[i] = fma2(st[2 * j + 1], make_float2(f.z, f.w), acc[i]);
+#pragma unroll
+          for (int x = 0; x < KC; ++x) {
+            acc[x][i] = fma2(st[x][2 * j], make_float2(f.x, f.y), acc[x][i]);
+            acc[x][i] = fma2(st[x][2 * j + 1], make_float2(f.z, f.w), acc[x][i]);
+          }
         }
-      float d[2 * C];
+      float d[NV];
 #pragma unroll
-      for (int i = 0; i < 2 * C; ++i) d[i] = acc[i].x + acc[i].y;
-      sum_over_lanes<2 * C, L>(d, lane);
-      const float* vs = tk + 2 * C * NP + col;
+      for (int v = 0; v < NV; ++v) d[v] = acc[v >> 3][v & 7].x + acc[v >> 3][v & 7].y;
+      fold_lanes<L, NV>(d, lane);
       const float4* cf = reinterpret_cast<const float4*>(tk + 2 * C * NP + C * PB);
-      float u[C], w[C], o[C], GC = 1.f;
+      float vt[KC][C], u[KC][C], w[KC][C], GC = 1.f;
 #pragma unroll
-      for (int i = 0; i < C; ++i) {
-        const float4 c0 = cf[3 * i], ck = cf[3 * i + 1], cq = cf[3 * i + 2];
-        float v = c0.x * vs[i * PB] - c0.y * d[i];
-        if (i > 0) v -= ck.x * u[i > 0 ? i - 1 : 0];
-        if (i > 1) v -= ck.y * u[i > 1 ? i - 2 : 0];
-        if (i > 2) v -= ck.z * u[i > 2 ? i - 3 : 0];
-        u[i] = v;
-        w[i] = c0.w * v;
-        float y = c0.z * d[C + i] + cq.x * v;
-        if (i > 0) y += cq.y * u[i > 0 ? i - 1 : 0];
-        if (i > 1) y += cq.z * u[i > 1 ? i - 2 : 0];
-        if (i > 2) y += cq.w * u[i > 2 ? i - 3 : 0];
-        o[i] = y;
-        if (i == C - 1) GC = c0.z;
+      for (int x = 0; x < KC; ++x) {
+        const float4 f = *reinterpret_cast<const float4*>(tk + 2 * C * NP + C * (col + x * CPW));
+        vt[x][0] = f.x; vt[x][1] = f.y; vt[x][2] = f.z; vt[x][3] = f.w;
       }
 #pragma unroll
-      for (int j = 0; j < NR4; ++j) {
-        st[2 * j] = mul2(st[2 * j], make_float2(GC, GC));
-        st[2 * j + 1] = mul2(st[2 * j + 1], make_float2(GC, GC));
+      for (int i = 0; i < C; ++i) {
+        const float4 cb = cf[3 * i], ck = cf[3 * i + 1];
+#pragma unroll
+        for (int x = 0; x < KC; ++x) {
+          const int v = i + 8 * x;           // S^T k_i
+          float t = cb.x * vt[x][i] - cb.y * __shfl_sync(0xffffffffu, d[v / M], v % M, L);
+          if (i > 0) t -= ck.x * u[x][0];
+          if (i > 1) t -= ck.y * u[x][1];
+          if (i > 2) t -= ck.z * u[x][2];
+          u[x][i] = t;
+          w[x][i] = cb.w * t;
+        }
+        if (i == C - 1) GC = cb.z;
+      }
+      {                                      // the lane that holds S^T q_i finishes and stores token i
+        const float G = cf[3 * (l % C)].z;
+        const float4 cq = cf[3 * (l % C) + 2];
+#pragma unroll
+        for (int x = 0; x < NV / M; ++x) {
+          const int v = x * M + l % M, c = KC == 1 ? 0 : v >> 3;      // column; lanes differ in it only when M = 16
+          constexpr bool kMixed = KC == 2 && M == 16;
+          const float* uc = u[kMixed ? 0 : (x * M) >> 3];
+          float y = G * d[x];
+          y += cq.x * (kMixed && c ? u[KC - 1][0] : uc[0]);
+          y += cq.y * (kMixed && c ? u[KC - 1][1] : uc[1]);
+          y += cq.z * (kMixed && c ? u[KC - 1][2] : uc[2]);
+          y += cq.w * (kMixed && c ? u[KC - 1][3] : uc[3]);
+          if ((v & 4) && l < NV && (c ? colok[KC - 1] : colok[0]) && left > 0) out[c * CPW] = y;
+        }
+        out += (long long)C * HP; left -= C;
+      }
+#pragma unroll
+      for (int x = 0; x < KC; ++x)
+#pragma unroll
+        for (int j = 0; j < 2 * NR4; ++j) st[x][j] = mul2(st[x][j], make_float2(GC, GC));
+#pragma unroll
+      for (int j = 0; j < NR4; ++j)
 #pragma unroll
         for (int i = 0; i < C; ++i) {
           const float4 f = kq4[i * (NP / 4) + j * L];
-          st[2 * j] = fma2(make_float2(w[i], w[i]), make_float2(f.x, f.y), st[2 * j]);
-          st[2 * j + 1] = fma2(make_float2(w[i], w[i]), make_float2(f.z, f.w), st[2 * j + 1]);
+#pragma unroll
+          for (int x = 0; x < KC; ++x) {
+            st[x][2 * j] = fma2(make_float2(w[x][i], w[x][i]), make_float2(f.x, f.y), st[x][2 * j]);
+            st[x][2 * j + 1] = fma2(make_float2(w[x][i], w[x][i]), make_float2(f.z, f.w), st[x][2 * j + 1]);
+          }
         }
-      }
-      const int j = (g0 + gg) * C + l;       // lane l < C stores token l of the group
-      const float y = l == 0 ? o[0] : l == 1 ? o[1] : l == 2 ? o[2] : o[3];
-      if (l < C && colok && j < q) a.out[(long long)(s + j) * HP + h * P + pc] = y;
     }
   }
 #pragma unroll
-  for (int j = 0; j < NR4; ++j)
+  for (int x = 0; x < KC; ++x)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int n = 4 * (l + L * j) + e;
-      if (colok && n < N) gS[(long long)n * P] = (e & 1) ? st[2 * j + e / 2].y : st[2 * j + e / 2].x;
-    }
+    for (int j = 0; j < NR4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = 4 * (l + L * j) + e;
+        if (colok[x] && n < N) gS[(long long)n * P + x * CPW] = (e & 1) ? st[x][2 * j + e / 2].y : st[x][2 * j + e / 2].x;
+      }
 }
 
 // ---------------------------------------------------------------------------------------------------------- single tokens
@@ -410,21 +450,34 @@ cudaError_t prepare(const HeadDeltaArgs& a, cudaStream_t s) {
   return last();
 }
 
-template <int L>
-cudaError_t scan(const HeadDeltaArgs& a, int warps, cudaStream_t s) {
-  const int need = (a.N + 4 * L - 1) / (4 * L), cpw = 32 / L, PB = warps * cpw;
-  auto go = [&](auto k, int nr4) -> cudaError_t {
-    const size_t smem = 2 * (size_t)kGroupsStaged * (2 * C * 4 * L * nr4 + C * PB + C * kCoef) * sizeof(float);
+// lanes per column group, steps of 4 L key rows, columns per thread and warps of the scan.  Many columns: few lanes and two columns per thread
+// need the fewest instructions.  Few columns (a prompt alone): a token's time is the serial instruction count of a warp, so one column per
+// thread and more lanes (not all 32: what a warp does whatever its share then weighs too much).
+struct ScanShape { int L, nr4, kc; };
+ScanShape scan_shape(const HeadDeltaArgs& a) {
+  int L = a.N <= 64 ? 4 : a.N <= 128 ? 8 : 16, kc = 2;
+  if ((long long)a.B * a.H * a.P <= 148 * 32) {
+    kc = 1;
+    while (L < 16 && a.N > 4 * L) L *= 2;
+  }
+  const int need = (a.N + 4 * L - 1) / (4 * L);
+  return {L, need <= 1 ? 1 : need <= 2 ? 2 : need <= 4 ? 4 : 8, kc};
+}
+
+template <int L, int KC>
+cudaError_t scan(const HeadDeltaArgs& a, const ScanShape& f, cudaStream_t s) {
+  constexpr int PB = kScanThreads / 32 * KC * (32 / L);
+  auto go = [&](auto k) -> cudaError_t {
+    const size_t smem = 2 * (size_t)kGroupsStaged * (2 * C * a.NP + C * PB + C * kCoef) * sizeof(float);
     const cudaError_t e = allow_smem(k, smem);
     if (e != cudaSuccess) return e;
-    k<<<dim3(a.B, a.H, (a.P + PB - 1) / PB), 32 * warps, smem, s>>>(a);
+    k<<<dim3(a.B, a.H, (a.P + PB - 1) / PB), kScanThreads, smem, s>>>(a);
     return last();
   };
-  if (need <= 1) return go(head_delta_scan_kernel<L, 1>, 1);
-  if (need <= 2) return go(head_delta_scan_kernel<L, 2>, 2);
-  if (need <= 4) return go(head_delta_scan_kernel<L, 4>, 4);
-  if (need <= 8) return go(head_delta_scan_kernel<L, 8>, 8);
-  return cudaErrorInvalidValue;
+  if (f.nr4 == 1) return go(head_delta_scan_kernel<L, 1, KC>);
+  if (f.nr4 == 2) return go(head_delta_scan_kernel<L, 2, KC>);
+  if (f.nr4 == 4) return go(head_delta_scan_kernel<L, 4, KC>);
+  return go(head_delta_scan_kernel<L, 8, KC>);
 }
 
 }  // namespace
@@ -433,27 +486,25 @@ bool head_delta_supported(int N) { return N >= 1 && N <= 512; }
 
 long long head_delta_workspace(const HeadDeltaArgs& a, int max_q) {
   int vw, lw;
-  return step_form(a, max_q, vw, lw) ? 0 : (long long)(a.T / C + a.B) * group_floats(a.G, a.H, a.N, a.P);
+  if (step_form(a, max_q, vw, lw)) return 0;
+  const ScanShape f = scan_shape(a);
+  return (long long)(a.T / C + a.B) * group_floats(a.G, a.H, 4 * f.L * f.nr4, a.P);
 }
 
-cudaError_t head_delta_launch(const HeadDeltaArgs& a, bool f32, int max_q, cudaStream_t s) {
+cudaError_t head_delta_launch(HeadDeltaArgs a, bool f32, int max_q, cudaStream_t s) {
   if (a.G < 1 || a.H % a.G != 0 || a.P < 1 || !head_delta_supported(a.N) || a.G > 3000) return cudaErrorInvalidValue;
   int vw, lw;
   if (step_form(a, max_q, vw, lw)) {
     if (vw == 4) AT_DISPATCH(f32, return (step<AT, 4>(a, lw, s)));
     AT_DISPATCH(f32, return (step<AT, 1>(a, lw, s)));
   }
-  if (a.pre == nullptr) return cudaErrorInvalidValue;
+  if (a.pre == nullptr || (reinterpret_cast<uintptr_t>(a.pre) & 15) != 0) return cudaErrorInvalidValue;
+  const ScanShape f = scan_shape(a);
+  a.NP = 4 * f.L * f.nr4;
   cudaError_t e = cudaSuccess;
   AT_DISPATCH(f32, e = prepare<AT>(a, s));
   if (e != cudaSuccess) return e;
-  // few lanes per column mean few shuffles, many mean short products and more CTAs: spread while the grid leaves SMs idle
-  int L = a.N <= 128 ? 4 : a.N <= 256 ? 8 : 16;
-  auto ctas = [&](int lanes) { const int pb = 4 * (32 / lanes); return (long long)a.B * a.H * ((a.P + pb - 1) / pb); };
-  while (L < 16 && ctas(L) < 148 && a.N > 4 * L) L *= 2;
-  const int cpw = 32 / L;
-  int warps = (a.P + cpw - 1) / cpw;
-  if (warps > 4) warps = 4;
-  return L == 4 ? scan<4>(a, warps, s) : L == 8 ? scan<8>(a, warps, s) : scan<16>(a, warps, s);
+  if (f.kc == 1) return f.L == 4 ? scan<4, 1>(a, f, s) : f.L == 8 ? scan<8, 1>(a, f, s) : scan<16, 1>(a, f, s);
+  return f.L == 4 ? scan<4, 2>(a, f, s) : f.L == 8 ? scan<8, 2>(a, f, s) : scan<16, 2>(a, f, s);
 }
 }  // namespace b200

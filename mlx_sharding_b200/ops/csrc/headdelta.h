@@ -15,9 +15,10 @@ struct HeadDeltaArgs {
   int B, T, H, G, N, P;
   float q_scale, unit_eps;
   float* pre;                               // head_delta_workspace floats (portions), unused by steps of single tokens
+  int NP;                                   // row width of the workspace (set by the launcher)
 };
 bool head_delta_supported(int N);
 // floats of workspace of a step whose longest portion has max_q tokens (0: none)
 long long head_delta_workspace(const HeadDeltaArgs& a, int max_q);
-cudaError_t head_delta_launch(const HeadDeltaArgs& a, bool f32, int max_q, cudaStream_t s);
+cudaError_t head_delta_launch(HeadDeltaArgs a, bool f32, int max_q, cudaStream_t s);
 }  // namespace b200

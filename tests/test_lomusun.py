@@ -191,7 +191,7 @@ def decays(dt, bias, A_log):
 @pytest.mark.parametrize("device,dtype,tol", DEVICES)
 @pytest.mark.parametrize("H,G,D,V,portions", [(4, 2, 6, 10, [13, 1, 9]), (3, 3, 5, 7, [2, 3, 1, 4, 5]), (2, 1, 128, 128, [40, 1, 2, 7]), (2, 2, 64, 40, [33, 1, 1]), (1, 1, 200, 16, [11, 1]),
                                               (4, 4, 33, 65, [1, 2, 30]), (8, 4, 16, 32, [70, 1, 5]), (2, 1, 300, 8, [9, 1]), (1, 1, 512, 4, [6, 1]), (1, 1, 530, 4, [6, 1]), (2, 1, 1, 3, [5, 1]),
-                                              (64, 32, 24, 8, [17, 1])])
+                                              (64, 32, 24, 8, [17, 1]), (40, 8, 20, 128, [9, 1, 6]), (40, 4, 100, 131, [7, 2]), (40, 2, 130, 120, [6, 3]), (3, 1, 70, 6, [10])])
 def test_delta_rule_alone(H, G, D, V, portions, device, dtype, tol):
     """The rule as an op: one sequence in portions that start inside a group of four tokens, the state carried in a dirty slot that must not be
     read at the first token; every lane layout of the kernels, sizes that are no multiple of 4, heads that share queries and keys."""
