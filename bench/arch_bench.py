@@ -655,6 +655,10 @@ def lomusun_kernel_table(width, dev, hbm):
         name = f"sigmoid_topk(correction, normalised) {phase}"
         add(name, timed(lambda: O.sigmoid_topk(z, E, k, corr, True, 1.5)), T * E * 4 + T * k * 8)
         add(f"group_softmax_topk (Gokapel) {phase}", timed(lambda: O.group_softmax_topk(z, corr, E, k, 4, 2)), T * E * 4 + T * k * 8, like=name)
+        rbytes = T * W * 2 + E * W * 4 + T * k * 8
+        name = f"sigmoid_router(product and choice) {phase}"
+        add(name, timed(lambda: O.sigmoid_router(xa, rw, E, k, corr, True, 1.5)), rbytes)
+        add(f"router_logits + group_softmax_topk (Gokapel) {phase}", timed(lambda: O.group_softmax_topk(O.router_logits(xa, rw), corr, E, k, 4, 2)), rbytes, like=name)
         idx, wts = O.sigmoid_topk(z, E, k, corr, True, 1.5)
         wg, wu = (LinearWeight(weight=(rn(E, F, W) * W ** -0.5).to(bf)) for _ in range(2))
         wd = LinearWeight(weight=(rn(E, W, F) * F ** -0.5).to(bf))
