@@ -3,7 +3,7 @@
 Kernel sources are plain CUDA (no torch headers) compiled by nvcc with
 ``-gencode arch=compute_100a,code=sm_100a -lineinfo``; only ``bindings.cpp`` sees torch.  nvcc
 cross-compiles without a GPU, so this runs on the CPU build box; the resulting ``.so`` travels to the
-GPU box with the repo snapshot (it is git-ignored, not gpurun-ignored).
+GPU box with the repo snapshot (it is git-ignored).
 
 ``python -m mlx_sharding_b200.ops.build [--force] [--verbose]``
 """

@@ -49,7 +49,7 @@ B200_DEVICE bool mbar_try_wait(uint64_t* bar, uint32_t parity) {
       : "memory");
   return ok != 0;
 }
-// Bounded wait: a protocol bug must trap (kernel error), never hang the GPU (gpurun strike policy).
+// Bounded wait: a protocol bug must trap (kernel error), never hang the GPU.
 B200_DEVICE void mbar_wait(uint64_t* bar, uint32_t parity) {
   uint32_t spins = 0;
   while (!mbar_try_wait(bar, parity)) {
